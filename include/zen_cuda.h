@@ -37,8 +37,8 @@ extern "C" {
 #pragma GCC visibility push(default)
 #endif
 
-/* GGML tensor type ids of the three formats on the path (GGUF tensor directory). */
-enum { ZEN_CUDA_Q4_0 = 2, ZEN_CUDA_Q8_0 = 8, ZEN_CUDA_Q6_K = 14, ZEN_CUDA_Q4_K = 12, ZEN_CUDA_Q5_K = 13 };
+/* GGML tensor type ids of the formats on the path (GGUF tensor directory). */
+enum { ZEN_CUDA_Q4_0 = 2, ZEN_CUDA_Q8_0 = 8, ZEN_CUDA_Q6_K = 14, ZEN_CUDA_Q4_K = 12, ZEN_CUDA_Q5_K = 13, ZEN_CUDA_BF16 = 30 };
 
 /* How activations enter the integer dot products.
  *   ZEN_CUDA_ACT_INT8 : one int8 code per element, bit-identical to the reference's
@@ -479,6 +479,114 @@ int zen_cuda_dev_attention_prefill(const float* d_q, const float* d_k_cache, con
 int zen_cuda_dev_silu_mul(const float* d_gate, const float* d_up, float* d_out, size_t count, void* stream);
 /* *d_pos += delta, in stream order (a step's last launch). */
 int zen_cuda_dev_advance_position(int* d_pos, int delta, void* stream);
+
+/* ---- bfloat16 decoders: dense products with bf16 matrices (zen_cuda_dev_upload with ZEN_CUDA_BF16, [rows][columns] row-major) and
+ * the operators of models with grouped norms, token shifts, windowed attention and recurrent state.  Vectors and rows are fp32
+ * unless a parameter says otherwise; "bf16" flags choose the element type of a product's input rows (pitch in elements). ---- */
+
+/* The end of a sublayer, per row of n values: x_new = x_in + norm(y) (x_in alone when y_a is NULL).  y = y_a; with y_b,
+ * y = (rms(y_a) * weight_a + rms(y_b) * weight_b) / 2.  norm: `groups` equal consecutive parts, each divided by
+ * sqrt(mean(part^2) + eps), the whole times norm_weight.  The row's reader sees x_new + (before - x_new) * shift (before: the
+ * previous row's x_new; the block's first row reads `before`), or with out_norm the grouped norm of x_new times out_norm, or x_new.
+ * x_out: where x_new goes (not x_in itself), or NULL.  keep: receives the last row of x_in, or NULL. */
+typedef struct zen_cuda_sublayer_end {
+    const float* x_in;
+    float* x_out;
+    const float* y_a;
+    const float* y_b;
+    const float* weight_a;
+    const float* weight_b;
+    const float* norm_weight;
+    float* keep;
+    const float* shift;
+    const float* before;
+    const float* out_norm;
+    uint32_t n, groups;
+    float eps;
+} zen_cuda_sublayer_end;
+int zen_cuda_dev_sublayer_end_rows(const zen_cuda_sublayer_end* end, size_t rows, void* d_view, size_t view_ld, int view_bf16, void* stream);
+
+/* Activations of a dense product's outputs: none, max(z, 0)^2, cap * tanh(z / cap). */
+enum { ZEN_CUDA_DENSE_PLAIN = 0, ZEN_CUDA_DENSE_SQUARED_RELU = 1, ZEN_CUDA_DENSE_SOFTCAP = 2 };
+#define ZEN_CUDA_DENSE_MAX_TASKS 4
+typedef struct zen_cuda_dense_task {
+    const zen_cuda_weights* w;
+    const float* d_x;          /* [columns]; ignored when the call carries a sublayer end */
+    float* d_y;                /* [rows] */
+    int act;
+    float cap;
+} zen_cuda_dense_task;
+/* One launch: d_y = act(W x) for every task, fp32 activations.  pre (or NULL): the input of the single task is what the sublayer
+ * end's reader sees, formed inside the launch. */
+int zen_cuda_dev_dense_gemv(const zen_cuda_dense_task* tasks, size_t count, const zen_cuda_sublayer_end* pre, void* stream);
+/* d_out[t][r] = act(sum_k x[t][k] w[r][k]) for a block of tokens.  exact 0: x is bf16 (16-byte aligned, pitch a multiple of 8) and the
+ * product runs on the tensor cores with fp32 accumulation; exact 1: x is fp32 and so is every multiply-add.  out_bf16: d_out is
+ * bf16 (exact 0 only). */
+int zen_cuda_dev_dense_gemm(const zen_cuda_weights* w, const void* d_x, size_t x_ld, size_t tokens, void* d_out, size_t out_ld, int out_bf16, int act,
+                            float cap, int exact, void* stream);
+
+/* d_out[t] = embed[tokens[t]] + positions[*d_pos + t]; positions NULL: the embedding alone. */
+int zen_cuda_dev_embed_rows_bf16(const zen_cuda_weights* embed, const zen_cuda_weights* positions, const int64_t* d_tokens, size_t tokens, const int* d_pos,
+                                 float* d_out, void* stream);
+/* Columns [0, n) of rows of pitch src_ld as a product's input [rows][ld], zeros behind them. */
+int zen_cuda_dev_rows_view(const float* d_src, size_t src_ld, size_t n, size_t rows, void* d_dst, size_t ld, int bf16, void* stream);
+/* Heads of `width` values (pitch head_ld in d_o) -> a product's input: each head divided by its root mean square and times weight
+ * (weight NULL: no norm), times sigmoid(gate): gate_mode 0 none, 1 one per head, 2 one per value (rows of pitch gate_ld). */
+int zen_cuda_dev_head_outputs_rows(const float* d_o, size_t rows, size_t heads, size_t width, size_t head_ld, const float* d_weight, float eps,
+                                   const float* d_gate, size_t gate_ld, int gate_mode, void* d_dst, size_t ld, int bf16, void* stream);
+
+/* Windowed attention with kept first tokens: position i sees j <= i when i - j < window or j < keep_first; bias != 0 takes
+ * slope_h * (i - j) off the scores, slope_h = 2^(-8 (h + 1) / heads).  q and k are RMS-normed per head (q_weight, k_weight, eps).
+ * Caches [max_positions][kv_heads][pitch], pitch = max(qk_dim, v_dim) rounded up to 32, at most 256. */
+typedef struct zen_cuda_window_attention {
+    uint32_t heads, kv_heads, qk_dim, v_dim, pitch;
+    uint32_t window, keep_first, bias, max_positions;
+    float scale, eps;
+    const float* q_weight;
+    const float* k_weight;
+    float* k_cache;
+    float* v_cache;
+} zen_cuda_window_attention;
+/* A block of rows: q, k, v are columns of the projection rows (pitch ld).  Norms q and k, appends k and v at *d_pos .., and
+ * attends; d_q and d_out are [tokens][heads][pitch]. */
+int zen_cuda_dev_window_attention_rows(const zen_cuda_window_attention* a, const float* d_proj_q, const float* d_proj_k, const float* d_proj_v, size_t ld,
+                                       size_t tokens, const int* d_pos, float* d_q, float* d_out, void* stream);
+/* One token in one launch; d_out [heads][v_dim], times sigmoid(d_gate[h]) when d_gate is given. */
+int zen_cuda_dev_window_attention_step(const zen_cuda_window_attention* a, const float* d_q, const float* d_k, const float* d_v, const float* d_gate,
+                                       const int* d_pos, float* d_out, void* stream);
+
+/* Mixers with a matrix state S [dim][vdim] per head, kept as [heads][vdim][pitch] fp32, pitch = dim rounded up to 32.
+ *   delta rule   S <- g * S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  q, k, v pass a causal convolution of `taps` taps per
+ *                channel and silu (ring [taps][2 kv_heads dim + heads vdim], slot = position mod taps), q and k become unit vectors
+ *                (q also times dim^-1/2), beta = sigmoid, g = exp(-exp(a_log) softplus(a2 a1 + dt_bias)); output gate sigmoid(g2 g1).
+ *   gated write  S <- f * S + (1 - f) v^T; o = S^T q; q = silu, f = lower + (1 - lower) sigmoid(. + f_bias).
+ * norm [vdim]: weight of the output's RMS norm per head.  dim and vdim at most 256. */
+typedef struct zen_cuda_linear_layer {
+    uint32_t heads, kv_heads, dim, vdim, taps;
+    float eps;
+    const float* conv;
+    const float* a_log;
+    const float* dt_bias;
+    const zen_cuda_weights* a2;
+    const zen_cuda_weights* g2;
+    const float* f_bias;
+    const float* lower;
+    const float* norm;
+    float* ring;
+    float* state;
+} zen_cuda_linear_layer;
+/* One token, from the projections to the output projection's input [heads * vdim], in one launch.
+ * d_proj: q | k | v | b | a1 | g1 (delta) or q | f | v (gated write). */
+int zen_cuda_dev_state_step(const zen_cuda_linear_layer* l, int delta, const float* d_proj, const int* d_pos, float* d_out, void* stream);
+/* A block: the scan's inputs from the projection rows.  Delta rule: d_q, d_k [tokens][kv_heads][pitch], d_g [tokens][heads][pitch],
+ * d_v [tokens][heads * vdim], d_beta [tokens][heads]; d_decay [tokens][decay_ld] = a2 a1 without the bias; the ring is brought up to date. */
+int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, const float* d_decay, size_t decay_ld, size_t tokens,
+                                   const int* d_pos, float* d_q, float* d_k, float* d_g, float* d_v, float* d_beta, void* stream);
+/* Gated write: d_q, d_f [tokens][heads][pitch]. */
+int zen_cuda_dev_gated_write_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, size_t tokens, float* d_q, float* d_f, void* stream);
+/* The recurrence over the block: d_out [tokens][heads][vdim].  d_v: rows of pitch v_ld.  d_k and d_beta: delta rule only. */
+int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int delta, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld,
+                            const float* d_beta, size_t tokens, float* d_out, void* stream);
 
 /* The device-side error channel.  Synchronises `stream` (NULL: the backend's own), then reads and clears the error word
  * the kernels set.  Returns

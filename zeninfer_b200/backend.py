@@ -24,7 +24,7 @@ _PKG = os.path.dirname(os.path.abspath(__file__))
 _LIB_PATH = os.path.join(_PKG, "lib", "libzen_cuda.so")
 
 ACT_INT8, ACT_FP32 = 1, 2
-FORMAT_IDS = {"Q8_0": blocks.Q8_0, "Q4_0": blocks.Q4_0, "Q6_K": blocks.Q6_K, "Q4_K": blocks.Q4_K, "Q5_K": blocks.Q5_K}
+FORMAT_IDS = {"Q8_0": blocks.Q8_0, "Q4_0": blocks.Q4_0, "Q6_K": blocks.Q6_K, "Q4_K": blocks.Q4_K, "Q5_K": blocks.Q5_K, "BF16": blocks.BF16}
 
 # every symbol include/zen_cuda.h declares; the CPU test-suite checks the library exports them all
 ABI_SYMBOLS = (
@@ -46,6 +46,9 @@ ABI_SYMBOLS = (
     "zen_cuda_dev_embed_q8_0", "zen_cuda_dev_rms_norm", "zen_cuda_dev_rope_kv_append", "zen_cuda_dev_attention", "zen_cuda_dev_silu_mul",
     "zen_cuda_dev_advance_position", "zen_cuda_dev_gemv_swiglu", "zen_cuda_dev_attention_block", "zen_cuda_dev_gemv_fused",
     "zen_cuda_dev_embed_rows_q8_0", "zen_cuda_dev_rope_kv_append_rows", "zen_cuda_dev_attention_prefill",
+    "zen_cuda_dev_sublayer_end_rows", "zen_cuda_dev_dense_gemv", "zen_cuda_dev_dense_gemm", "zen_cuda_dev_embed_rows_bf16", "zen_cuda_dev_rows_view",
+    "zen_cuda_dev_head_outputs_rows", "zen_cuda_dev_window_attention_rows", "zen_cuda_dev_window_attention_step", "zen_cuda_dev_state_step",
+    "zen_cuda_dev_delta_inputs_rows", "zen_cuda_dev_gated_write_inputs_rows", "zen_cuda_dev_state_scan",
 )
 
 
@@ -86,6 +89,28 @@ class GemvListItem(C.Structure):
 
 class PickSegment(C.Structure):
     _fields_ = [("base", C.c_void_p), ("len", C.c_uint32), ("first_index", C.c_uint32), ("token_stride", C.c_uint32), ("reserved", C.c_uint32)]
+
+
+DENSE_PLAIN, DENSE_SQUARED_RELU, DENSE_SOFTCAP = 0, 1, 2
+
+
+class SublayerEnd(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x_in", "x_out", "y_a", "y_b", "weight_a", "weight_b", "norm_weight", "keep", "shift", "before", "out_norm")] + [
+        ("n", C.c_uint32), ("groups", C.c_uint32), ("eps", C.c_float)]
+
+
+class DenseTask(C.Structure):
+    _fields_ = [("w", C.c_void_p), ("d_x", C.c_void_p), ("d_y", C.c_void_p), ("act", C.c_int), ("cap", C.c_float)]
+
+
+class WindowAttention(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "qk_dim", "v_dim", "pitch", "window", "keep_first", "bias", "max_positions")] + [
+        ("scale", C.c_float), ("eps", C.c_float)] + [(n, C.c_void_p) for n in ("q_weight", "k_weight", "k_cache", "v_cache")]
+
+
+class LinearLayer(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "taps")] + [("eps", C.c_float)] + [
+        (n, C.c_void_p) for n in ("conv", "a_log", "dt_bias", "a2", "g2", "f_bias", "lower", "norm", "ring", "state")]
 
 
 def load_library(path: str | None = None) -> C.CDLL:
@@ -184,6 +209,18 @@ def load_library(path: str | None = None) -> C.CDLL:
     lib.zen_cuda_dev_attention_prefill.argtypes = [vp, vp, vp, vp, vp, sz, sz, sz, sz, C.c_float, sz, sz, vp]
     lib.zen_cuda_dev_attention_block.argtypes = [vp, vp, vp, vp, vp, sz, vp, vp, vp, vp, sz, sz, sz, C.c_float, sz, sz, vp]
     lib.zen_cuda_dev_advance_position.argtypes = [vp, i, vp]
+    lib.zen_cuda_dev_sublayer_end_rows.argtypes = [C.POINTER(SublayerEnd), sz, vp, sz, i, vp]
+    lib.zen_cuda_dev_dense_gemv.argtypes = [C.POINTER(DenseTask), sz, C.POINTER(SublayerEnd), vp]
+    lib.zen_cuda_dev_dense_gemm.argtypes = [vp, vp, sz, sz, vp, sz, i, i, C.c_float, i, vp]
+    lib.zen_cuda_dev_embed_rows_bf16.argtypes = [vp, vp, vp, sz, vp, vp, vp]
+    lib.zen_cuda_dev_rows_view.argtypes = [vp, sz, sz, sz, vp, sz, i, vp]
+    lib.zen_cuda_dev_head_outputs_rows.argtypes = [vp, sz, sz, sz, sz, vp, C.c_float, vp, sz, i, vp, sz, i, vp]
+    lib.zen_cuda_dev_window_attention_rows.argtypes = [C.POINTER(WindowAttention), vp, vp, vp, sz, sz, vp, vp, vp, vp]
+    lib.zen_cuda_dev_window_attention_step.argtypes = [C.POINTER(WindowAttention), vp, vp, vp, vp, vp, vp, vp]
+    lib.zen_cuda_dev_state_step.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp]
+    lib.zen_cuda_dev_delta_inputs_rows.argtypes = [C.POINTER(LinearLayer), vp, sz, vp, sz, sz, vp, vp, vp, vp, vp, vp, vp]
+    lib.zen_cuda_dev_gated_write_inputs_rows.argtypes = [C.POINTER(LinearLayer), vp, sz, sz, vp, vp, vp]
+    lib.zen_cuda_dev_state_scan.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp, sz, vp, sz, vp, vp]
     return lib
 
 
@@ -583,6 +620,66 @@ class Backend:
     def dev_advance_position(self, d_pos: int, delta: int = 1, stream: int = 0) -> None:
         if not self.lib.zen_cuda_dev_advance_position(d_pos, delta, stream):
             self._fail("dev_advance_position")
+
+    # ---- bfloat16 decoders (the structures are the header's; addresses are plain ints) ----
+    def dev_sublayer_end_rows(self, end: SublayerEnd, rows: int, d_view: int | None, view_ld: int, view_bf16: bool, stream: int = 0) -> None:
+        """The residual add with its grouped norm over a block of rows, and the next product's input."""
+        if not self.lib.zen_cuda_dev_sublayer_end_rows(C.byref(end), rows, d_view, view_ld, int(view_bf16), stream):
+            self._fail("dev_sublayer_end_rows")
+
+    def dev_dense_gemv(self, tasks: Sequence[tuple[int, int | None, int]], stream: int = 0, *, pre: SublayerEnd | None = None, act: int = DENSE_PLAIN,
+                       cap: float = 0.0) -> None:
+        """One launch of bf16 products with single fp32 vectors: (handle, d_x, d_y) each; pre: the input is formed inside."""
+        arr = (DenseTask * len(tasks))(*[DenseTask(h, x, y, act, cap) for h, x, y in tasks])
+        if not self.lib.zen_cuda_dev_dense_gemv(arr, len(tasks), C.byref(pre) if pre is not None else None, stream):
+            self._fail("dev_dense_gemv")
+
+    def dev_dense_gemm(self, handle: int, d_x: int, x_ld: int, tokens: int, d_out: int, out_ld: int, stream: int = 0, *, out_bf16: bool = False,
+                       act: int = DENSE_PLAIN, cap: float = 0.0, exact: bool = False) -> None:
+        """A bf16 matrix times a block of tokens: bf16 rows on the tensor cores, or (exact) fp32 rows in fp32 multiply-adds."""
+        if not self.lib.zen_cuda_dev_dense_gemm(handle, d_x, x_ld, tokens, d_out, out_ld, int(out_bf16), act, cap, int(exact), stream):
+            self._fail("dev_dense_gemm")
+
+    def dev_embed_rows_bf16(self, embed: int, positions: int | None, d_tokens: int, tokens: int, d_pos: int, d_out: int, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_embed_rows_bf16(embed, positions, d_tokens, tokens, d_pos, d_out, stream):
+            self._fail("dev_embed_rows_bf16")
+
+    def dev_rows_view(self, d_src: int, src_ld: int, n: int, rows: int, d_dst: int, ld: int, bf16: bool, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_rows_view(d_src, src_ld, n, rows, d_dst, ld, int(bf16), stream):
+            self._fail("dev_rows_view")
+
+    def dev_head_outputs_rows(self, d_o: int, rows: int, heads: int, width: int, head_ld: int, d_dst: int, ld: int, bf16: bool, stream: int = 0, *,
+                              weight: int | None = None, eps: float = 0.0, gate: int | None = None, gate_ld: int = 0, gate_mode: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_head_outputs_rows(d_o, rows, heads, width, head_ld, weight, eps, gate, gate_ld, gate_mode, d_dst, ld, int(bf16), stream):
+            self._fail("dev_head_outputs_rows")
+
+    def dev_window_attention_rows(self, a: WindowAttention, d_q: int, d_k: int, d_v: int, ld: int, tokens: int, d_pos: int, d_q_normed: int, d_out: int,
+                                  stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_window_attention_rows(C.byref(a), d_q, d_k, d_v, ld, tokens, d_pos, d_q_normed, d_out, stream):
+            self._fail("dev_window_attention_rows")
+
+    def dev_window_attention_step(self, a: WindowAttention, d_q: int, d_k: int, d_v: int, d_gate: int | None, d_pos: int, d_out: int, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_window_attention_step(C.byref(a), d_q, d_k, d_v, d_gate, d_pos, d_out, stream):
+            self._fail("dev_window_attention_step")
+
+    def dev_state_step(self, layer: LinearLayer, delta: bool, d_proj: int, d_pos: int, d_out: int, stream: int = 0) -> None:
+        """One token through a mixer with a matrix state: from its projections to its output projection's input."""
+        if not self.lib.zen_cuda_dev_state_step(C.byref(layer), int(delta), d_proj, d_pos, d_out, stream):
+            self._fail("dev_state_step")
+
+    def dev_delta_inputs_rows(self, layer: LinearLayer, d_proj: int, ld: int, d_decay: int, decay_ld: int, tokens: int, d_pos: int, d_q: int, d_k: int,
+                              d_g: int, d_v: int, d_beta: int, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_delta_inputs_rows(C.byref(layer), d_proj, ld, d_decay, decay_ld, tokens, d_pos, d_q, d_k, d_g, d_v, d_beta, stream):
+            self._fail("dev_delta_inputs_rows")
+
+    def dev_gated_write_inputs_rows(self, layer: LinearLayer, d_proj: int, ld: int, tokens: int, d_q: int, d_f: int, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_gated_write_inputs_rows(C.byref(layer), d_proj, ld, tokens, d_q, d_f, stream):
+            self._fail("dev_gated_write_inputs_rows")
+
+    def dev_state_scan(self, layer: LinearLayer, delta: bool, d_q: int, d_k: int | None, d_g: int, d_v: int, v_ld: int, d_beta: int | None, tokens: int,
+                       d_out: int, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_state_scan(C.byref(layer), int(delta), d_q, d_k, d_g, d_v, v_ld, d_beta, tokens, d_out, stream):
+            self._fail("dev_state_scan")
 
     def dev_check(self, stream: int = 0) -> None:
         """Synchronises `stream` and raises if a kernel reported through the device-side error word (a bounded wait that

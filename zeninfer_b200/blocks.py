@@ -22,6 +22,7 @@ from __future__ import annotations
 import numpy as np
 
 Q8_0, Q4_0, Q6_K, Q4_K, Q5_K = 8, 2, 14, 12, 13  # GGML type ids
+BF16 = 30                                        # not a block format: rows of bfloat16, packed and decoded below
 BLOCK_ELEMENTS = {Q8_0: 32, Q4_0: 32, Q6_K: 256, Q4_K: 256, Q5_K: 256}
 BLOCK_BYTES = {Q8_0: 34, Q4_0: 18, Q6_K: 210, Q4_K: 144, Q5_K: 176}
 NAMES = {Q8_0: "Q8_0", Q4_0: "Q4_0", Q6_K: "Q6_K", Q4_K: "Q4_K", Q5_K: "Q5_K"}
@@ -198,3 +199,14 @@ def dequantize(fmt: int, packed: np.ndarray, rows: int, columns: int) -> np.ndar
         ms = (dmin * mn)[..., None]
         return (ds * q.astype(np.float32) - ms).reshape(rows, columns)
     raise ValueError(fmt)
+
+
+def to_bf16(w: np.ndarray) -> np.ndarray:
+    """fp32 -> bfloat16 bit patterns (uint16), round to nearest even; finite values only."""
+    u = np.ascontiguousarray(w, np.float32).view(np.uint32)
+    return ((u + np.uint32(0x7FFF) + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def from_bf16(bits: np.ndarray) -> np.ndarray:
+    """bfloat16 bit patterns (uint16) -> fp32, exact."""
+    return (np.ascontiguousarray(bits, np.uint16).astype(np.uint32) << 16).view(np.float32)

@@ -5,7 +5,9 @@
 """
 from __future__ import annotations
 
+import fcntl
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -13,12 +15,13 @@ import sys
 PKG = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(PKG, "csrc")
 LIB_DIR = os.path.join(PKG, "lib")
+OBJ_DIR = os.path.join(LIB_DIR, "obj")
 LIB = os.path.join(LIB_DIR, "libzen_cuda.so")
 INCLUDE = os.path.join(os.path.dirname(PKG), "include")
 
 NVCC_FLAGS = [
     "-std=c++17", "-O3", "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo",
-    "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden", "-shared",
+    "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
 ]
 
 
@@ -26,25 +29,55 @@ def _sources() -> list[str]:
     return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
 
 
-def _newest_input() -> float:
-    files = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(INCLUDE, "zen_cuda.h")]
-    return max(os.path.getmtime(f) for f in files)
+def _inputs(source: str) -> set[str]:
+    """A translation unit and everything of this repository it includes."""
+    seen, todo = set(), [source]
+    while todo:
+        path = os.path.normpath(todo.pop())
+        if path in seen or not os.path.exists(path):
+            continue
+        seen.add(path)
+        with open(path) as f:
+            todo += [os.path.join(os.path.dirname(path), name) for name in re.findall(r'^#include "([^"]+)"', f.read(), re.M)]
+    return seen
+
+
+def _stale(target: str, inputs) -> bool:
+    return not os.path.exists(target) or os.path.getmtime(target) < max(os.path.getmtime(f) for f in inputs)
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
-    """Returns the path of the built library; raises if nvcc is missing or compilation fails."""
-    if not force and os.path.exists(LIB) and os.path.getmtime(LIB) >= _newest_input():
+    """Returns the path of the built library; raises if nvcc is missing or compilation fails.  Translation units are compiled
+    side by side, and only those whose sources changed; processes that ask for the library at the same time build it once."""
+    inputs = {src: _inputs(src) for src in _sources()}
+    everything = set().union(*inputs.values())
+    if not force and not _stale(LIB, everything):
         return LIB
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not os.path.exists(nvcc):
         if os.path.exists(LIB):
             return LIB  # a prebuilt library travelled with the tree
         raise RuntimeError("nvcc not found and no prebuilt libzen_cuda.so")
-    os.makedirs(LIB_DIR, exist_ok=True)
-    cmd = [nvcc, *NVCC_FLAGS, "-I", INCLUDE, "-o", LIB, *_sources()]
-    if verbose:
-        cmd.insert(1, "-Xptxas=-v")
-    subprocess.run(cmd, check=True)
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not force and not _stale(LIB, everything):
+            return LIB
+        flags = ["-Xptxas=-v", *NVCC_FLAGS] if verbose else NVCC_FLAGS
+        jobs, objects = [], []
+        for src, needs in inputs.items():
+            obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
+            objects.append(obj)
+            if force or _stale(obj, needs):
+                cmd = [nvcc, *flags, "-I", INCLUDE, "-c", "-o", obj, src]
+                jobs.append((cmd, subprocess.Popen(cmd)))
+        codes = [(cmd, job.wait()) for cmd, job in jobs]
+        for cmd, code in codes:
+            if code:
+                raise subprocess.CalledProcessError(code, cmd)
+        fresh = LIB + ".new"
+        subprocess.run([nvcc, *NVCC_FLAGS, "-shared", "-o", fresh, *objects], check=True)
+        os.replace(fresh, LIB)
     return LIB
 
 

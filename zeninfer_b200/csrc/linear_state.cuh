@@ -1,0 +1,418 @@
+// Mixers with a matrix state per head, S [dim][vdim] in fp32, carried from token to token:
+//
+//   delta rule    S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q      (g per key channel)
+//   gated write   S <- f * S + (1 - f) v^T;           o = S^T q                       (f per key channel, no key)
+//
+// state_scan_kernel walks a block of tokens with the state in registers, state_step_kernel takes one token and does everything
+// between the layer's input projections and its output projection.  The kernels around the scan form its inputs (short causal
+// convolution, unit norms, decays, gates) for all tokens at once.
+//
+// Device layout of a state: [heads][vdim][pitch], pitch = dim rounded up to 32 and zero beyond dim, so that eight lanes read a
+// column's rows as consecutive 16-byte words.  The convolution keeps the inputs of the last `taps` tokens in a ring
+// [taps][channels] whose slot is the position modulo taps: a token reads the taps - 1 slots before its own and nobody else
+// writes those, so it needs no second buffer.
+#pragma once
+#include "gemv_bf16.cuh"
+
+namespace zk {
+
+__device__ __forceinline__ float silu_f(float z) { return z * logistic(z); }
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z + log1pf(expf(-z)) : log1pf(expf(z)); }
+constexpr float kUnitEps = 1e-6f;
+
+struct LinearLayer {
+    uint32_t heads, kv_heads, dim, vdim, pitch;
+    uint32_t taps;                 // delta rule: convolution taps
+    uint32_t rank_a, rank_g;       // delta rule: ranks of the decay's and the output gate's projections
+    uint32_t a2_ld, g2_ld;
+    const float* conv;             // [2 kv_heads dim + heads vdim][taps]: q, k, v channels
+    const float* a_log;            // [heads]
+    const float* dt_bias;          // [heads][dim]
+    const __nv_bfloat16* a2;       // [heads dim][a2_ld]
+    const __nv_bfloat16* g2;       // [heads vdim][g2_ld]
+    const float* f_bias;           // gated write: [heads][dim]
+    const float* lower;            // gated write: [heads][dim]
+    const float* norm;             // [vdim]
+    float* ring;                   // [taps][channels]
+    float* state;                  // [heads][vdim][pitch]
+    float eps;
+};
+__host__ __device__ inline uint32_t linear_channels(const LinearLayer& l) { return 2 * l.kv_heads * l.dim + l.heads * l.vdim; }
+
+// Convolution of channel c at block row t (position pos + t), then silu.  x: projection rows of pitch ld, channel c at column c;
+// rows before the block come from the ring, tokens before the sequence's start are zeros.
+__device__ __forceinline__ float conv_silu(const LinearLayer& l, const float* __restrict__ x, uint32_t ld, int t, int pos, uint32_t c, uint32_t channels) {
+    float y = 0.0f;
+    for (uint32_t j = 0; j < l.taps; ++j) {
+        const int back = static_cast<int>(l.taps - 1 - j), s = t - back, at = pos + s;
+        if (at < 0) continue;
+        const float v = s >= 0 ? __ldcg(x + static_cast<size_t>(s) * ld + c) : l.ring[static_cast<size_t>(static_cast<uint32_t>(at) % l.taps) * channels + c];
+        y = fmaf(l.conv[static_cast<size_t>(c) * l.taps + j], v, y);
+    }
+    return silu_f(y);
+}
+
+// ---- inputs of the scan for a block of tokens -------------------------------------------------------------------------
+
+// Delta rule.  proj [T][ld]: q | k | v | b columns; decay [T][heads dim] = W_a2 W_a1 h.  One CTA per token.
+//   q, k [T][kv_heads][pitch] unit vectors (q also times dim^-1/2), g [T][heads][pitch], v [T][heads vdim], beta [T][heads].
+__global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld,
+                                                                const float* __restrict__ decay, uint32_t decay_ld, const int* __restrict__ pos_ptr,
+                                                                float* __restrict__ q, float* __restrict__ k, float* __restrict__ g, float* __restrict__ v,
+                                                                float* __restrict__ beta) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = static_cast<int>(blockIdx.x), pos = *pos_ptr;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, channels = linear_channels(l), kd = l.kv_heads * l.dim;
+    for (uint32_t i = warp; i < 2 * l.kv_heads; i += 8) {          // a warp takes a q or k head
+        const bool is_q = i < l.kv_heads;
+        const uint32_t head = is_q ? i : i - l.kv_heads, c0 = (is_q ? 0u : kd) + head * l.dim;
+        float* dst = (is_q ? q : k) + (static_cast<size_t>(t) * l.kv_heads + head) * l.pitch;
+        float val[8], ss = 0.0f;                                   // pitch <= 256
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const uint32_t d = lane + 32 * j;
+            val[j] = d < l.dim ? conv_silu(l, proj, ld, t, pos, c0 + d, channels) : 0.0f;
+            ss += val[j] * val[j];
+        }
+        float inv = 1.0f / sqrtf(warp_sum(ss) + kUnitEps);
+        if (is_q) inv *= 1.0f / sqrtf(static_cast<float>(l.dim));
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (lane + 32 * j < l.pitch) dst[lane + 32 * j] = val[j] * inv;
+    }
+    for (uint32_t i = threadIdx.x; i < l.heads * l.vdim; i += 256) v[static_cast<size_t>(t) * l.heads * l.vdim + i] = conv_silu(l, proj, ld, t, pos, 2 * kd + i, channels);
+    for (uint32_t i = threadIdx.x; i < l.heads; i += 256) beta[static_cast<size_t>(t) * l.heads + i] = logistic(proj[static_cast<size_t>(t) * ld + channels + i]);
+    for (uint32_t i = threadIdx.x; i < l.heads * l.pitch; i += 256) {
+        const uint32_t h = i / l.pitch, d = i % l.pitch;
+        float gate = 0.0f;
+        if (d < l.dim) gate = expf(-expf(l.a_log[h]) * softplus_f(decay[static_cast<size_t>(t) * decay_ld + h * l.dim + d] + l.dt_bias[h * l.dim + d]));
+        g[static_cast<size_t>(t) * l.heads * l.pitch + i] = gate;
+    }
+}
+
+// The ring after a block of T tokens: the inputs of its last min(T, taps) tokens.  Runs after the kernel above.
+__global__ void __launch_bounds__(256) conv_ring_update_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld, uint32_t tokens,
+                                                               const int* __restrict__ pos_ptr) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t channels = linear_channels(l), c = blockIdx.x * 256 + threadIdx.x, pos = static_cast<uint32_t>(*pos_ptr);
+    if (c >= channels) return;
+    for (uint32_t t = tokens > l.taps ? tokens - l.taps : 0; t < tokens; ++t)
+        l.ring[static_cast<size_t>((pos + t) % l.taps) * channels + c] = proj[static_cast<size_t>(t) * ld + c];
+}
+
+// Gated write.  proj [T][ld]: q | f columns.  q, f [T][heads][pitch]; f = 1 beyond dim (the padding neither decays nor writes).
+__global__ void __launch_bounds__(256) gated_write_inputs_rows_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld,
+                                                                      float* __restrict__ q, float* __restrict__ f) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    for (uint32_t i = threadIdx.x; i < l.heads * l.pitch; i += 256) {
+        const uint32_t h = i / l.pitch, d = i % l.pitch, c = h * l.dim + d;
+        float qv = 0.0f, fv = 1.0f;
+        if (d < l.dim) {
+            qv = silu_f(proj[t * ld + c]);
+            fv = l.lower[c] + (1.0f - l.lower[c]) * logistic(proj[t * ld + l.heads * l.dim + c] + l.f_bias[c]);
+        }
+        q[t * l.heads * l.pitch + i] = qv;
+        f[t * l.heads * l.pitch + i] = fv;
+    }
+}
+
+// ---- the scan --------------------------------------------------------------------------------------------------------
+
+struct ScanParams {
+    const float* q;        // [T][q_heads][pitch]
+    const float* k;        // [T][q_heads][pitch]; delta rule only
+    const float* g;        // [T][heads][pitch]
+    const float* v;        // [T][v_ld], head h's values at column h * vdim
+    const float* beta;     // [T][heads]; delta rule only
+    float* state;          // [heads][vdim][pitch]
+    float* out;            // [T][heads][vdim]
+    uint32_t tokens, heads, q_heads, vdim, v_ld;
+};
+
+constexpr int kScanThreads = 128, kScanColumns = 32, kScanTokens = 8;    // columns of S per CTA; tokens per staged block
+template <int kQuads, bool kDelta>
+__host__ __device__ constexpr uint32_t scan_token_floats() { return (kDelta ? 3 : 2) * kQuads * 32 + kScanColumns + 4; }
+template <int kQuads, bool kDelta>
+__host__ __device__ constexpr uint32_t scan_smem_bytes() { return 2 * kScanTokens * scan_token_floats<kQuads, kDelta>() * 4; }
+
+__device__ __forceinline__ void cp_async_4(float* smem_dst, const float* gmem_src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst))), "l"(gmem_src) : "memory");
+}
+
+// A CTA takes 32 columns of one head's state (its value channels), a warp eight of them.  A column's rows are spread over eight
+// lanes, lane `part` holding the 16-byte words part, part + 8, ...; a lane holds two columns, so a word of q, k or g read from
+// shared memory serves both.  The state never leaves the registers between the block's first and last token; arithmetic is packed
+// fp32 pairs.  kQuads = pitch / 32.  Grid: (ceil(vdim / 32), heads).
+template <int kQuads, bool kDelta>
+__global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_constant__ ScanParams p) {
+    constexpr uint32_t kPitch = kQuads * 32, kToken = scan_token_floats<kQuads, kDelta>();
+    constexpr uint32_t kG = 0, kQ = kPitch, kK = 2 * kPitch, kV = (kDelta ? 3 : 2) * kPitch, kB = kV + kScanColumns;
+    extern __shared__ __align__(16) float scan_smem[];
+    pdl_launch_dependents();
+    const uint32_t h = blockIdx.y, qh = h / (p.heads / p.q_heads), col_base = blockIdx.x * kScanColumns;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7;
+    const uint32_t local = warp * 8 + (lane >> 3) * 2, c0 = col_base + local;      // this lane's columns: c0, c0 + 1
+    const bool on0 = c0 < p.vdim, on1 = c0 + 1 < p.vdim;
+    pdl_wait();
+    uint64_t s[2][kQuads][2];
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const float* src = p.state + (static_cast<size_t>(h) * p.vdim + c0 + c) * kPitch + part * 4;
+#pragma unroll
+        for (int i = 0; i < kQuads; ++i) {
+            const float4 w = (c ? on1 : on0) ? __ldcg(reinterpret_cast<const float4*>(src + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            s[c][i][0] = pf_pack(w.x, w.y);
+            s[c][i][1] = pf_pack(w.z, w.w);
+        }
+    }
+    auto stage = [&](uint32_t t0, uint32_t buf) {
+        float* dst = scan_smem + buf * kScanTokens * kToken;
+        const uint32_t n = min(static_cast<uint32_t>(kScanTokens), p.tokens - t0);
+        constexpr uint32_t kWords = kPitch / 4, kRows = kDelta ? 3 : 2;
+        for (uint32_t i = threadIdx.x; i < n * kRows * kWords; i += kScanThreads) {
+            const uint32_t t = i / (kRows * kWords), rest = i % (kRows * kWords), row = rest / kWords, word = rest % kWords;
+            const float* src = row == 0 ? p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch
+                                        : (row == 1 ? p.q : p.k) + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch;
+            cp_async_16(dst + t * kToken + row * kPitch + word * 4, src + word * 4, 16);
+        }
+        for (uint32_t i = threadIdx.x; i < n * kScanColumns; i += kScanThreads) {
+            const uint32_t t = i / kScanColumns, c = i % kScanColumns;
+            float* d = dst + t * kToken + kV + c;
+            if (col_base + c < p.vdim) cp_async_4(d, p.v + static_cast<size_t>(t0 + t) * p.v_ld + h * p.vdim + col_base + c); else *d = 0.0f;
+        }
+        if (kDelta && threadIdx.x < n) cp_async_4(dst + threadIdx.x * kToken + kB, p.beta + static_cast<size_t>(t0 + threadIdx.x) * p.heads + h);
+        cp_async_commit();
+    };
+    const uint64_t zero2 = pf_pack(0.0f, 0.0f);
+    stage(0, 0);
+    uint32_t buf = 0;
+    for (uint32_t t0 = 0; t0 < p.tokens; t0 += kScanTokens, buf ^= 1u) {
+        const bool more = t0 + kScanTokens < p.tokens;
+        if (more) stage(t0 + kScanTokens, buf ^ 1u);
+        if (more) cp_async_wait<1>(); else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t n = min(static_cast<uint32_t>(kScanTokens), p.tokens - t0);
+        const float* tok = scan_smem + buf * kScanTokens * kToken;
+#pragma unroll 2
+        for (uint32_t t = 0; t < n; ++t, tok += kToken) {
+            uint64_t g[kQuads][2], q[kQuads][2], k[kQuads][2];
+#pragma unroll
+            for (int i = 0; i < kQuads; ++i) {
+                const float4 a = reinterpret_cast<const float4*>(tok + kG)[i * 8 + part], b = reinterpret_cast<const float4*>(tok + kQ)[i * 8 + part];
+                g[i][0] = pf_pack(a.x, a.y); g[i][1] = pf_pack(a.z, a.w);
+                q[i][0] = pf_pack(b.x, b.y); q[i][1] = pf_pack(b.z, b.w);
+                if (kDelta) {
+                    const float4 c = reinterpret_cast<const float4*>(tok + kK)[i * 8 + part];
+                    k[i][0] = pf_pack(c.x, c.y); k[i][1] = pf_pack(c.z, c.w);
+                } else {
+                    k[i][0] = pf_pack(1.0f - a.x, 1.0f - a.y); k[i][1] = pf_pack(1.0f - a.z, 1.0f - a.w);
+                }
+            }
+            const float2 v2 = *reinterpret_cast<const float2*>(tok + kV + local);
+            float u[2] = {v2.x, v2.y};
+            if (kDelta) {
+                const float beta = tok[kB];
+                float dot[2];
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    uint64_t d0 = zero2, d1 = zero2;
+#pragma unroll
+                    for (int i = 0; i < kQuads; ++i) {
+                        s[c][i][0] = pf_mul(s[c][i][0], g[i][0]);
+                        s[c][i][1] = pf_mul(s[c][i][1], g[i][1]);
+                        d0 = pf_fma(s[c][i][0], k[i][0], d0);
+                        d1 = pf_fma(s[c][i][1], k[i][1], d1);
+                    }
+                    float a, b, e, f;
+                    pf_unpack(d0, a, b);
+                    pf_unpack(d1, e, f);
+                    dot[c] = (a + b) + (e + f);
+                }
+#pragma unroll
+                for (int o = 1; o < 8; o <<= 1) {
+                    dot[0] += __shfl_xor_sync(0xffffffffu, dot[0], o);
+                    dot[1] += __shfl_xor_sync(0xffffffffu, dot[1], o);
+                }
+                u[0] = beta * (u[0] - dot[0]);
+                u[1] = beta * (u[1] - dot[1]);
+            }
+            float out[2];
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const uint64_t uu = pf_pack(u[c], u[c]);
+                uint64_t d0 = zero2, d1 = zero2;
+#pragma unroll
+                for (int i = 0; i < kQuads; ++i) {
+                    if (kDelta) {
+                        s[c][i][0] = pf_fma(k[i][0], uu, s[c][i][0]);
+                        s[c][i][1] = pf_fma(k[i][1], uu, s[c][i][1]);
+                    } else {
+                        s[c][i][0] = pf_fma(k[i][0], uu, pf_mul(s[c][i][0], g[i][0]));
+                        s[c][i][1] = pf_fma(k[i][1], uu, pf_mul(s[c][i][1], g[i][1]));
+                    }
+                    d0 = pf_fma(s[c][i][0], q[i][0], d0);
+                    d1 = pf_fma(s[c][i][1], q[i][1], d1);
+                }
+                float a, b, e, f;
+                pf_unpack(d0, a, b);
+                pf_unpack(d1, e, f);
+                out[c] = (a + b) + (e + f);
+            }
+            // the two columns' sums over eight lanes: odd lanes end with column c0 + 1, even lanes with c0
+            const bool odd = part & 1;
+            float o = (odd ? out[1] : out[0]) + __shfl_xor_sync(0xffffffffu, odd ? out[0] : out[1], 1);
+            o += __shfl_xor_sync(0xffffffffu, o, 2);
+            o += __shfl_xor_sync(0xffffffffu, o, 4);
+            if (part < 2 && (part ? on1 : on0)) p.out[(static_cast<size_t>(t0 + t) * p.heads + h) * p.vdim + c0 + part] = o;
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        float* dst = p.state + (static_cast<size_t>(h) * p.vdim + c0 + c) * kPitch + part * 4;
+        if (!(c ? on1 : on0)) continue;
+#pragma unroll
+        for (int i = 0; i < kQuads; ++i) {
+            float4 w;
+            pf_unpack(s[c][i][0], w.x, w.y);
+            pf_unpack(s[c][i][1], w.z, w.w);
+            *reinterpret_cast<float4*>(dst + i * 32) = w;
+        }
+    }
+}
+
+// ---- one token -------------------------------------------------------------------------------------------------------
+
+// One CTA per head: everything from the projections of one token to the output projection's input.  proj: delta rule
+// q | k | v | b | a1 | g1, gated write q | f | v.  out [heads][vdim].
+constexpr int kStepThreads = 512;
+template <bool kDelta>
+__global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj,
+                                                                  const int* __restrict__ pos_ptr, float* __restrict__ out) {
+    constexpr uint32_t kWarps = kStepThreads / 32;
+    __shared__ __align__(16) float q[256], k[256], g[256];
+    __shared__ float v[256], o[256], gate[256];
+    const uint32_t h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7, quads = l.pitch / 32;
+    pdl_launch_dependents();
+    pdl_wait();
+    // the first columns' state words are on their way while the token's vectors are formed
+    float* const state = l.state + static_cast<size_t>(h) * l.vdim * l.pitch + part * 4;
+    uint32_t col = warp * 4 + (lane >> 3);
+    float4 pre[8];
+#pragma unroll
+    for (uint32_t i = 0; i < 8; ++i)
+        pre[i] = (i < quads && col < l.vdim) ? __ldcg(reinterpret_cast<const float4*>(state + static_cast<size_t>(col) * l.pitch + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    float beta = 0.0f;
+    if (kDelta) {
+        const int pos = *pos_ptr;
+        const uint32_t channels = linear_channels(l), kd = l.kv_heads * l.dim, qh = h / (l.heads / l.kv_heads);
+        const float* low_a = proj + channels + l.heads;
+        const float* low_g = low_a + l.rank_a;
+        beta = logistic(__ldcg(proj + channels + h));
+        const bool owner = h % (l.heads / l.kv_heads) == 0;        // one CTA per q/k head keeps its ring
+        float* slot = l.ring + static_cast<size_t>(static_cast<uint32_t>(pos) % l.taps) * channels;
+        for (uint32_t i = threadIdx.x; i < 2 * l.pitch + l.vdim; i += kStepThreads) {
+            const bool is_v = i >= 2 * l.pitch, is_k = !is_v && i >= l.pitch;
+            const uint32_t d = is_v ? i - 2 * l.pitch : is_k ? i - l.pitch : i;
+            float y = 0.0f;
+            if (is_v || d < l.dim) {
+                const uint32_t c = is_v ? 2 * kd + h * l.vdim + d : (is_k ? kd : 0u) + qh * l.dim + d;
+                y = conv_silu(l, proj, 0, 0, pos, c, channels);
+                if (is_v || owner) slot[c] = __ldcg(proj + c);
+            }
+            (is_v ? v : is_k ? k : q)[d] = y;
+        }
+        // decays and output gate: rows of the rank projections, eight lanes to a row
+        const float a_scale = -expf(l.a_log[h]);
+        for (uint32_t r0 = warp * 4; r0 < l.pitch + l.vdim; r0 += kWarps * 4) {
+            const uint32_t r = r0 + (lane >> 3);
+            const bool is_g = r >= l.pitch;                        // a row of the gate
+            const uint32_t d = is_g ? r - l.pitch : r, ld = is_g ? l.g2_ld : l.a2_ld, rank = is_g ? l.rank_g : l.rank_a;
+            const bool live = is_g ? d < l.vdim : d < l.dim;
+            const __nv_bfloat16* w = is_g ? l.g2 + static_cast<size_t>(h * l.vdim + d) * ld : l.a2 + static_cast<size_t>(h * l.dim + d) * ld;
+            const float* low = is_g ? low_g : low_a;
+            float acc = 0.0f;
+            if (live)
+                for (uint32_t c = part * 8; c < ld; c += 64) {
+                    const uint4 ww = __ldg(reinterpret_cast<const uint4*>(w + c));
+                    float x[8];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) x[j] = c + j < rank ? __ldcg(low + c + j) : 0.0f;
+                    dense_fma8(ww, x, acc);
+                }
+#pragma unroll
+            for (int s = 1; s < 8; s <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, s);
+            if (part == 0) {
+                if (is_g) { if (live) gate[d] = logistic(acc); }
+                else g[d] = live ? expf(a_scale * softplus_f(acc + l.dt_bias[h * l.dim + d])) : 0.0f;
+            }
+        }
+        __syncthreads();
+        if (warp < 2) {                                            // unit norms: warp 0 takes q, warp 1 k
+            float* x = warp ? k : q;
+            float ss = 0.0f;
+            for (uint32_t d = lane; d < l.pitch; d += 32) ss += x[d] * x[d];
+            float inv = 1.0f / sqrtf(warp_sum(ss) + kUnitEps);
+            if (!warp) inv *= 1.0f / sqrtf(static_cast<float>(l.dim));
+            for (uint32_t d = lane; d < l.pitch; d += 32) x[d] *= inv;
+        }
+    } else {
+        for (uint32_t d = threadIdx.x; d < l.pitch; d += kStepThreads) {
+            const uint32_t c = h * l.dim + d;
+            float qv = 0.0f, fv = 1.0f;
+            if (d < l.dim) {
+                qv = silu_f(__ldcg(proj + c));
+                fv = l.lower[c] + (1.0f - l.lower[c]) * logistic(__ldcg(proj + l.heads * l.dim + c) + l.f_bias[c]);
+            }
+            q[d] = qv;
+            g[d] = fv;
+            k[d] = 1.0f - fv;
+        }
+        for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) v[i] = __ldcg(proj + 2 * l.heads * l.dim + h * l.vdim + i);
+    }
+    __syncthreads();
+    // a warp takes four columns at a time, eight lanes to a column
+    for (uint32_t base = warp * 4; base < l.vdim; base += kWarps * 4) {
+        col = base + (lane >> 3);
+        const bool on = col < l.vdim;
+        float* mine = state + static_cast<size_t>(col) * l.pitch;
+        float4 s[8];
+        float u = on ? v[col] : 0.0f, dot = 0.0f;
+#pragma unroll
+        for (uint32_t i = 0; i < 8; ++i) {
+            if (i >= quads) break;
+            s[i] = base == warp * 4 ? pre[i] : on ? __ldcg(reinterpret_cast<const float4*>(mine + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 gg = reinterpret_cast<const float4*>(g)[i * 8 + part], kk = reinterpret_cast<const float4*>(k)[i * 8 + part];
+            s[i] = make_float4(s[i].x * gg.x, s[i].y * gg.y, s[i].z * gg.z, s[i].w * gg.w);
+            if (kDelta) dot += s[i].x * kk.x + s[i].y * kk.y + s[i].z * kk.z + s[i].w * kk.w;
+        }
+        if (kDelta) {
+#pragma unroll
+            for (int b = 1; b < 8; b <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, b);
+            u = beta * (u - dot);
+        }
+        float acc = 0.0f;
+#pragma unroll
+        for (uint32_t i = 0; i < 8; ++i) {
+            if (i >= quads) break;
+            const float4 qq = reinterpret_cast<const float4*>(q)[i * 8 + part], kk = reinterpret_cast<const float4*>(k)[i * 8 + part];
+            s[i] = make_float4(fmaf(kk.x, u, s[i].x), fmaf(kk.y, u, s[i].y), fmaf(kk.z, u, s[i].z), fmaf(kk.w, u, s[i].w));
+            acc += s[i].x * qq.x + s[i].y * qq.y + s[i].z * qq.z + s[i].w * qq.w;
+            if (on) *reinterpret_cast<float4*>(mine + i * 32) = s[i];
+        }
+#pragma unroll
+        for (int b = 1; b < 8; b <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, b);
+        if (on && part == 0) o[col] = acc;
+    }
+    __syncthreads();
+    float ss = 0.0f;
+    for (uint32_t i = lane; i < l.vdim; i += 32) ss += o[i] * o[i];          // every warp forms the head's norm itself
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(l.vdim) + l.eps);
+    for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) out[h * l.vdim + i] = o[i] * inv * l.norm[i] * (kDelta ? gate[i] : 1.0f);
+}
+
+}  // namespace zk

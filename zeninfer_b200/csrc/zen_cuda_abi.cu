@@ -32,6 +32,7 @@
 #include "gemv_list.cuh"
 #include "gemv_q8_0.cuh"
 #include "greedy_pick.cuh"
+#include "host_state.h"
 #include "quantize_acts.cuh"
 #include "repack.cuh"
 #include "sample_pick.cuh"
@@ -48,23 +49,6 @@ struct zen_cuda_gemv_list {
     int digits{};
     size_t smem{};
     uint64_t algorithmic_bytes{};  // raw GGUF bytes of all tensors + fp32 inputs and outputs
-};
-
-struct zen_cuda_weights {
-    int format{};
-    size_t rows{}, cols{};
-    uint32_t nb{}, nbp{};     // blocks per row, padded to 8
-    void* plane[4]{};         // format-specific planes (see repack.cuh)
-    void* d_tile_maps{};      // Q8_0 rows of several K segments: zk::GemvTileMaps in device memory (see make_tile_maps), else null
-    int kernel_format{};      // what the decode kernel is instantiated for: the format, or zk::kFormatQ6KCodes for Q6_K with unpacked codes
-    // Two-digit planes under one scale per 256 weights (gemm_groups.cuh), built at the tensor's first many-row product and
-    // kept: wh, wl [rows][cols] int8, units [rows][cols / 256] fp32.
-    mutable void* g_hi{};
-    mutable void* g_lo{};
-    mutable float* g_unit{};
-    mutable size_t g_bytes{};
-    size_t device_bytes{};
-    size_t raw_bytes{};
 };
 
 namespace {
@@ -166,6 +150,7 @@ bool opted_out() {
 bool apply_wait_budget(State& s, unsigned ms) {
     const long long cycles = ms ? static_cast<long long>(ms) * std::max(1, s.clock_khz) : zk::kDefaultWaitBudgetCycles;
     ZC_CUDA(s, cudaMemcpyToSymbol(zk::g_wait_budget_cycles, &cycles, sizeof cycles));
+    if (!zk_host::set_dense_wait_budget(cycles)) return set_error(s, "setting the dense kernels' wait budget failed");
     return true;
 }
 
@@ -314,8 +299,43 @@ void plane_sizes(int fmt, size_t nrows, size_t cols, size_t plane_bytes[4], bool
 bool make_tile_maps(State& s, zen_cuda_weights* w);   // defined with the other tensor-map code below
 bool make_kq_tile_maps(State& s, zen_cuda_weights* w);
 
+// A bfloat16 matrix: one plane [rows][ld], ld = cols rounded up to eight elements (16 bytes), zero beyond cols.
+zen_cuda_weights* upload_bf16_locked(State& s, const uint8_t* host, size_t rows_total, size_t cols, size_t first_row, size_t nrows) {
+    if (!host || !nrows || !cols || first_row + nrows > rows_total || nrows > 0x7fffffffu || cols > 0x7ffffff0u) {
+        set_error(s, "upload: bad shape");
+        return nullptr;
+    }
+    const auto t0 = clock_type::now();
+    auto* w = new zen_cuda_weights;
+    w->format = w->kernel_format = ZEN_CUDA_BF16;
+    w->rows = nrows; w->cols = cols;
+    w->nbp = static_cast<uint32_t>((cols + 7) & ~size_t(7));
+    w->raw_bytes = nrows * cols * 2;
+    w->device_bytes = nrows * static_cast<size_t>(w->nbp) * 2;
+    bool ok = cudaMalloc(&w->plane[0], w->device_bytes) == cudaSuccess;
+    if (ok && w->nbp == cols) {
+        ok = stream_to_device(s, w->plane[0], host + first_row * cols * 2, w->raw_bytes);
+    } else if (ok) {
+        ok = cudaMemsetAsync(w->plane[0], 0, w->device_bytes, s.copy_stream) == cudaSuccess &&
+             cudaMemcpy2DAsync(w->plane[0], static_cast<size_t>(w->nbp) * 2, host + first_row * cols * 2, cols * 2, cols * 2, nrows, cudaMemcpyHostToDevice,
+                               s.copy_stream) == cudaSuccess;
+    }
+    ok = ok && cudaStreamSynchronize(s.copy_stream) == cudaSuccess;
+    if (!ok) {
+        set_error(s, std::string("upload: ") + cudaGetErrorString(cudaGetLastError()));
+        if (w->plane[0]) cudaFree(w->plane[0]);
+        delete w;
+        return nullptr;
+    }
+    s.stats.upload_bytes += w->raw_bytes;
+    s.stats.weight_bytes += w->device_bytes;
+    s.stats.upload_us += us_since(t0);
+    return w;
+}
+
 // Uploads rows [first_row, first_row+nrows) and re-lays them out into planes on the device.
 zen_cuda_weights* upload_locked(State& s, int fmt, const uint8_t* host, size_t rows_total, size_t cols, size_t first_row, size_t nrows) {
+    if (fmt == ZEN_CUDA_BF16) return upload_bf16_locked(s, host, rows_total, cols, first_row, nrows);
     const uint32_t be = block_elems(fmt), bb = block_bytes(fmt);
     if (!bb || !host || !nrows || !cols || cols % be || first_row + nrows > rows_total) {
         set_error(s, "upload: bad shape or format");
@@ -1794,6 +1814,26 @@ bool host_ffn(State& s, const uint8_t* gate, const uint8_t* up, const uint8_t* d
 
 }  // namespace
 
+// What the bfloat16 and linear-state entry points (zen_cuda_dense.cu) share with this file.
+namespace zk_host {
+Entry::Entry(void* stream_arg) : lock(state().mutex), ok(false), stream{}, d_error{}, encode_tiled{}, sm_count{}, smem_optin{}, pdl{} {
+    State& s = state();
+    if (!init_locked(s)) return;
+    ok = true;
+    stream = stream_arg ? static_cast<cudaStream_t>(stream_arg) : s.stream;
+    d_error = s.d_error;
+    encode_tiled = s.encode_tiled;
+    sm_count = s.sm_count;
+    smem_optin = s.smem_optin;
+    pdl = s.pdl;
+}
+int Entry::fail(const std::string& why) { set_error(state(), why); return 0; }
+int Entry::leave(cudaError_t e, const char* what) {
+    ++state().stats.dispatches;
+    return e == cudaSuccess ? 1 : fail(std::string(what) + ": " + cudaGetErrorString(e));
+}
+}  // namespace zk_host
+
 extern "C" {
 
 int zen_cuda_enabled(void) {
@@ -2457,11 +2497,11 @@ bool enqueue_attention(State& s, cudaStream_t st, bool fused, const float* d_q, 
     auto launch = [&](auto kernel) {
         return fused ? launch_pdl(s, kernel, grid, block, smem, st, d_q, static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), d_pos, d_out,
                                   static_cast<uint32_t>(heads), static_cast<uint32_t>(kv_heads), static_cast<uint32_t>(head_dim), scale, static_cast<uint32_t>(window),
-                                  static_cast<uint32_t>(max_positions), s.d_error, d_k, d_v, d_cos, d_sin, static_cast<uint32_t>(pairs), d_k_cache, d_v_cache)
+                                  static_cast<uint32_t>(max_positions), s.d_error, d_k, d_v, d_cos, d_sin, static_cast<uint32_t>(pairs), d_k_cache, d_v_cache, zk::AttnWindow{})
                      : launch_pdl(s, kernel, grid, block, smem, st, d_q, static_cast<const float*>(d_k_cache), static_cast<const float*>(d_v_cache), d_pos, d_out,
                                   static_cast<uint32_t>(heads), static_cast<uint32_t>(kv_heads), static_cast<uint32_t>(head_dim), scale, static_cast<uint32_t>(window),
                                   static_cast<uint32_t>(max_positions), s.d_error, static_cast<const float*>(nullptr), static_cast<const float*>(nullptr),
-                                  static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), 0u, static_cast<float*>(nullptr), static_cast<float*>(nullptr));
+                                  static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), 0u, static_cast<float*>(nullptr), static_cast<float*>(nullptr), zk::AttnWindow{});
     };
     const cudaError_t e = fused ? (wide ? launch(zk::attention_decode_kernel<true, true>) : launch(zk::attention_decode_kernel<true, false>))
                                 : (wide ? launch(zk::attention_decode_kernel<false, true>) : launch(zk::attention_decode_kernel<false, false>));
@@ -2532,7 +2572,7 @@ int zen_cuda_dev_attention_prefill(const float* d_q, const float* d_k_cache, con
             done = true;
         }
         return launch_pdl(s, kernel, grid, block, smem, st, d_q, d_k_cache, d_v_cache, d_pos, d_out, static_cast<uint32_t>(tokens), static_cast<uint32_t>(heads),
-                          static_cast<uint32_t>(kv_heads), scale, static_cast<uint32_t>(window), static_cast<uint32_t>(max_positions), s.d_error);
+                          static_cast<uint32_t>(kv_heads), scale, static_cast<uint32_t>(window), static_cast<uint32_t>(max_positions), s.d_error, zk::AttnWindow{});
     };
     auto by_heads = [&](auto dim) {
         constexpr int kD = decltype(dim)::value;

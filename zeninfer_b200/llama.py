@@ -33,6 +33,7 @@ import numpy as np
 
 from . import blocks
 from .backend import ACT_FP32, ACT_INT8, Backend
+from .decoder import Decoder
 
 
 @dataclass(frozen=True)
@@ -102,7 +103,7 @@ def rope_tables(cfg: LlamaConfig, positions: int) -> tuple[np.ndarray, np.ndarra
     return np.cos(angle).astype(np.float32), np.sin(angle).astype(np.float32)
 
 
-class LlamaDecoder:
+class LlamaDecoder(Decoder):
     """Holds the resident model and the step's device buffers.  `tensors` yields (name, array, is_matrix) as
     synthetic_tensors does; matrices must be Q8_0 raw blocks [rows, row_bytes]."""
 
@@ -127,7 +128,7 @@ class LlamaDecoder:
         with act_mode=ACT_INT8 reproduces it (prompt blocks go through the two-digit tensor-core product, leftover prompt
         tokens one by one outside the step graphs)."""
         import torch
-        self.torch, self.be, self.cfg, self.act_mode = torch, backend, cfg, act_mode
+        self.cfg, self.act_mode = cfg, act_mode
         self.prompt_act_mode = prompt_act_mode if prompt_act_mode not in (None, act_mode) else None
         self.fuse = "nsr" if fused is True else "" if fused is False else str(fused)
         if "p" in self.fuse and "s" in self.fuse:
@@ -150,9 +151,7 @@ class LlamaDecoder:
                 raise ValueError(f"cut = {cut!r}")
         self.col_cut = self.world > 1 and cut == "rows+cols"
         self.gather_kind, self.peer = gather if self.world > 1 else "none", None
-        self.dev = device if device is not None else torch.device("cuda", torch.cuda.current_device())
-        self.max_positions = max_positions or cfg.context
-        self.stream = torch.cuda.Stream(device=self.dev)
+        self._init_runtime(backend, cfg.vocab, max_positions or cfg.context, device)
         self.h: dict[str, int] = {}        # matrix name -> resident handle
         self.norm: dict[str, "torch.Tensor"] = {}
         shapes = {name: shape for name, shape, _ in tensor_plan(cfg)}
@@ -180,9 +179,8 @@ class LlamaDecoder:
         self.x, self.xn, self.tmp = torch.zeros(E, **f32), torch.zeros(E, **f32), torch.zeros(E, **f32)
         self.q, self.k, self.v, self.att = torch.zeros(QW // w, **f32), torch.zeros(KW // w, **f32), torch.zeros(KW // w, **f32), torch.zeros(QW, **f32)
         self.gate, self.up, self.hid = torch.zeros(F // w, **f32), torch.zeros(F // w, **f32), torch.zeros(F, **f32)
-        self.logits = torch.zeros(V, **f32)
-        self.k_cache = torch.zeros((cfg.layers, self.max_positions, KW // w), **f32)
-        self.v_cache = torch.zeros((cfg.layers, self.max_positions, KW // w), **f32)
+        self.k_cache = self.sequence.add("k", (cfg.layers, self.max_positions, KW // w))
+        self.v_cache = self.sequence.add("v", (cfg.layers, self.max_positions, KW // w))
         mine = lambda t: t[self.rank * (t.numel() // w):(self.rank + 1) * (t.numel() // w)]     # the piece this rank's rows produce
         self.x_mine, self.att_mine, self.hid_mine, self.logits_mine = mine(self.x), mine(self.att), mine(self.hid), mine(self.logits)
         if self.gather_kind == "peer":
@@ -191,10 +189,6 @@ class LlamaDecoder:
             self.peer = shard.PeerGather(backend, w, self.rank, (slot + 3) & ~3, group=group)     # collective: handles travel through the group
         cos, sin = rope_tables(cfg, self.max_positions)
         self.cos, self.sin = torch.from_numpy(cos).to(self.dev), torch.from_numpy(sin).to(self.dev)
-        self.pos = torch.zeros(1, dtype=torch.int32, device=self.dev)
-        self.token = torch.zeros(1, dtype=torch.int64, device=self.dev)
-        self.host_token = torch.zeros(1, dtype=torch.int64).pin_memory()   # generate() feeds every step from the host, as the reference does
-        self.graph_layers = self.graph_head = None
 
     @classmethod
     def from_gguf(cls, backend: Backend, path: str, **kwargs) -> "LlamaDecoder":
@@ -286,48 +280,7 @@ class LlamaDecoder:
         self._gather(self.logits, self.logits_mine)
         self.be.dev_greedy_pick([(self.logits.data_ptr(), self.cfg.vocab, 0, self.cfg.vocab)], 1, self.token.data_ptr(), self.stream.cuda_stream)
 
-    def capture(self) -> None:
-        """Runs one throw-away step (kernel attributes are set on first launch), then captures the two graphs."""
-        torch = self.torch
-        self.sync_ranks()
-        with torch.cuda.stream(self.stream):
-            self.reset()
-            self._enqueue_layers()
-            self._enqueue_head()
-            self.stream.synchronize()
-            self.graph_layers, self.graph_head = torch.cuda.CUDAGraph(), torch.cuda.CUDAGraph()
-            # with collectives in the graph, other threads of the process (the collective library's watchdog) may call
-            # the runtime during the capture: only this thread's calls belong to it
-            mode = dict(capture_error_mode="thread_local") if self.world > 1 else {}
-            with torch.cuda.graph(self.graph_layers, stream=self.stream, **mode):
-                self._enqueue_layers()
-            with torch.cuda.graph(self.graph_head, stream=self.stream, **mode):
-                self._enqueue_head()
-            self.stream.synchronize()
-        self.reset()
-
-    def reset(self) -> None:
-        with self.torch.cuda.stream(self.stream):
-            self.pos.zero_()
-            self.token.zero_()
-        self.stream.synchronize()
-
-    def step(self, want_token: bool) -> None:
-        """Consumes the token in self.token at position self.pos; with want_token the pick replaces self.token."""
-        with self.torch.cuda.stream(self.stream):
-            if self.graph_layers is not None:
-                self.graph_layers.replay()
-                if want_token:
-                    self.graph_head.replay()
-            else:
-                self._enqueue_layers()
-                if want_token:
-                    self._enqueue_head()
-
     # ---- prefill: a block of prompt tokens through the tensor-core products ----
-    PREFILL_CHUNK = 512     # tokens per block (buffers are sized for it)
-    PREFILL_MIN = 16        # shorter blocks go token by token
-
     def _prefill_buffers(self):
         if getattr(self, "_pf", None) is None:
             torch, cfg, T, w = self.torch, self.cfg, self.PREFILL_CHUNK, self.world
@@ -437,77 +390,29 @@ class LlamaDecoder:
             self.token.copy_(self.block_picks[tail_count - 1:tail_count])
         return self.block_logits[:tail_count]
 
-    def feed_prompt(self, prompt: list[int], batched_prefill: bool | None = None) -> None:
-        """Enqueues the whole prompt from position self.pos on, ending with the first pick (left in self.token).  Blocks of
-        at least PREFILL_MIN tokens go through prefill() when batched_prefill (default: wherever can_prefill_blocks()), the
-        rest token by token."""
-        torch = self.torch
-        ids = torch.tensor(prompt, dtype=torch.int64).pin_memory()
-        if batched_prefill is None:
-            batched_prefill = self.can_prefill_blocks()
-        with torch.cuda.stream(self.stream):
-            done = 0
-            if batched_prefill and len(prompt) >= self.PREFILL_MIN:
-                d_ids = ids.to(self.dev, non_blocking=True)
-                while len(prompt) - done >= self.PREFILL_MIN:
-                    n = min(self.PREFILL_CHUNK, len(prompt) - done)
-                    self.prefill(d_ids[done:done + n], n)
-                    done += n
-                if done == len(prompt):
-                    self._enqueue_head()      # the first pick, from the last prompt token's hidden state
-            for i in range(done, len(prompt)):
-                self.token.copy_(ids[i:i + 1], non_blocking=True)
-                last = i + 1 == len(prompt)
-                if self.prompt_act_mode is None:
-                    self.step(want_token=last)
-                    continue
-                decode_mode, self.act_mode = self.act_mode, self.prompt_act_mode
-                try:
-                    self._enqueue_layers()            # eager: the captured graphs hold the decode mode
-                finally:
-                    self.act_mode = decode_mode
-                if last:
-                    self._enqueue_head()              # a single-token product: the decode mode
+    def _prompt_token(self, last: bool) -> None:
+        if self.prompt_act_mode is None:
+            self.step(want_token=last)
+            return
+        decode_mode, self.act_mode = self.act_mode, self.prompt_act_mode
+        try:
+            self._enqueue_layers()            # eager: the captured graphs hold the decode mode
+        finally:
+            self.act_mode = decode_mode
+        if last:
+            self._enqueue_head()              # a single-token product: the decode mode
 
-    def _sample(self, temperature: float, top_k: int, top_p: float, u: float) -> None:
-        """Replaces the greedy pick in self.token by a draw from the filtered distribution of self.logits."""
-        self.be.dev_sample(self.logits.data_ptr(), self.cfg.vocab, temperature, top_k, top_p, u, self.token.data_ptr(), self.stream.cuda_stream)
-
-    def generate(self, prompt: list[int], max_new: int, on_token=None, batched_prefill: bool | None = None, temperature: float = 0.0,
-                 top_k: int = 0, top_p: float = 1.0, seed: int = 0) -> list[int]:
-        """Generation: the prompt, then max_new picks (each read back, as the reference's per-token callback does).  With
-        temperature <= 0 the picks are greedy; otherwise every token is drawn on the device from the temperature / top-k /
-        top-p distribution of the step's logits (GenerationOptions, sample_logits :391-418), with one uniform number per
-        token from a host generator seeded with `seed` (the generator stays on the host, as the reference's does).  The
-        prompt goes through prefill() in blocks (in the prompt's activation mode) on one GPU and on a column-cut sharded
-        decoder with an NCCL group, token by token otherwise; batched_prefill overrides the choice.
-        Raises when the context would overflow."""
-        torch = self.torch
-        if not prompt or len(prompt) + max_new > self.max_positions:
-            raise ValueError("prompt + max_new exceeds the configured positions")
-        self.reset()
-        self.sync_ranks()
-        out: list[int] = []
-        rng = np.random.default_rng(seed) if temperature > 0.0 else None
-        with torch.cuda.stream(self.stream):
-            self.feed_prompt(prompt, batched_prefill)
-            for n in range(max_new):
-                if rng is not None:               # the step left the greedy pick in self.token: draw instead
-                    self._sample(temperature, top_k, top_p, float(rng.random()))
-                tok = int(self.token.item())      # device -> host read of the step's result
-                out.append(tok)
-                if on_token:
-                    on_token(tok)
-                if n + 1 < max_new:
-                    self.host_token[0] = tok      # host -> device: the next step's input comes from the caller's side
-                    self.token.copy_(self.host_token, non_blocking=True)
-                    self.step(want_token=True)
-        self.be.dev_check(self.stream.cuda_stream)
-        return out
-
-    def last_logits(self) -> np.ndarray:
+    def _block_logits(self, rows: list[int]):
+        if self.world != 1:
+            raise ValueError("the sharded decoder keeps only its shard of the logits; use one GPU")
+        torch, st = self.torch, self.stream.cuda_stream
+        xn = self._prefill_buffers()["xn"][torch.tensor(rows, device=self.dev)]      # normalised with the output norm by the block's last step
+        out = torch.zeros((len(rows), self.cfg.vocab), dtype=torch.float32, device=self.dev)
+        for i in range(0, len(rows), 8):
+            n = min(8, len(rows) - i)
+            self.be.dev_gemv([self.h["output.weight"]], [out[i].data_ptr()], xn[i].data_ptr(), n, self.act_mode, st)
         self.stream.synchronize()
-        return self.logits.cpu().numpy()
+        return out
 
     def close(self) -> None:
         self.stream.synchronize()
