@@ -557,7 +557,7 @@ int zen_cuda_dev_window_attention_step(const zen_cuda_window_attention* a, const
 
 /* Mixers with a matrix state S [dim][vdim] per head, kept as [heads][vdim][pitch] fp32, pitch = dim rounded up to 32.
  *   delta rule   S <- g * S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  q, k, v pass a causal convolution of `taps` taps per
- *                channel and silu (ring [taps][2 kv_heads dim + heads vdim], slot = position mod taps), q and k become unit vectors
+ *                channel (conv [taps][channels]) and silu (ring [taps][2 kv_heads dim + heads vdim], slot = position mod taps), q and k become unit vectors
  *                (q also times dim^-1/2), beta = sigmoid, g = exp(-exp(a_log) softplus(a2 a1 + dt_bias)); output gate sigmoid(g2 g1).
  *   gated write  S <- f * S + (1 - f) v^T; o = S^T q; q = silu, f = lower + (1 - lower) sigmoid(. + f_bias).
  * norm [vdim]: weight of the output's RMS norm per head.  dim and vdim at most 256. */

@@ -25,7 +25,7 @@ struct LinearLayer {
     uint32_t taps;                 // delta rule: convolution taps
     uint32_t rank_a, rank_g;       // delta rule: ranks of the decay's and the output gate's projections
     uint32_t a2_ld, g2_ld;
-    const float* conv;             // [2 kv_heads dim + heads vdim][taps]: q, k, v channels
+    const float* conv;             // [taps][channels]: q, k, v channels
     const float* a_log;            // [heads]
     const float* dt_bias;          // [heads][dim]
     const __nv_bfloat16* a2;       // [heads dim][a2_ld]
@@ -43,18 +43,20 @@ __host__ __device__ inline uint32_t linear_channels(const LinearLayer& l) { retu
 // rows before the block come from the ring, tokens before the sequence's start are zeros.
 __device__ __forceinline__ float conv_silu(const LinearLayer& l, const float* __restrict__ x, uint32_t ld, int t, int pos, uint32_t c, uint32_t channels) {
     float y = 0.0f;
-    for (uint32_t j = 0; j < l.taps; ++j) {
-        const int back = static_cast<int>(l.taps - 1 - j), s = t - back, at = pos + s;
-        if (at < 0) continue;
-        const float v = s >= 0 ? __ldcg(x + static_cast<size_t>(s) * ld + c) : l.ring[static_cast<size_t>(static_cast<uint32_t>(at) % l.taps) * channels + c];
-        y = fmaf(l.conv[static_cast<size_t>(c) * l.taps + j], v, y);
+    const int taps = static_cast<int>(l.taps);
+#pragma unroll 4
+    for (int j = 0; j < taps; ++j) {
+        const int s = t - (taps - 1 - j), at = pos + s;
+        const float* src = s >= 0 ? x + static_cast<size_t>(s) * ld + c : l.ring + static_cast<size_t>(static_cast<uint32_t>(max(at, 0)) % l.taps) * channels + c;
+        const float v = at >= 0 ? __ldcg(src) : 0.0f;
+        y = fmaf(__ldg(l.conv + static_cast<size_t>(j) * channels + c), v, y);
     }
     return silu_f(y);
 }
 
 // ---- inputs of the scan for a block of tokens -------------------------------------------------------------------------
 
-// Delta rule.  proj [T][ld]: q | k | v | b columns; decay [T][heads dim] = W_a2 W_a1 h.  One CTA per token.
+// Delta rule.  proj [T][ld]: q | k | v | b columns; decay [T][heads dim] = W_a2 W_a1 h.  Grid: (tokens, CTAs that share a token).
 //   q, k [T][kv_heads][pitch] unit vectors (q also times dim^-1/2), g [T][heads][pitch], v [T][heads vdim], beta [T][heads].
 __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld,
                                                                 const float* __restrict__ decay, uint32_t decay_ld, const int* __restrict__ pos_ptr,
@@ -63,8 +65,9 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
     pdl_launch_dependents();
     pdl_wait();
     const int t = static_cast<int>(blockIdx.x), pos = *pos_ptr;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, channels = linear_channels(l), kd = l.kv_heads * l.dim;
-    for (uint32_t i = warp; i < 2 * l.kv_heads; i += 8) {          // a warp takes a q or k head
+    const uint32_t warp = blockIdx.y * 8 + (threadIdx.x >> 5), warps = gridDim.y * 8, lane = threadIdx.x & 31, channels = linear_channels(l), kd = l.kv_heads * l.dim;
+    const uint32_t first = blockIdx.y * 256 + threadIdx.x, step = gridDim.y * 256;
+    for (uint32_t i = warp; i < 2 * l.kv_heads; i += warps) {      // a warp takes a q or k head
         const bool is_q = i < l.kv_heads;
         const uint32_t head = is_q ? i : i - l.kv_heads, c0 = (is_q ? 0u : kd) + head * l.dim;
         float* dst = (is_q ? q : k) + (static_cast<size_t>(t) * l.kv_heads + head) * l.pitch;
@@ -81,13 +84,13 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
         for (int j = 0; j < 8; ++j)
             if (lane + 32 * j < l.pitch) dst[lane + 32 * j] = val[j] * inv;
     }
-    for (uint32_t i = threadIdx.x; i < l.heads * l.vdim; i += 256) v[static_cast<size_t>(t) * l.heads * l.vdim + i] = conv_silu(l, proj, ld, t, pos, 2 * kd + i, channels);
-    for (uint32_t i = threadIdx.x; i < l.heads; i += 256) beta[static_cast<size_t>(t) * l.heads + i] = logistic(proj[static_cast<size_t>(t) * ld + channels + i]);
-    for (uint32_t i = threadIdx.x; i < l.heads * l.pitch; i += 256) {
-        const uint32_t h = i / l.pitch, d = i % l.pitch;
-        float gate = 0.0f;
-        if (d < l.dim) gate = expf(-expf(l.a_log[h]) * softplus_f(decay[static_cast<size_t>(t) * decay_ld + h * l.dim + d] + l.dt_bias[h * l.dim + d]));
-        g[static_cast<size_t>(t) * l.heads * l.pitch + i] = gate;
+    for (uint32_t i = first; i < l.heads * l.vdim; i += step) v[static_cast<size_t>(t) * l.heads * l.vdim + i] = conv_silu(l, proj, ld, t, pos, 2 * kd + i, channels);
+    for (uint32_t i = first; i < l.heads; i += step) beta[static_cast<size_t>(t) * l.heads + i] = logistic(proj[static_cast<size_t>(t) * ld + channels + i]);
+    for (uint32_t h = warp; h < l.heads; h += warps) {             // a warp takes a head's decays
+        const float rate = -expf(l.a_log[h]);
+        const float* src = decay + static_cast<size_t>(t) * decay_ld + h * l.dim;
+        for (uint32_t d = lane; d < l.pitch; d += 32)
+            g[(static_cast<size_t>(t) * l.heads + h) * l.pitch + d] = d < l.dim ? expf(rate * softplus_f(src[d] + l.dt_bias[h * l.dim + d])) : 0.0f;
     }
 }
 
@@ -133,11 +136,11 @@ struct ScanParams {
     uint32_t tokens, heads, q_heads, vdim, v_ld;
 };
 
-constexpr int kScanThreads = 128, kScanColumns = 32, kScanTokens = 8;    // columns of S per CTA; tokens per staged block
+constexpr int kScanThreads = 128, kScanColumns = 32, kScanTokens = 8, kScanStages = 4;    // columns of S per CTA; tokens per staged block; blocks in flight
 template <int kQuads, bool kDelta>
 __host__ __device__ constexpr uint32_t scan_token_floats() { return (kDelta ? 3 : 2) * kQuads * 32 + kScanColumns + 4; }
 template <int kQuads, bool kDelta>
-__host__ __device__ constexpr uint32_t scan_smem_bytes() { return 2 * kScanTokens * scan_token_floats<kQuads, kDelta>() * 4; }
+__host__ __device__ constexpr uint32_t scan_smem_bytes() { return kScanStages * kScanTokens * scan_token_floats<kQuads, kDelta>() * 4; }
 
 __device__ __forceinline__ void cp_async_4(float* smem_dst, const float* gmem_src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst))), "l"(gmem_src) : "memory");
@@ -146,7 +149,10 @@ __device__ __forceinline__ void cp_async_4(float* smem_dst, const float* gmem_sr
 // A CTA takes 32 columns of one head's state (its value channels), a warp eight of them.  A column's rows are spread over eight
 // lanes, lane `part` holding the 16-byte words part, part + 8, ...; a lane holds two columns, so a word of q, k or g read from
 // shared memory serves both.  The state never leaves the registers between the block's first and last token; arithmetic is packed
-// fp32 pairs.  kQuads = pitch / 32.  Grid: (ceil(vdim / 32), heads).
+// fp32 pairs.  Tokens go in groups of eight: only the delta rule's own sum is reduced token by token (it is what the next token
+// waits for); the read-outs of a group stay as partial sums and are reduced together, after which lane `part` holds token `part`'s.
+// A group's missing tokens at the end of the block are staged as g = 1 and zeros: they leave the state as it is.
+// kQuads = pitch / 32.  Grid: (ceil(vdim / 32), heads).
 template <int kQuads, bool kDelta>
 __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_constant__ ScanParams p) {
     constexpr uint32_t kPitch = kQuads * 32, kToken = scan_token_floats<kQuads, kDelta>();
@@ -158,6 +164,37 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_c
     const uint32_t local = warp * 8 + (lane >> 3) * 2, c0 = col_base + local;      // this lane's columns: c0, c0 + 1
     const bool on0 = c0 < p.vdim, on1 = c0 + 1 < p.vdim;
     pdl_wait();
+    auto stage = [&](uint32_t t0, uint32_t buf) {
+        float* dst = scan_smem + buf * kScanTokens * kToken;
+        constexpr uint32_t kWords = kPitch / 4, kRows = kDelta ? 3 : 2;
+#pragma unroll 4
+        for (uint32_t i = threadIdx.x; i < kScanTokens * kRows * kWords; i += kScanThreads) {
+            const uint32_t t = i / (kRows * kWords), rest = i % (kRows * kWords), row = rest / kWords, word = rest % kWords;
+            float* d = dst + t * kToken + row * kPitch + word * 4;
+            if (t0 + t < p.tokens) {
+                const float* src = row == 0 ? p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch
+                                            : (row == 1 ? p.q : p.k) + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch;
+                cp_async_16(d, src + word * 4, 16);
+            } else {
+                const float fill = row == 0 ? 1.0f : 0.0f;
+                *reinterpret_cast<float4*>(d) = make_float4(fill, fill, fill, fill);
+            }
+        }
+#pragma unroll
+        for (uint32_t i = threadIdx.x; i < kScanTokens * kScanColumns; i += kScanThreads) {
+            const uint32_t t = i / kScanColumns, c = i % kScanColumns;
+            float* d = dst + t * kToken + kV + c;
+            if (col_base + c < p.vdim && t0 + t < p.tokens) cp_async_4(d, p.v + static_cast<size_t>(t0 + t) * p.v_ld + h * p.vdim + col_base + c); else *d = 0.0f;
+        }
+        if (kDelta && threadIdx.x < kScanTokens) {
+            float* d = dst + threadIdx.x * kToken + kB;
+            if (t0 + threadIdx.x < p.tokens) cp_async_4(d, p.beta + static_cast<size_t>(t0 + threadIdx.x) * p.heads + h); else *d = 0.0f;
+        }
+    };
+    for (uint32_t i = 0; i < kScanStages - 1; ++i) {
+        if (i * kScanTokens < p.tokens) stage(i * kScanTokens, i);
+        cp_async_commit();
+    }
     uint64_t s[2][kQuads][2];
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
@@ -169,36 +206,18 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_c
             s[c][i][1] = pf_pack(w.z, w.w);
         }
     }
-    auto stage = [&](uint32_t t0, uint32_t buf) {
-        float* dst = scan_smem + buf * kScanTokens * kToken;
-        const uint32_t n = min(static_cast<uint32_t>(kScanTokens), p.tokens - t0);
-        constexpr uint32_t kWords = kPitch / 4, kRows = kDelta ? 3 : 2;
-        for (uint32_t i = threadIdx.x; i < n * kRows * kWords; i += kScanThreads) {
-            const uint32_t t = i / (kRows * kWords), rest = i % (kRows * kWords), row = rest / kWords, word = rest % kWords;
-            const float* src = row == 0 ? p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch
-                                        : (row == 1 ? p.q : p.k) + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch;
-            cp_async_16(dst + t * kToken + row * kPitch + word * 4, src + word * 4, 16);
-        }
-        for (uint32_t i = threadIdx.x; i < n * kScanColumns; i += kScanThreads) {
-            const uint32_t t = i / kScanColumns, c = i % kScanColumns;
-            float* d = dst + t * kToken + kV + c;
-            if (col_base + c < p.vdim) cp_async_4(d, p.v + static_cast<size_t>(t0 + t) * p.v_ld + h * p.vdim + col_base + c); else *d = 0.0f;
-        }
-        if (kDelta && threadIdx.x < n) cp_async_4(dst + threadIdx.x * kToken + kB, p.beta + static_cast<size_t>(t0 + threadIdx.x) * p.heads + h);
-        cp_async_commit();
-    };
     const uint64_t zero2 = pf_pack(0.0f, 0.0f);
-    stage(0, 0);
-    uint32_t buf = 0;
-    for (uint32_t t0 = 0; t0 < p.tokens; t0 += kScanTokens, buf ^= 1u) {
-        const bool more = t0 + kScanTokens < p.tokens;
-        if (more) stage(t0 + kScanTokens, buf ^ 1u);
-        if (more) cp_async_wait<1>(); else cp_async_wait<0>();
-        __syncthreads();
-        const uint32_t n = min(static_cast<uint32_t>(kScanTokens), p.tokens - t0);
-        const float* tok = scan_smem + buf * kScanTokens * kToken;
-#pragma unroll 2
-        for (uint32_t t = 0; t < n; ++t, tok += kToken) {
+    uint32_t group = 0;
+    for (uint32_t t0 = 0; t0 < p.tokens; t0 += kScanTokens, ++group) {
+        cp_async_wait<kScanStages - 2>();           // this group's copies have landed (this thread's; the barrier covers the others')
+        __syncthreads();                            // ... and everybody is done with the buffer filled next
+        const uint32_t ahead = t0 + (kScanStages - 1) * kScanTokens;
+        if (ahead < p.tokens) stage(ahead, (group + kScanStages - 1) % kScanStages);
+        cp_async_commit();
+        const float* tok = scan_smem + (group % kScanStages) * kScanTokens * kToken;
+        float out[2][kScanTokens];
+#pragma unroll
+        for (int t = 0; t < kScanTokens; ++t, tok += kToken) {
             uint64_t g[kQuads][2], q[kQuads][2], k[kQuads][2];
 #pragma unroll
             for (int i = 0; i < kQuads; ++i) {
@@ -240,7 +259,6 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_c
                 u[0] = beta * (u[0] - dot[0]);
                 u[1] = beta * (u[1] - dot[1]);
             }
-            float out[2];
 #pragma unroll
             for (int c = 0; c < 2; ++c) {
                 const uint64_t uu = pf_pack(u[c], u[c]);
@@ -260,16 +278,21 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_c
                 float a, b, e, f;
                 pf_unpack(d0, a, b);
                 pf_unpack(d1, e, f);
-                out[c] = (a + b) + (e + f);
+                out[c][t] = (a + b) + (e + f);
             }
-            // the two columns' sums over eight lanes: odd lanes end with column c0 + 1, even lanes with c0
-            const bool odd = part & 1;
-            float o = (odd ? out[1] : out[0]) + __shfl_xor_sync(0xffffffffu, odd ? out[0] : out[1], 1);
-            o += __shfl_xor_sync(0xffffffffu, o, 2);
-            o += __shfl_xor_sync(0xffffffffu, o, 4);
-            if (part < 2 && (part ? on1 : on0)) p.out[(static_cast<size_t>(t0 + t) * p.heads + h) * p.vdim + c0 + part] = o;
         }
-        __syncthreads();
+        // eight partial read-outs per column over eight lanes: each exchange halves the tokens a lane carries
+        const bool b2 = part & 4, b1 = part & 2, b0 = part & 1;
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+            float r4[4], r2[2];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) r4[i] = (b2 ? out[c][i + 4] : out[c][i]) + __shfl_xor_sync(0xffffffffu, b2 ? out[c][i] : out[c][i + 4], 4);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) r2[i] = (b1 ? r4[i + 2] : r4[i]) + __shfl_xor_sync(0xffffffffu, b1 ? r4[i] : r4[i + 2], 2);
+            const float o = (b0 ? r2[1] : r2[0]) + __shfl_xor_sync(0xffffffffu, b0 ? r2[0] : r2[1], 1);
+            if ((c ? on1 : on0) && t0 + part < p.tokens) p.out[(static_cast<size_t>(t0 + part) * p.heads + h) * p.vdim + c0 + c] = o;
+        }
     }
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
@@ -298,6 +321,29 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_c
     __shared__ float v[256], o[256], gate[256];
     const uint32_t h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7, quads = l.pitch / 32;
     pdl_launch_dependents();
+    // rows of the rank projections, eight lanes to a row (decays first, then the gate): weights, so their first kAhead words per
+    // lane are fetched while the previous launch is still running
+    constexpr uint32_t kAhead = 8;
+    uint4 ahead[kAhead];
+    const uint32_t words = kDelta ? (max(l.a2_ld, l.g2_ld) + 63) / 64 : 0;      // 16-byte words per lane and row
+    auto rank_row = [&](uint32_t r, uint32_t& ld) -> const __nv_bfloat16* {     // null: padding
+        const bool is_g = r >= l.pitch;
+        const uint32_t d = is_g ? r - l.pitch : r;
+        ld = is_g ? l.g2_ld : l.a2_ld;
+        if (d >= (is_g ? l.vdim : l.dim)) return nullptr;
+        return is_g ? l.g2 + static_cast<size_t>(h * l.vdim + d) * ld : l.a2 + static_cast<size_t>(h * l.dim + d) * ld;
+    };
+    if (kDelta) {
+        uint32_t r = warp * 4 + (lane >> 3), word = 0;
+#pragma unroll
+        for (uint32_t i = 0; i < kAhead; ++i) {
+            uint32_t ld;
+            const __nv_bfloat16* w = rank_row(r, ld);
+            const uint32_t c = (word * 8 + part) * 8;
+            ahead[i] = w && c < ld ? __ldg(reinterpret_cast<const uint4*>(w + c)) : make_uint4(0, 0, 0, 0);
+            if (++word == words) { word = 0; r += kWarps * 4; }
+        }
+    }
     pdl_wait();
     // the first columns' state words are on their way while the token's vectors are formed
     float* const state = l.state + static_cast<size_t>(h) * l.vdim * l.pitch + part * 4;
@@ -326,30 +372,38 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_c
             }
             (is_v ? v : is_k ? k : q)[d] = y;
         }
-        // decays and output gate: rows of the rank projections, eight lanes to a row
+        // decays and output gate
         const float a_scale = -expf(l.a_log[h]);
-        for (uint32_t r0 = warp * 4; r0 < l.pitch + l.vdim; r0 += kWarps * 4) {
-            const uint32_t r = r0 + (lane >> 3);
-            const bool is_g = r >= l.pitch;                        // a row of the gate
-            const uint32_t d = is_g ? r - l.pitch : r, ld = is_g ? l.g2_ld : l.a2_ld, rank = is_g ? l.rank_g : l.rank_a;
-            const bool live = is_g ? d < l.vdim : d < l.dim;
-            const __nv_bfloat16* w = is_g ? l.g2 + static_cast<size_t>(h * l.vdim + d) * ld : l.a2 + static_cast<size_t>(h * l.dim + d) * ld;
+        uint32_t r = warp * 4 + (lane >> 3), word = 0;
+        float acc = 0.0f;
+        auto take = [&](const uint4& w) {
+            const bool is_g = r >= l.pitch;
             const float* low = is_g ? low_g : low_a;
-            float acc = 0.0f;
-            if (live)
-                for (uint32_t c = part * 8; c < ld; c += 64) {
-                    const uint4 ww = __ldg(reinterpret_cast<const uint4*>(w + c));
-                    float x[8];
+            const uint32_t c = (word * 8 + part) * 8, rank = is_g ? l.rank_g : l.rank_a;
+            float x[8];
 #pragma unroll
-                    for (int j = 0; j < 8; ++j) x[j] = c + j < rank ? __ldcg(low + c + j) : 0.0f;
-                    dense_fma8(ww, x, acc);
-                }
+            for (int j = 0; j < 8; ++j) x[j] = c + j < rank ? __ldcg(low + c + j) : 0.0f;
+            dense_fma8(w, x, acc);
+            if (++word < words) return;
 #pragma unroll
             for (int s = 1; s < 8; s <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, s);
-            if (part == 0) {
-                if (is_g) { if (live) gate[d] = logistic(acc); }
-                else g[d] = live ? expf(a_scale * softplus_f(acc + l.dt_bias[h * l.dim + d])) : 0.0f;
+            if (part == 0 && r < l.pitch + l.vdim) {
+                if (is_g) gate[r - l.pitch] = logistic(acc);
+                else g[r] = r < l.dim ? expf(a_scale * softplus_f(acc + l.dt_bias[h * l.dim + r])) : 0.0f;
             }
+            acc = 0.0f;
+            word = 0;
+            r += kWarps * 4;
+        };
+        // r - lane / 8 and word are the same in all lanes of a warp, so the loops below do not diverge around the shuffles
+#pragma unroll
+        for (uint32_t i = 0; i < kAhead; ++i)
+            if (r - (lane >> 3) < l.pitch + l.vdim) take(ahead[i]);
+        while (r - (lane >> 3) < l.pitch + l.vdim) {
+            uint32_t ld;
+            const __nv_bfloat16* w = rank_row(r, ld);
+            const uint32_t c = (word * 8 + part) * 8;
+            take(w && c < ld ? __ldg(reinterpret_cast<const uint4*>(w + c)) : make_uint4(0, 0, 0, 0));
         }
         __syncthreads();
         if (warp < 2) {                                            // unit norms: warp 0 takes q, warp 1 k

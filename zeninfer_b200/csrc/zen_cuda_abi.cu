@@ -639,6 +639,7 @@ bool enqueue_gemv(State& s, const zen_cuda_weights* const* w, float* const* d_y,
             return set_error(s, "gemv gather: a chained input needs one token and columns == world x slot_floats");
         p.gather = *gather;
     }
+    if (w[0]->format == ZEN_CUDA_BF16) return set_error(s, "gemv: a bfloat16 matrix goes through zen_cuda_dev_dense_gemv");
     if (w[0]->format != ZEN_CUDA_Q8_0) {
         if (act_mode != ZEN_CUDA_ACT_FP32) return set_error(s, "gemv: Q4_0, Q6_K, Q4_K and Q5_K take fp32-equivalent activations only");
         if (d_gate || d_norm_weight || accumulate || swiglu_pair) return set_error(s, "gemv: fused inputs, outputs and accumulation are Q8_0 paths");

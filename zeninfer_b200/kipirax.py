@@ -211,7 +211,7 @@ class KipiraxDecoder(Decoder):
                 L.update(proj=matrix(*[(f"{p}mix.{n}", r) for n, r in rows]), o=[matrix((p + "mix.o", W), columns=m.heads * m.vdim)],
                          a2=matrix((p + "mix.a2", m.heads * m.dim), columns=rank_a), g2=matrix((p + "mix.g2", m.heads * m.vdim), columns=rank_g),
                          rank_a=rank_a, rank_g=rank_g)
-                conv = self.torch.cat([vector(f"{p}mix.{n}.conv", (r, m.conv)) for n, r in rows[:3]])
+                conv = self.torch.cat([vector(f"{p}mix.{n}.conv", (r, m.conv)) for n, r in rows[:3]]).t().contiguous()      # [taps][channels]
                 keep = dict(conv=conv, a_log=vector(p + "mix.A_log", (m.heads,)), dt_bias=vector(p + "mix.dt_bias", (m.heads * m.dim,)),
                             norm=vector(p + "mix.norm", (m.vdim,)), ring=add(p + "ring", (m.conv, m.channels)),
                             state=add(p + "state", (m.heads, m.vdim, round_up(m.dim, 32)), start_zero=True))
@@ -422,34 +422,32 @@ class KipiraxDecoder(Decoder):
         self.handles.clear()
 
 
+def random_tensor(name: str, shape: tuple[int, ...], rng: np.random.Generator) -> np.ndarray:
+    """One tensor of a made-up model, fp32: matrices N(0, 1 / columns), norm weights near one, decays, bounds and shifts in their
+    usual ranges."""
+    z = rng.standard_normal(shape, dtype=np.float32)
+    kind = name.split(".", 1)[-1]
+    if name in ("embed", "pos"):
+        w = z * 0.5
+    elif kind == "shift":
+        w = 1.0 / (1.0 + np.exp(-z))
+    elif kind.endswith("lower"):
+        w = 0.9 / (1.0 + np.exp(-z))
+    elif kind.endswith("A_log"):
+        w = np.log(1.0 + 3.0 * rng.random(shape, dtype=np.float32))
+    elif kind.endswith("dt_bias"):
+        w = z - 3.0
+    elif len(shape) == 2:
+        w = z * shape[1] ** -0.5
+    else:
+        w = z if kind.endswith("f.b") else 1.0 + 0.1 * z
+    return w.astype(np.float32)
+
+
 def random_tensors(cfg: KipiraxConfig, rank_a: int, rank_g: int, seed: int) -> dict[str, np.ndarray]:
-    """A made-up model as bfloat16 bit patterns: matrices N(0, 1 / columns), norm weights near one, decays, bounds and shifts in
-    their usual ranges."""
+    """A made-up model as bfloat16 bit patterns."""
     rng = np.random.default_rng(seed)
-    out = {}
-    for name, shape in tensor_plan(cfg, rank_a, rank_g):
-        z = rng.standard_normal(shape, dtype=np.float32)
-        kind = name.split(".", 1)[-1]
-        if name in ("embed", "pos"):
-            w = z * np.float32(0.5)
-        elif kind == "shift":
-            w = 1.0 / (1.0 + np.exp(-z))
-        elif kind.endswith("lower"):
-            w = 0.9 / (1.0 + np.exp(-z))
-        elif kind.endswith("A_log"):
-            w = np.log(1.0 + 3.0 * rng.random(shape, dtype=np.float32))
-        elif kind.endswith("dt_bias"):
-            w = z - 3.0
-        elif kind.endswith(".conv"):
-            w = z * np.float32(shape[1] ** -0.5)
-        elif len(shape) == 1 and not kind.endswith("f.b"):
-            w = 1.0 + np.float32(0.1) * z
-        elif len(shape) == 1:
-            w = z
-        else:
-            w = z * np.float32(shape[1] ** -0.5)
-        out[name] = blocks.to_bf16(w.astype(np.float32))
-    return out
+    return {name: blocks.to_bf16(random_tensor(name, shape, rng)) for name, shape in tensor_plan(cfg, rank_a, rank_g)}
 
 
-__all__ = ["KipiraxConfig", "KipiraxDecoder", "random_tensors", "tensor_plan"]
+__all__ = ["KipiraxConfig", "KipiraxDecoder", "random_tensor", "random_tensors", "tensor_plan"]
