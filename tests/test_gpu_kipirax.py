@@ -321,7 +321,8 @@ def run_linear(be, kind, m, case, cuts):
 
 
 @pytest.mark.parametrize("m", [dict(heads=4, kv_heads=2, dim=20, vdim=28, conv=3, rank_a=10, rank_g=7), dict(heads=3, kv_heads=1, dim=64, vdim=33, conv=1, rank_a=8, rank_g=70),
-                               dict(heads=2, kv_heads=2, dim=130, vdim=65, conv=6, rank_a=140, rank_g=3), dict(heads=1, kv_heads=1, dim=256, vdim=256, conv=4, rank_a=16, rank_g=300)])
+                               dict(heads=2, kv_heads=2, dim=130, vdim=65, conv=6, rank_a=140, rank_g=3), dict(heads=1, kv_heads=1, dim=256, vdim=256, conv=4, rank_a=16, rank_g=300), dict(heads=2, kv_heads=1, dim=18, vdim=40, conv=11, rank_a=5, rank_g=9),
+                               dict(heads=2, kv_heads=2, dim=32, vdim=32, conv=8, rank_a=64, rank_g=64)])
 @pytest.mark.parametrize("cuts", CUTS)
 def test_delta_rule(be, m, cuts):
     case = linear_case(be, "delta", m["dim"], **m)

@@ -2,10 +2,8 @@
 //
 //   * one CTA per SM owns a contiguous slice of the launch's rows (over all its tensors); its sixteen warps split K in units of
 //     256 columns (and, where K has fewer units than warps, the row groups too), eight rows per step: a lane holds 16 bytes of
-//     each of eight rows and eight values of x, so a step keeps eight 16-byte loads per lane in flight and the next step's
-//     loads are issued before this step's arithmetic;
-//   * weights are constants: the first step's loads go out before the previous grid has finished (griddepcontrol), and the rest
-//     of the slice is pulled into L2;
+//     each of eight rows and eight values of x, and two steps' loads (sixteen 16-byte words per lane) are in flight;
+//   * weights are constants: the first two steps' loads go out before the previous grid has finished (griddepcontrol);
 //   * the prologue can finish the sublayer before it (row_ops.cuh: grouped norm, residual add, token shift or output norm), so
 //     a decode step needs no launches for them: every CTA forms the input vector itself, CTA 0 stores the residual stream;
 //   * the epilogue applies the product's activation (squared ReLU, or the logits' soft cap) in fp32.
@@ -87,10 +85,23 @@ __global__ void __launch_bounds__(kDenseThreads, 1) gemv_bf16_kernel(const __gri
         for (int i = 0; i < kDenseRows; ++i)
             v[i] = (w.r + i < w.r_end && col < t.ld) ? __ldg(reinterpret_cast<const uint4*>(base + static_cast<size_t>(i) * t.ld)) : make_uint4(0, 0, 0, 0);
     };
-    Walk cur{0, 0, 0, 0};
-    enter(cur);
-    uint4 next_w[kDenseRows];
-    if (cur.ti < p.tasks) load(cur, next_w);
+    auto advance = [&](Walk& w) {    // to the step after w
+        const bool row_done = w.u + p.k_split >= dense_units(p.task[w.ti].ld);
+        w.u += p.k_split;
+        if (row_done) {
+            w.u = part;
+            w.r += teams * kDenseRows;
+            if (w.r >= w.r_end) { ++w.ti; enter(w); }
+        }
+    };
+    // two steps' weights are in flight at any time: while one buffer is used up, the other's loads are on their way
+    uint4 buf0[kDenseRows], buf1[kDenseRows];
+    Walk w0{0, 0, 0, 0}, w1;
+    enter(w0);
+    if (w0.ti < p.tasks) load(w0, buf0);
+    w1 = w0;
+    if (w1.ti < p.tasks) advance(w1);
+    if (w1.ti < p.tasks) load(w1, buf1);
 
     // the input vectors in shared memory, each padded with zeros to whole units; then per-row partial sums of the slice
     float* xs = dense_smem;
@@ -122,55 +133,51 @@ __global__ void __launch_bounds__(kDenseThreads, 1) gemv_bf16_kernel(const __gri
     float acc[kDenseRows];
 #pragma unroll
     for (int i = 0; i < kDenseRows; ++i) acc[i] = 0.0f;
-    uint32_t x_base = 0, x_task = 0;                              // where the current task's input starts in xs
-    while (cur.ti < p.tasks) {
-        uint4 w[kDenseRows];
-#pragma unroll
-        for (int i = 0; i < kDenseRows; ++i) w[i] = next_w[i];
-        Walk nxt = cur;
-        const DenseTask& t = p.task[cur.ti];
-        const uint32_t units = dense_units(t.ld);
-        nxt.u += p.k_split;
-        const bool row_done = nxt.u >= units;
-        if (row_done) {
-            nxt.u = part;
-            nxt.r += teams * kDenseRows;
-            if (nxt.r >= nxt.r_end) { ++nxt.ti; enter(nxt); }
-        }
-        if (nxt.ti < p.tasks) load(nxt, next_w);
-        for (; x_task < cur.ti; ++x_task) x_base += dense_units(p.task[x_task].ld) * kDenseUnit;
-        const float4* xv = reinterpret_cast<const float4*>(xs + (p.has_prologue ? 0u : x_base) + cur.u * kDenseUnit + lane * 8);
+    auto consume = [&](const Walk& at, const uint4 (&w)[kDenseRows]) {
+        const DenseTask& t = p.task[at.ti];
+        uint32_t x_base = 0;                                      // where the task's input starts in xs
+        for (uint32_t i = 0; i < at.ti; ++i) x_base += dense_units(p.task[i].ld) * kDenseUnit;
+        const float4* xv = reinterpret_cast<const float4*>(xs + x_base + at.u * kDenseUnit + lane * 8);
         const float4 x0 = xv[0], x1 = xv[1];
         const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
         for (int i = 0; i < kDenseRows; ++i) dense_fma8(w[i], x, acc[i]);
-        if (row_done) {
-            // eight sums over 32 lanes; at each of the first three exchanges a lane keeps half of the rows it carries
+        if (at.u + p.k_split < dense_units(t.ld)) return;
+        // the row group is done: eight sums over 32 lanes; at each of the first three exchanges a lane keeps half of the rows it carries
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const bool hi = lane & 16;
-                const float keep = hi ? acc[i + 4] : acc[i], give = hi ? acc[i] : acc[i + 4];
-                acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, 16);
-            }
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const bool hi = lane & 8;
-                const float keep = hi ? acc[i + 2] : acc[i], give = hi ? acc[i] : acc[i + 2];
-                acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, 8);
-            }
-            {
-                const bool hi = lane & 4;
-                const float keep = hi ? acc[1] : acc[0], give = hi ? acc[0] : acc[1];
-                acc[0] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
-            }
-            acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 2);
-            acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
-            const uint32_t mine = ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);
-            if ((lane & 3) == 0 && cur.r + mine < cur.r_end) sums[static_cast<size_t>(t.first_row + cur.r + mine - slice0) * p.k_split + part] = acc[0];
-#pragma unroll
-            for (int i = 0; i < kDenseRows; ++i) acc[i] = 0.0f;
+        for (int i = 0; i < 4; ++i) {
+            const bool hi = lane & 16;
+            const float keep = hi ? acc[i + 4] : acc[i], give = hi ? acc[i] : acc[i + 4];
+            acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, 16);
         }
-        cur = nxt;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const bool hi = lane & 8;
+            const float keep = hi ? acc[i + 2] : acc[i], give = hi ? acc[i] : acc[i + 2];
+            acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, 8);
+        }
+        {
+            const bool hi = lane & 4;
+            const float keep = hi ? acc[1] : acc[0], give = hi ? acc[0] : acc[1];
+            acc[0] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+        }
+        acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 2);
+        acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
+        const uint32_t mine = ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);
+        if ((lane & 3) == 0 && at.r + mine < at.r_end) sums[static_cast<size_t>(t.first_row + at.r + mine - slice0) * p.k_split + part] = acc[0];
+#pragma unroll
+        for (int i = 0; i < kDenseRows; ++i) acc[i] = 0.0f;
+    };
+    while (w0.ti < p.tasks) {
+        consume(w0, buf0);
+        w0 = w1;
+        if (w0.ti < p.tasks) advance(w0);
+        if (w0.ti < p.tasks) load(w0, buf0);
+        if (w1.ti >= p.tasks) break;
+        consume(w1, buf1);
+        w1 = w0;
+        if (w1.ti < p.tasks) advance(w1);
+        if (w1.ti < p.tasks) load(w1, buf1);
     }
     __syncthreads();
     for (uint32_t i = threadIdx.x; i < slice1 - slice0; i += kDenseThreads) {

@@ -56,41 +56,98 @@ __device__ __forceinline__ float conv_silu(const LinearLayer& l, const float* __
 
 // ---- inputs of the scan for a block of tokens -------------------------------------------------------------------------
 
-// Delta rule.  proj [T][ld]: q | k | v | b columns; decay [T][heads dim] = W_a2 W_a1 h.  Grid: (tokens, CTAs that share a token).
+constexpr int kStrip = 8;          // tokens a warp takes at a time: a channel's inputs stay in registers while the taps slide over them
+constexpr int kMaxSlidingTaps = 8; // more taps than this are read again for every token
+
+// y[i] = silu(convolution) of channel c at tokens t0 .. t0 + n - 1 (n <= kStrip; the rest is not used).
+__device__ __forceinline__ void conv_silu_strip(const LinearLayer& l, const float* __restrict__ x, uint32_t ld, int t0, int n, int pos, uint32_t c,
+                                                uint32_t channels, float (&y)[kStrip]) {
+    const int taps = static_cast<int>(l.taps);
+    if (taps > kMaxSlidingTaps) {
+#pragma unroll
+        for (int i = 0; i < kStrip; ++i)
+            if (i < n) y[i] = conv_silu(l, x, ld, t0 + i, pos, c, channels);
+        return;
+    }
+    float w[kMaxSlidingTaps], in[kMaxSlidingTaps - 1 + kStrip];       // w right-aligned: w[7] is the current token's; in[7 + i]: token t0 + i
+#pragma unroll
+    for (int j = 0; j < kMaxSlidingTaps; ++j) {
+        const int tap = j - (kMaxSlidingTaps - taps);
+        w[j] = tap >= 0 ? __ldg(l.conv + static_cast<size_t>(tap) * channels + c) : 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < kMaxSlidingTaps - 1 + kStrip; ++i) {
+        const int s = t0 + i - (kMaxSlidingTaps - 1), at = pos + s;   // block row, position
+        in[i] = 0.0f;
+        if (at >= 0 && s >= t0 - (taps - 1) && s < t0 + n)
+            in[i] = s >= 0 ? __ldcg(x + static_cast<size_t>(s) * ld + c) : l.ring[static_cast<size_t>(static_cast<uint32_t>(at) % l.taps) * channels + c];
+    }
+#pragma unroll
+    for (int i = 0; i < kStrip; ++i) {
+        float sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < kMaxSlidingTaps; ++j) sum = fmaf(w[j], in[i + j], sum);
+        y[i] = silu_f(sum);
+    }
+}
+
+// Delta rule.  proj [T][ld]: q | k | v | b columns; decay [T][heads dim] = W_a2 W_a1 h.
 //   q, k [T][kv_heads][pitch] unit vectors (q also times dim^-1/2), g [T][heads][pitch], v [T][heads vdim], beta [T][heads].
-__global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld,
+// A warp takes (strip of tokens, item): a q or k head, 32 value channels, or a head's decays.  Grid: (strips, CTAs that share one).
+__global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld, uint32_t tokens,
                                                                 const float* __restrict__ decay, uint32_t decay_ld, const int* __restrict__ pos_ptr,
                                                                 float* __restrict__ q, float* __restrict__ k, float* __restrict__ g, float* __restrict__ v,
                                                                 float* __restrict__ beta) {
     pdl_launch_dependents();
     pdl_wait();
-    const int t = static_cast<int>(blockIdx.x), pos = *pos_ptr;
-    const uint32_t warp = blockIdx.y * 8 + (threadIdx.x >> 5), warps = gridDim.y * 8, lane = threadIdx.x & 31, channels = linear_channels(l), kd = l.kv_heads * l.dim;
-    const uint32_t first = blockIdx.y * 256 + threadIdx.x, step = gridDim.y * 256;
-    for (uint32_t i = warp; i < 2 * l.kv_heads; i += warps) {      // a warp takes a q or k head
-        const bool is_q = i < l.kv_heads;
-        const uint32_t head = is_q ? i : i - l.kv_heads, c0 = (is_q ? 0u : kd) + head * l.dim;
-        float* dst = (is_q ? q : k) + (static_cast<size_t>(t) * l.kv_heads + head) * l.pitch;
-        float val[8], ss = 0.0f;                                   // pitch <= 256
+    const int t0 = static_cast<int>(blockIdx.x) * kStrip, n = min(kStrip, static_cast<int>(tokens) - t0), pos = *pos_ptr;
+    const uint32_t lane = threadIdx.x & 31, channels = linear_channels(l), kd = l.kv_heads * l.dim, nv = l.heads * l.vdim;
+    const uint32_t qk_items = 2 * l.kv_heads, v_items = (nv + 31) / 32, items = qk_items + v_items + l.heads;
+    for (uint32_t item = blockIdx.y * 8 + (threadIdx.x >> 5); item < items; item += gridDim.y * 8) {
+        float y[kStrip];
+        if (item < qk_items) {
+            const bool is_q = item < l.kv_heads;
+            const uint32_t head = is_q ? item : item - l.kv_heads, c0 = (is_q ? 0u : kd) + head * l.dim;
+            float* dst = (is_q ? q : k) + (static_cast<size_t>(t0) * l.kv_heads + head) * l.pitch;
+            const float scale = is_q ? 1.0f / sqrtf(static_cast<float>(l.dim)) : 1.0f;
+            float ss[kStrip];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const uint32_t d = lane + 32 * j;
-            val[j] = d < l.dim ? conv_silu(l, proj, ld, t, pos, c0 + d, channels) : 0.0f;
-            ss += val[j] * val[j];
+            for (int i = 0; i < kStrip; ++i) ss[i] = 0.0f;
+            for (uint32_t d = lane; d < l.pitch; d += 32) {            // unscaled first: a lane reads back only what it wrote
+#pragma unroll
+                for (int i = 0; i < kStrip; ++i) y[i] = 0.0f;
+                if (d < l.dim) conv_silu_strip(l, proj, ld, t0, n, pos, c0 + d, channels, y);
+#pragma unroll
+                for (int i = 0; i < kStrip; ++i)
+                    if (i < n) { ss[i] += y[i] * y[i]; dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] = y[i]; }
+            }
+#pragma unroll
+            for (int i = 0; i < kStrip; ++i) ss[i] = scale / sqrtf(warp_sum(ss[i]) + kUnitEps);
+            for (uint32_t d = lane; d < l.pitch; d += 32) {
+#pragma unroll
+                for (int i = 0; i < kStrip; ++i)
+                    if (i < n) dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] *= ss[i];
+            }
+        } else if (item < qk_items + v_items) {
+            const uint32_t c = (item - qk_items) * 32 + lane;
+            if (c >= nv) continue;
+            conv_silu_strip(l, proj, ld, t0, n, pos, 2 * kd + c, channels, y);
+#pragma unroll
+            for (int i = 0; i < kStrip; ++i)
+                if (i < n) v[static_cast<size_t>(t0 + i) * nv + c] = y[i];
+        } else {
+            const uint32_t h = item - qk_items - v_items;
+            const float rate = -expf(l.a_log[h]);
+            for (uint32_t d = lane; d < l.pitch; d += 32) {
+                const float bias = d < l.dim ? l.dt_bias[h * l.dim + d] : 0.0f;
+#pragma unroll
+                for (int i = 0; i < kStrip; ++i)
+                    if (i < n)
+                        g[(static_cast<size_t>(t0 + i) * l.heads + h) * l.pitch + d] =
+                            d < l.dim ? expf(rate * softplus_f(__ldcg(decay + static_cast<size_t>(t0 + i) * decay_ld + h * l.dim + d) + bias)) : 0.0f;
+            }
+            if (static_cast<int>(lane) < n) beta[static_cast<size_t>(t0 + lane) * l.heads + h] = logistic(__ldcg(proj + static_cast<size_t>(t0 + lane) * ld + channels + h));
         }
-        float inv = 1.0f / sqrtf(warp_sum(ss) + kUnitEps);
-        if (is_q) inv *= 1.0f / sqrtf(static_cast<float>(l.dim));
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
-            if (lane + 32 * j < l.pitch) dst[lane + 32 * j] = val[j] * inv;
-    }
-    for (uint32_t i = first; i < l.heads * l.vdim; i += step) v[static_cast<size_t>(t) * l.heads * l.vdim + i] = conv_silu(l, proj, ld, t, pos, 2 * kd + i, channels);
-    for (uint32_t i = first; i < l.heads; i += step) beta[static_cast<size_t>(t) * l.heads + i] = logistic(proj[static_cast<size_t>(t) * ld + channels + i]);
-    for (uint32_t h = warp; h < l.heads; h += warps) {             // a warp takes a head's decays
-        const float rate = -expf(l.a_log[h]);
-        const float* src = decay + static_cast<size_t>(t) * decay_ld + h * l.dim;
-        for (uint32_t d = lane; d < l.pitch; d += 32)
-            g[(static_cast<size_t>(t) * l.heads + h) * l.pitch + d] = d < l.dim ? expf(rate * softplus_f(src[d] + l.dt_bias[h * l.dim + d])) : 0.0f;
     }
 }
 

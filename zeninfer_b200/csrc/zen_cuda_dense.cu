@@ -281,7 +281,9 @@ int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* 
     ZC_ENTER(stream, linear_ok(l, 1) && d_proj && d_decay && decay_ld >= size_t(l->heads) * l->dim && tokens && tokens <= 0x7fffffffu && d_pos && d_q && d_k && d_g && d_v &&
                          d_beta, "delta_inputs_rows");
     const zk::LinearLayer d = device_form(*l, 1);
-    const cudaError_t r = launch(e, zk::delta_inputs_rows_kernel, dim3(u32(tokens), std::max(1u, std::min(8u, l->heads / 4))), dim3(256), 0, d, d_proj, u32(ld), d_decay, u32(decay_ld), d_pos, d_q, d_k, d_g, d_v, d_beta);
+    const uint32_t items = 2 * l->kv_heads + (l->heads * l->vdim + 31) / 32 + l->heads, share = std::max(1u, std::min(64u, (items + 15) / 16));
+    const cudaError_t r = launch(e, zk::delta_inputs_rows_kernel, dim3(u32((tokens + zk::kStrip - 1) / zk::kStrip), share), dim3(256), 0, d, d_proj, u32(ld), u32(tokens),
+                                 d_decay, u32(decay_ld), d_pos, d_q, d_k, d_g, d_v, d_beta);
     if (!e.leave(r, "delta_inputs_rows")) return 0;
     return e.leave(launch(e, zk::conv_ring_update_kernel, dim3((zk::linear_channels(d) + 255) / 256), dim3(256), 0, d, d_proj, u32(ld), u32(tokens), d_pos),
                    "delta_inputs_rows: ring");

@@ -333,12 +333,17 @@ class KipiraxDecoder(Decoder):
                 hidden=torch.zeros((T, round_up(most(L["ff"] or 1 for L in self.layers), 8)), **view),
                 mixed=torch.zeros((T, round_up(most([m.heads * m.vdim for m in deltas] + [max(m.left.heads * m.left.vdim, m.right.heads * m.right.vdim) for m in pairs]), 8)), **view),
                 low=torch.zeros((T, round_up(most(max(L["rank_a"], L["rank_g"]) for L in self.layers if "delta" in L), 8)), **view),
-                q=row(most([m.kv_heads * pitch(m.dim) for m in deltas] + [m.right.heads * pitch(m.right.dim) for m in pairs] + [m.left.heads * m.left.pitch for m in pairs])),
+                q=row(most([m.kv_heads * pitch(m.dim) for m in deltas] + [m.left.heads * m.left.pitch for m in pairs])),
                 k=row(most(m.kv_heads * pitch(m.dim) for m in deltas)),
                 g=row(most([m.heads * pitch(m.dim) for m in deltas] + [m.right.heads * pitch(m.right.dim) for m in pairs])),
                 v=row(most(m.heads * m.vdim for m in deltas)), beta=row(most(m.heads for m in deltas)),
                 decay=row(most(m.heads * m.dim for m in deltas)), gate=row(most(m.heads * m.vdim for m in deltas)),
-                o=row(most([m.heads * m.vdim for m in deltas] + [max(m.left.heads * m.left.pitch, m.right.heads * m.right.vdim) for m in pairs])))
+                o=row(most([m.heads * m.vdim for m in deltas] + [max(m.left.heads * m.left.pitch, m.right.heads * m.right.vdim) for m in pairs])),
+                # the right branch of a parallel mixer runs beside the left one
+                right_q=row(most(m.right.heads * pitch(m.right.dim) for m in pairs)), right_o=row(most(m.right.heads * m.right.vdim for m in pairs)),
+                right_mixed=torch.zeros((T, round_up(most(m.right.heads * m.right.vdim for m in pairs), 8)), **view))
+            self.side = torch.cuda.Stream(device=self.dev)
+            self._fork, self._join = torch.cuda.Event(), torch.cuda.Event()
         return self._pf
 
     def prefill(self, d_tokens, count: int) -> None:
@@ -381,13 +386,18 @@ class KipiraxDecoder(Decoder):
                 gemm(L["o"][0], P(b["mixed"]), ld(width), P(b["y"][0]), W)
             else:
                 a, r = m.left, m.right
+                self._fork.record(self.stream)
+                self.side.wait_event(self._fork)
+                on_side = self.side.cuda_stream
+                be.dev_gated_write_inputs_rows(L["write"], at("right.q"), N, T, P(b["right_q"]), P(b["g"]), on_side)
+                be.dev_state_scan(L["write"], False, P(b["right_q"]), None, P(b["g"]), at("right.v"), N, None, T, P(b["right_o"]), on_side)
+                be.dev_head_outputs_rows(P(b["right_o"]), T, r.heads, r.vdim, r.vdim, P(b["right_mixed"]), ld(r.heads * r.vdim), bf16, on_side, weight=L["write"].norm, eps=cfg.eps)
+                self._join.record(self.side)
                 be.dev_window_attention_rows(L["window"], at("left.q"), at("left.k"), at("left.v"), N, T, P(self.pos), P(b["q"]), P(b["o"]), st)
                 be.dev_head_outputs_rows(P(b["o"]), T, a.heads, a.vdim, a.pitch, P(b["mixed"]), ld(a.heads * a.vdim), bf16, st, gate=at("left.g"), gate_ld=N, gate_mode=1)
                 gemm(L["o"][0], P(b["mixed"]), ld(a.heads * a.vdim), P(b["y"][0]), W)
-                be.dev_gated_write_inputs_rows(L["write"], at("right.q"), N, T, P(b["q"]), P(b["g"]), st)
-                be.dev_state_scan(L["write"], False, P(b["q"]), None, P(b["g"]), at("right.v"), N, None, T, P(b["o"]), st)
-                be.dev_head_outputs_rows(P(b["o"]), T, r.heads, r.vdim, r.vdim, P(b["mixed"]), ld(r.heads * r.vdim), bf16, st, weight=L["write"].norm, eps=cfg.eps)
-                gemm(L["o"][1], P(b["mixed"]), ld(r.heads * r.vdim), P(b["y"][1]), W)
+                self.stream.wait_event(self._join)
+                gemm(L["o"][1], P(b["right_mixed"]), ld(r.heads * r.vdim), P(b["y"][1]), W)
             pending = self._after_mixer(L, b["x"][cur], b["y"][:len(L["o"])])
             if L["ff"] is not None:
                 end()
