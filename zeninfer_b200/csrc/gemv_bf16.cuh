@@ -123,6 +123,7 @@ __global__ void __launch_bounds__(kDenseThreads, 1) gemv_bf16_kernel(const __gri
         for (uint32_t ti = 0; ti < p.tasks; ++ti) {
             const DenseTask& t = p.task[ti];
             const uint32_t padded = dense_units(t.ld) * kDenseUnit;
+#pragma unroll 8
             for (uint32_t i = threadIdx.x; i < padded; i += kDenseThreads) xs[x_floats + i] = i < t.K ? __ldcg(t.x + i) : 0.0f;
             x_floats += padded;
         }

@@ -369,18 +369,21 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_c
 
 // One CTA per head: everything from the projections of one token to the output projection's input.  proj: delta rule
 // q | k | v | b | a1 | g1, gated write q | f | v.  out [heads][vdim].
-constexpr int kStepThreads = 512;
-template <bool kDelta>
-__global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj,
+// kMaxQuads: most 16-byte words a lane holds of a column (pitch / 32): up to four, a CTA of 1024 threads takes 128 columns at a time.
+__host__ __device__ constexpr int step_threads(int max_quads) { return max_quads <= 4 ? 1024 : 512; }
+__host__ __device__ inline uint32_t step_low_floats(const LinearLayer& l) { return ((l.rank_a + 63) & ~63u) + ((l.rank_g + 63) & ~63u); }
+template <bool kDelta, int kMaxQuads>
+__global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj,
                                                                   const int* __restrict__ pos_ptr, float* __restrict__ out) {
-    constexpr uint32_t kWarps = kStepThreads / 32;
+    constexpr uint32_t kStepThreads = step_threads(kMaxQuads), kWarps = kStepThreads / 32;
+    extern __shared__ __align__(16) float low[];                   // delta rule: a1 and g1 outputs, each padded with zeros to 64
     __shared__ __align__(16) float q[256], k[256], g[256];
     __shared__ float v[256], o[256], gate[256];
     const uint32_t h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7, quads = l.pitch / 32;
     pdl_launch_dependents();
     // rows of the rank projections, eight lanes to a row (decays first, then the gate): weights, so their first kAhead words per
     // lane are fetched while the previous launch is still running
-    constexpr uint32_t kAhead = 8;
+    constexpr uint32_t kAhead = kMaxQuads <= 4 ? 4 : 8;
     uint4 ahead[kAhead];
     const uint32_t words = kDelta ? (max(l.a2_ld, l.g2_ld) + 63) / 64 : 0;      // 16-byte words per lane and row
     auto rank_row = [&](uint32_t r, uint32_t& ld) -> const __nv_bfloat16* {     // null: padding
@@ -405,16 +408,20 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_c
     // the first columns' state words are on their way while the token's vectors are formed
     float* const state = l.state + static_cast<size_t>(h) * l.vdim * l.pitch + part * 4;
     uint32_t col = warp * 4 + (lane >> 3);
-    float4 pre[8];
+    float4 pre[kMaxQuads];
 #pragma unroll
-    for (uint32_t i = 0; i < 8; ++i)
+    for (uint32_t i = 0; i < kMaxQuads; ++i)
         pre[i] = (i < quads && col < l.vdim) ? __ldcg(reinterpret_cast<const float4*>(state + static_cast<size_t>(col) * l.pitch + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
     float beta = 0.0f;
     if (kDelta) {
         const int pos = *pos_ptr;
         const uint32_t channels = linear_channels(l), kd = l.kv_heads * l.dim, qh = h / (l.heads / l.kv_heads);
-        const float* low_a = proj + channels + l.heads;
-        const float* low_g = low_a + l.rank_a;
+        const uint32_t pad_a = (l.rank_a + 63) & ~63u;
+        for (uint32_t i = threadIdx.x; i < step_low_floats(l); i += kStepThreads) {
+            const bool is_g = i >= pad_a;
+            const uint32_t c = is_g ? i - pad_a : i;
+            low[i] = c < (is_g ? l.rank_g : l.rank_a) ? __ldcg(proj + channels + l.heads + (is_g ? l.rank_a : 0u) + c) : 0.0f;
+        }
         beta = logistic(__ldcg(proj + channels + h));
         const bool owner = h % (l.heads / l.kv_heads) == 0;        // one CTA per q/k head keeps its ring
         float* slot = l.ring + static_cast<size_t>(static_cast<uint32_t>(pos) % l.taps) * channels;
@@ -429,19 +436,22 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_c
             }
             (is_v ? v : is_k ? k : q)[d] = y;
         }
+        __syncthreads();
         // decays and output gate
         const float a_scale = -expf(l.a_log[h]);
         uint32_t r = warp * 4 + (lane >> 3), word = 0;
         float acc = 0.0f;
         auto take = [&](const uint4& w) {
             const bool is_g = r >= l.pitch;
-            const float* low = is_g ? low_g : low_a;
-            const uint32_t c = (word * 8 + part) * 8, rank = is_g ? l.rank_g : l.rank_a;
-            float x[8];
-#pragma unroll
-            for (int j = 0; j < 8; ++j) x[j] = c + j < rank ? __ldcg(low + c + j) : 0.0f;
-            dense_fma8(w, x, acc);
-            if (++word < words) return;
+            const uint32_t c = (word * 8 + part) * 8;
+            if (c < (is_g ? l.g2_ld : l.a2_ld)) {
+                const float4* in = reinterpret_cast<const float4*>(low + (is_g ? pad_a : 0u) + c);
+                const float4 x0 = in[0], x1 = in[1];
+                const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+                dense_fma8(w, x, acc);
+            }
+            ++word;
+            if (word != words) return;
 #pragma unroll
             for (int s = 1; s < 8; s <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, s);
             if (part == 0 && r < l.pitch + l.vdim) {
@@ -491,10 +501,10 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_c
         col = base + (lane >> 3);
         const bool on = col < l.vdim;
         float* mine = state + static_cast<size_t>(col) * l.pitch;
-        float4 s[8];
+        float4 s[kMaxQuads];
         float u = on ? v[col] : 0.0f, dot = 0.0f;
 #pragma unroll
-        for (uint32_t i = 0; i < 8; ++i) {
+        for (uint32_t i = 0; i < kMaxQuads; ++i) {
             if (i >= quads) break;
             s[i] = base == warp * 4 ? pre[i] : on ? __ldcg(reinterpret_cast<const float4*>(mine + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
             const float4 gg = reinterpret_cast<const float4*>(g)[i * 8 + part], kk = reinterpret_cast<const float4*>(k)[i * 8 + part];
@@ -508,7 +518,7 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(const __grid_c
         }
         float acc = 0.0f;
 #pragma unroll
-        for (uint32_t i = 0; i < 8; ++i) {
+        for (uint32_t i = 0; i < kMaxQuads; ++i) {
             if (i >= quads) break;
             const float4 qq = reinterpret_cast<const float4*>(q)[i * 8 + part], kk = reinterpret_cast<const float4*>(k)[i * 8 + part];
             s[i] = make_float4(fmaf(kk.x, u, s[i].x), fmaf(kk.y, u, s[i].y), fmaf(kk.z, u, s[i].z), fmaf(kk.w, u, s[i].w));

@@ -271,9 +271,12 @@ int zen_cuda_dev_window_attention_step(const zen_cuda_window_attention* a, const
 int zen_cuda_dev_state_step(const zen_cuda_linear_layer* l, int delta, const float* d_proj, const int* d_pos, float* d_out, void* stream) {
     ZC_ENTER(stream, linear_ok(l, delta) && d_proj && d_pos && d_out, "state_step");
     const zk::LinearLayer d = device_form(*l, delta);
-    return e.leave(delta ? launch(e, zk::state_step_kernel<true>, dim3(l->heads), dim3(zk::kStepThreads), 0, d, d_proj, d_pos, d_out)
-                         : launch(e, zk::state_step_kernel<false>, dim3(l->heads), dim3(zk::kStepThreads), 0, d, d_proj, d_pos, d_out),
-                   "state_step");
+    const bool small = d.pitch <= 128;
+    auto go = [&](auto kernel, size_t smem) { return launch(e, kernel, dim3(l->heads), dim3(zk::step_threads(small ? 4 : 8)), smem, d, d_proj, d_pos, d_out); };
+    const size_t low = delta ? zk::step_low_floats(d) * sizeof(float) : 0;
+    const cudaError_t r = delta ? (small ? go(zk::state_step_kernel<true, 4>, low) : go(zk::state_step_kernel<true, 8>, low))
+                                : (small ? go(zk::state_step_kernel<false, 4>, 0) : go(zk::state_step_kernel<false, 8>, 0));
+    return e.leave(r, "state_step");
 }
 
 int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, const float* d_decay, size_t decay_ld, size_t tokens, const int* d_pos,
