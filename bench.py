@@ -1229,9 +1229,9 @@ def run_kipirax(args) -> dict | None:
                     "dense_gemm down": (gemm(ld_["down"], F, W), 2 * W * F + T * (2 * F + 4 * W), 2 * T * W * F, tensor_peak),
                     "delta_inputs_rows": (lambda: be.dev_delta_inputs_rows(ld_["delta"], P(b["proj"]), ld_["proj_rows"], P(b["decay"]), H * D, T, P(dec.pos), P(b["q"]), P(b["k"]), P(b["g"]),
                                                                            P(b["v"]), P(b["beta"]), st), T * H * D * 4 * 8, 0, 1),
-                    "delta state_scan": (lambda: be.dev_state_scan(ld_["delta"], True, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), H * D, P(b["beta"]), T, P(b["o"]), st),
+                    "delta state_scan": (lambda: be.dev_state_scan(ld_["delta"], True, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), H * D, P(b["beta"]), T, P(b["scan"]), b["scan"].numel(), P(b["o"]), st),
                                          T * H * D * 4 * 5 + state, 0, 1),
-                    "gated state_scan": (lambda: be.dev_state_scan(lp["write"], False, P(b["q"]), None, P(b["g"]), P(b["v"]), H * D, None, T, P(b["o"]), st), T * H * D * 4 * 4 + state, 0, 1),
+                    "gated state_scan": (lambda: be.dev_state_scan(lp["write"], False, P(b["q"]), None, P(b["g"]), P(b["v"]), H * D, None, T, P(b["right_scan"]), b["right_scan"].numel(), P(b["o"]), st), T * H * D * 4 * 4 + state, 0, 1),
                     "head_outputs_rows": (lambda: be.dev_head_outputs_rows(P(b["o"]), T, H, D, D, P(b["mixed"]), H * D, True, st, weight=ld_["delta"].norm, eps=1e-6, gate=P(b["gate"]),
                                                                            gate_ld=H * D, gate_mode=2), T * H * D * 10, 0, 1),
                     "window_attention_rows (+ norms, append)": (lambda: be.dev_window_attention_rows(lp["window"], P(b["proj"]), P(b["proj"]) + 4 * H * D, P(b["proj"]) + 4 * (H + G) * D,

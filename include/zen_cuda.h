@@ -584,9 +584,11 @@ int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* 
                                    const int* d_pos, float* d_q, float* d_k, float* d_g, float* d_v, float* d_beta, void* stream);
 /* Gated write: d_q, d_f [tokens][heads][pitch]. */
 int zen_cuda_dev_gated_write_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, size_t tokens, float* d_q, float* d_f, void* stream);
-/* The recurrence over the block: d_out [tokens][heads][vdim].  d_v: rows of pitch v_ld.  d_k and d_beta: delta rule only. */
+/* The recurrence over the block: d_out [tokens][heads][vdim].  d_v: rows of pitch v_ld.  d_k and d_beta: delta rule only.  The
+ * workspace (16-byte aligned) holds what is formed for every eight tokens before the recurrence runs. */
+size_t zen_cuda_state_scan_workspace_bytes(const zen_cuda_linear_layer* l, int delta, size_t tokens);
 int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int delta, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld,
-                            const float* d_beta, size_t tokens, float* d_out, void* stream);
+                            const float* d_beta, size_t tokens, void* d_workspace, size_t workspace_bytes, float* d_out, void* stream);
 
 /* The device-side error channel.  Synchronises `stream` (NULL: the backend's own), then reads and clears the error word
  * the kernels set.  Returns

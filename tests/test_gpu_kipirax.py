@@ -288,6 +288,7 @@ def run_linear(be, kind, m, case, cuts):
     pitch, N = round_up(dim, 32), proj.shape[1]
     P = lambda t: t.data_ptr()
     dp, pos, got, done = dev(proj), dev([0], np.int32), np.zeros_like(want), 0
+    ws = zeros(be.state_scan_workspace_bytes(layer, kind == "delta", T) // 4)
     q, k, gd, v, beta, o = zeros(T, g, pitch), zeros(T, g, pitch), zeros(T, h, pitch), zeros(T, h * vdim), zeros(T, h), zeros(T, h, vdim)
     y, at = zeros(T, h * vdim), {}
     col = 0
@@ -301,11 +302,11 @@ def run_linear(be, kind, m, case, cuts):
             be.dev_dense_gemm(extra["a2"], P(row) + 4 * at["a1"], N, n, P(decay), h * dim, exact=True)
             be.dev_dense_gemm(extra["g2"], P(row) + 4 * at["g1"], N, n, P(gate), h * vdim, exact=True)
             be.dev_delta_inputs_rows(layer, P(row), N, P(decay), h * dim, n, P(pos), P(q), P(k), P(gd), P(v), P(beta))
-            be.dev_state_scan(layer, True, P(q), P(k), P(gd), P(v), h * vdim, P(beta), n, P(o))
+            be.dev_state_scan(layer, True, P(q), P(k), P(gd), P(v), h * vdim, P(beta), n, P(ws), 4 * ws.numel(), P(o))
             be.dev_head_outputs_rows(P(o), n, h, vdim, vdim, P(y), h * vdim, False, weight=layer.norm, eps=layer.eps, gate=P(gate), gate_ld=h * vdim, gate_mode=2)
         else:
             be.dev_gated_write_inputs_rows(layer, P(row), N, n, P(q), P(gd))
-            be.dev_state_scan(layer, False, P(q), None, P(gd), P(row) + 4 * at["v"], N, None, n, P(o))
+            be.dev_state_scan(layer, False, P(q), None, P(gd), P(row) + 4 * at["v"], N, None, n, P(ws), 4 * ws.numel(), P(o))
             be.dev_head_outputs_rows(P(o), n, h, vdim, vdim, P(y), h * vdim, False, weight=layer.norm, eps=layer.eps)
         got[done:done + n] = host(y)[:n]
         done += n
@@ -355,7 +356,10 @@ def test_scan_keeps_a_write_far_away(be):
     P = lambda t: t.data_ptr()
     layer = LinearLayer(h, h, dim, vdim, 1, 1e-5, conv=P(dummy), a_log=P(dummy), dt_bias=P(dummy), a2=a2, g2=g2, norm=P(norm), ring=P(dummy), state=P(state))
     d = [dev(t) for t in (q, k, g, v, beta)]
-    be.dev_state_scan(layer, True, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(out))
+    ws = zeros(be.state_scan_workspace_bytes(layer, True, T) // 4)
+    be.dev_state_scan(layer, True, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(ws), 4 * ws.numel(), P(out))
+    with pytest.raises(BackendError):
+        be.dev_state_scan(layer, True, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(ws), 4 * ws.numel() - 4, P(out))
     close(host(out)[-1], v[3], 1e-4)
     be.dev_free(a2), be.dev_free(g2)
 

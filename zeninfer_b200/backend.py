@@ -48,7 +48,7 @@ ABI_SYMBOLS = (
     "zen_cuda_dev_embed_rows_q8_0", "zen_cuda_dev_rope_kv_append_rows", "zen_cuda_dev_attention_prefill",
     "zen_cuda_dev_sublayer_end_rows", "zen_cuda_dev_dense_gemv", "zen_cuda_dev_dense_gemm", "zen_cuda_dev_embed_rows_bf16", "zen_cuda_dev_rows_view",
     "zen_cuda_dev_head_outputs_rows", "zen_cuda_dev_window_attention_rows", "zen_cuda_dev_window_attention_step", "zen_cuda_dev_state_step",
-    "zen_cuda_dev_delta_inputs_rows", "zen_cuda_dev_gated_write_inputs_rows", "zen_cuda_dev_state_scan",
+    "zen_cuda_dev_delta_inputs_rows", "zen_cuda_dev_gated_write_inputs_rows", "zen_cuda_dev_state_scan", "zen_cuda_state_scan_workspace_bytes",
 )
 
 
@@ -220,7 +220,9 @@ def load_library(path: str | None = None) -> C.CDLL:
     lib.zen_cuda_dev_state_step.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp]
     lib.zen_cuda_dev_delta_inputs_rows.argtypes = [C.POINTER(LinearLayer), vp, sz, vp, sz, sz, vp, vp, vp, vp, vp, vp, vp]
     lib.zen_cuda_dev_gated_write_inputs_rows.argtypes = [C.POINTER(LinearLayer), vp, sz, sz, vp, vp, vp]
-    lib.zen_cuda_dev_state_scan.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp, sz, vp, sz, vp, vp]
+    lib.zen_cuda_dev_state_scan.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp, sz, vp, sz, vp, sz, vp, vp]
+    lib.zen_cuda_state_scan_workspace_bytes.argtypes = [C.POINTER(LinearLayer), i, sz]
+    lib.zen_cuda_state_scan_workspace_bytes.restype = sz
     return lib
 
 
@@ -676,9 +678,12 @@ class Backend:
         if not self.lib.zen_cuda_dev_gated_write_inputs_rows(C.byref(layer), d_proj, ld, tokens, d_q, d_f, stream):
             self._fail("dev_gated_write_inputs_rows")
 
+    def state_scan_workspace_bytes(self, layer: LinearLayer, delta: bool, tokens: int) -> int:
+        return int(self.lib.zen_cuda_state_scan_workspace_bytes(C.byref(layer), int(delta), tokens))
+
     def dev_state_scan(self, layer: LinearLayer, delta: bool, d_q: int, d_k: int | None, d_g: int, d_v: int, v_ld: int, d_beta: int | None, tokens: int,
-                       d_out: int, stream: int = 0) -> None:
-        if not self.lib.zen_cuda_dev_state_scan(C.byref(layer), int(delta), d_q, d_k, d_g, d_v, v_ld, d_beta, tokens, d_out, stream):
+                       d_workspace: int, workspace_bytes: int, d_out: int, stream: int = 0) -> None:
+        if not self.lib.zen_cuda_dev_state_scan(C.byref(layer), int(delta), d_q, d_k, d_g, d_v, v_ld, d_beta, tokens, d_workspace, workspace_bytes, d_out, stream):
             self._fail("dev_state_scan")
 
     def dev_check(self, stream: int = 0) -> None:

@@ -11,6 +11,7 @@ import re
 import shutil
 import subprocess
 import sys
+import time
 
 PKG = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(PKG, "csrc")
@@ -64,7 +65,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
         if not force and not _stale(LIB, everything):
             return LIB
         flags = ["-Xptxas=-v", *NVCC_FLAGS] if verbose else NVCC_FLAGS
-        jobs, objects = [], []
+        jobs, objects, began = [], [], time.time()
         for src, needs in inputs.items():
             obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
             objects.append(obj)
@@ -75,8 +76,10 @@ def build(force: bool = False, verbose: bool = False) -> str:
         for cmd, code in codes:
             if code:
                 raise subprocess.CalledProcessError(code, cmd)
+            os.utime(cmd[cmd.index("-o") + 1], (began, began))     # a source edited while it was compiled is newer than its object
         fresh = LIB + ".new"
         subprocess.run([nvcc, *NVCC_FLAGS, "-shared", "-o", fresh, *objects], check=True)
+        os.utime(fresh, (began, began))
         os.replace(fresh, LIB)
     return LIB
 

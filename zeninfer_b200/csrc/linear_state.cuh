@@ -3,8 +3,8 @@
 //   delta rule    S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q      (g per key channel)
 //   gated write   S <- f * S + (1 - f) v^T;           o = S^T q                       (f per key channel, no key)
 //
-// state_scan_kernel walks a block of tokens with the state in registers, state_step_kernel takes one token and does everything
-// between the layer's input projections and its output projection.  The kernels around the scan form its inputs (short causal
+// state_scan_kernel walks a block of tokens, eight at a time, with the state in registers; state_step_kernel takes one token and
+// does everything between the layer's input projections and its output projection.  The kernels around the scan form its inputs (short causal
 // convolution, unit norms, decays, gates) for all tokens at once.
 //
 // Device layout of a state: [heads][vdim][pitch], pitch = dim rounded up to 32 and zero beyond dim, so that eight lanes read a
@@ -181,6 +181,21 @@ __global__ void __launch_bounds__(256) gated_write_inputs_rows_kernel(const __gr
 }
 
 // ---- the scan --------------------------------------------------------------------------------------------------------
+//
+// Eight tokens at a time.  With S the state before a group and G_t = g_1 ... g_t (channel by channel), unrolling the recurrence gives
+//
+//   u_t = beta_t (v_t - (k_t G_t) . S - sum_{s<t} A_ts u_s)      A_ts = sum_d k_t k_s g_{s+1} ... g_t
+//   o_t = (q_t G_t) . S + sum_{s<=t} B_ts u_s                    B_ts = sum_d q_t k_s g_{s+1} ... g_t
+//   S  <- G_8 S + sum_s (k_s g_{s+1} ... g_8) u_s
+//
+// so that all products with S of a group are independent of one another, and what is sequential is an 8 x 8 triangular system:
+// u = T (v - (k G) . S) with T = (1 + diag(beta) A)^-1 diag(beta).  Only products of decays appear, never a quotient, so nothing
+// overflows however strong they are.  state_groups_kernel forms, for every group and head at once, the scaled vectors and the
+// small matrices T and M (o_t = (q_t G_t) . S + sum_s M_ts w_s with w = v - (k G) . S, M = B T); state_scan_kernel walks the groups.
+// The gated write has u = v and k = 1 - f: no T, and M = B.
+//
+// A group's record, fp32: [k G: 8 x pitch, delta rule only] [q G: 8 x pitch] [k g...: 8 x pitch] [G_8: pitch] [T: 8 x 8, delta only]
+// [M: 8 x 8].  Missing tokens at the end of a block have g = 1, k = q = beta = 0 and leave the state as it is.
 
 struct ScanParams {
     const float* q;        // [T][q_heads][pitch]
@@ -188,181 +203,262 @@ struct ScanParams {
     const float* g;        // [T][heads][pitch]
     const float* v;        // [T][v_ld], head h's values at column h * vdim
     const float* beta;     // [T][heads]; delta rule only
+    float* records;        // [groups][heads][record]
     float* state;          // [heads][vdim][pitch]
     float* out;            // [T][heads][vdim]
     uint32_t tokens, heads, q_heads, vdim, v_ld;
 };
 
-constexpr int kScanThreads = 128, kScanColumns = 32, kScanTokens = 8, kScanStages = 4;    // columns of S per CTA; tokens per staged block; blocks in flight
+constexpr int kGroup = 8;                                                    // tokens per group
+constexpr int kScanThreads = 128, kScanColumns = 32, kScanStages = 4;       // columns of S per CTA; groups in flight
+__host__ __device__ constexpr uint32_t scan_record_floats(uint32_t pitch, bool delta) { return (delta ? 25 : 17) * pitch + (delta ? 128 : 64); }
 template <int kQuads, bool kDelta>
-__host__ __device__ constexpr uint32_t scan_token_floats() { return (kDelta ? 3 : 2) * kQuads * 32 + kScanColumns + 4; }
+__host__ __device__ constexpr uint32_t scan_smem_bytes() {
+    return (kScanStages * (scan_record_floats(kQuads * 32, kDelta) + kGroup * kScanColumns) + (kScanThreads / 32) * kGroup * 8) * 4;
+}
+
+// 64 values per lane -> their sums over the warp, two per lane: lane l keeps values 2 l and 2 l + 1.
+__device__ __forceinline__ void warp_sum64(float (&v)[64], int lane) {
+#pragma unroll
+    for (int o = 16; o >= 1; o >>= 1) {
+        const bool hi = lane & o;
+#pragma unroll
+        for (int i = 0; i < 2 * o; ++i) v[i] = (hi ? v[i + 2 * o] : v[i]) + __shfl_xor_sync(0xffffffffu, hi ? v[i] : v[i + 2 * o], o);
+    }
+}
+
+// One warp per (group, head); a lane takes channels lane, lane + 32, ...  Grid: ceil(groups * heads / 4).
 template <int kQuads, bool kDelta>
-__host__ __device__ constexpr uint32_t scan_smem_bytes() { return kScanStages * kScanTokens * scan_token_floats<kQuads, kDelta>() * 4; }
+__global__ void __launch_bounds__(128) state_groups_kernel(const __grid_constant__ ScanParams p) {
+    constexpr uint32_t kPitch = kQuads * 32, kRecord = scan_record_floats(kPitch, kDelta);
+    __shared__ float sums[4][64], t_matrix[4][64];
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t groups = (p.tokens + kGroup - 1) / kGroup, item = blockIdx.x * 4 + warp;
+    if (item >= groups * p.heads) return;                       // whole warps leave; there is no block barrier below
+    const uint32_t h = item % p.heads, t0 = item / p.heads * kGroup, qh = h / (p.heads / p.q_heads);
+    float* rec = p.records + static_cast<size_t>(item) * kRecord;
+    float* const q_out = rec + (kDelta ? 8 * kPitch : 0);
+    float* const k_out = q_out + 8 * kPitch;
+    float* const g_out = k_out + 8 * kPitch;
+    // entry of (t, s): A's at t (t - 1) / 2 + s for s < t, B's at 28 + t (t + 1) / 2 + s for s <= t
+    float acc[64];
+#pragma unroll
+    for (int i = 0; i < 64; ++i) acc[i] = 0.0f;
+#pragma unroll 1
+    for (int j = 0; j < kQuads; ++j) {
+        const uint32_t d = lane + 32 * j;
+        float g[kGroup], k[kGroup], q[kGroup];
+#pragma unroll
+        for (int t = 0; t < kGroup; ++t) {
+            const bool on = t0 + t < p.tokens;
+            g[t] = on ? __ldcg(p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch + d) : 1.0f;
+            q[t] = on ? __ldcg(p.q + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch + d) : 0.0f;
+            k[t] = !kDelta ? 1.0f - g[t] : on ? __ldcg(p.k + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch + d) : 0.0f;
+        }
+        float run = 1.0f;
+#pragma unroll
+        for (int t = 0; t < kGroup; ++t) {
+            run *= g[t];
+            if (kDelta) rec[t * kPitch + d] = k[t] * run;
+            q_out[t * kPitch + d] = q[t] * run;
+        }
+        g_out[d] = run;
+#pragma unroll
+        for (int s = 0; s < kGroup; ++s) {
+            float w = k[s];
+            acc[28 + s * (s + 1) / 2 + s] = fmaf(q[s], w, acc[28 + s * (s + 1) / 2 + s]);
+#pragma unroll
+            for (int t = s + 1; t < kGroup; ++t) {
+                w *= g[t];
+                if (kDelta) acc[t * (t - 1) / 2 + s] = fmaf(k[t], w, acc[t * (t - 1) / 2 + s]);
+                acc[28 + t * (t + 1) / 2 + s] = fmaf(q[t], w, acc[28 + t * (t + 1) / 2 + s]);
+            }
+            k_out[s * kPitch + d] = w;
+        }
+    }
+    warp_sum64(acc, lane);
+    sums[warp][2 * lane] = acc[0];
+    sums[warp][2 * lane + 1] = acc[1];
+    __syncwarp();
+    float* const m_out = g_out + kPitch + (kDelta ? 64 : 0);
+    if (kDelta) {
+        if (lane < kGroup) {                                    // column `lane` of T by forward substitution
+            float column[kGroup];
+#pragma unroll
+            for (int t = 0; t < kGroup; ++t) {
+                float r = static_cast<int>(lane) == t ? 1.0f : 0.0f;
+#pragma unroll
+                for (int s = 0; s < t; ++s) r = fmaf(-sums[warp][t * (t - 1) / 2 + s], column[s], r);
+                column[t] = t0 + t < p.tokens ? r * __ldcg(p.beta + static_cast<size_t>(t0 + t) * p.heads + h) : 0.0f;
+                t_matrix[warp][t * 8 + lane] = column[t];
+                g_out[kPitch + t * 8 + lane] = column[t];
+            }
+        }
+        __syncwarp();
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {                               // two entries of M per lane
+        const int t = (lane * 2 + e) / 8, c = (lane * 2 + e) % 8;
+        float m = 0.0f;
+        if (kDelta) {
+            for (int s = c; s <= t; ++s) m = fmaf(sums[warp][28 + t * (t + 1) / 2 + s], t_matrix[warp][s * 8 + c], m);
+        } else if (c <= t) {
+            m = sums[warp][28 + t * (t + 1) / 2 + c];
+        }
+        m_out[t * 8 + c] = m;
+    }
+}
 
 __device__ __forceinline__ void cp_async_4(float* smem_dst, const float* gmem_src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst))), "l"(gmem_src) : "memory");
 }
+__device__ __forceinline__ uint64_t pf_add(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
 
-// A CTA takes 32 columns of one head's state (its value channels), a warp eight of them.  A column's rows are spread over eight
-// lanes, lane `part` holding the 16-byte words part, part + 8, ...; a lane holds two columns, so a word of q, k or g read from
-// shared memory serves both.  The state never leaves the registers between the block's first and last token; arithmetic is packed
-// fp32 pairs.  Tokens go in groups of eight: only the delta rule's own sum is reduced token by token (it is what the next token
-// waits for); the read-outs of a group stay as partial sums and are reduced together, after which lane `part` holds token `part`'s.
-// A group's missing tokens at the end of the block are staged as g = 1 and zeros: they leave the state as it is.
-// kQuads = pitch / 32.  Grid: (ceil(vdim / 32), heads).
+// sums[t][c] (8 tokens x 4 pairs of columns, partial per lane) -> the warp's sum of token lane / 4, pair lane % 4.
+__device__ __forceinline__ uint64_t warp_sum_pairs(uint64_t (&v)[kGroup][4], uint32_t lane) {
+    auto exchange = [](uint64_t keep, uint64_t give, int o) { return pf_add(keep, __shfl_xor_sync(0xffffffffu, give, o)); };
+#pragma unroll
+    for (int o = 16, n = 4; n >= 1; o >>= 1, n >>= 1) {         // lane bits 4, 3, 2: the token's bits
+        const bool hi = lane & o;
+#pragma unroll
+        for (int t = 0; t < n; ++t)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) v[t][c] = exchange(hi ? v[t + n][c] : v[t][c], hi ? v[t][c] : v[t + n][c], o);
+    }
+    const bool b1 = lane & 2, b0 = lane & 1;
+    const uint64_t x = exchange(b1 ? v[0][2] : v[0][0], b1 ? v[0][0] : v[0][2], 2), y = exchange(b1 ? v[0][3] : v[0][1], b1 ? v[0][1] : v[0][3], 2);
+    return exchange(b0 ? y : x, b0 ? x : y, 1);
+}
+
+// A CTA takes 32 columns of one head's state (its value channels), a warp eight of them.  A lane holds channels lane, lane + 32, ...
+// of all eight columns, as four packed pairs of columns per channel, so a word of the record read from shared memory serves eight
+// multiply-adds and every lane of the warp reads a different one.  kQuads = pitch / 32.  Grid: (ceil(vdim / 32), heads).
 template <int kQuads, bool kDelta>
 __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_constant__ ScanParams p) {
-    constexpr uint32_t kPitch = kQuads * 32, kToken = scan_token_floats<kQuads, kDelta>();
-    constexpr uint32_t kG = 0, kQ = kPitch, kK = 2 * kPitch, kV = (kDelta ? 3 : 2) * kPitch, kB = kV + kScanColumns;
+    constexpr uint32_t kPitch = kQuads * 32, kRecord = scan_record_floats(kPitch, kDelta), kStage = kRecord + kGroup * kScanColumns;
+    constexpr uint32_t kQ = kDelta ? 8 * kPitch : 0, kK = kQ + 8 * kPitch, kG = kK + 8 * kPitch, kT = kG + kPitch, kM = kT + (kDelta ? 64 : 0);
     extern __shared__ __align__(16) float scan_smem[];
     pdl_launch_dependents();
-    const uint32_t h = blockIdx.y, qh = h / (p.heads / p.q_heads), col_base = blockIdx.x * kScanColumns;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7;
-    const uint32_t local = warp * 8 + (lane >> 3) * 2, c0 = col_base + local;      // this lane's columns: c0, c0 + 1
-    const bool on0 = c0 < p.vdim, on1 = c0 + 1 < p.vdim;
+    const uint32_t h = blockIdx.y, col_base = blockIdx.x * kScanColumns, groups = (p.tokens + kGroup - 1) / kGroup;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c0 = col_base + warp * 8;
+    float* const u_rows = scan_smem + kScanStages * kStage + warp * kGroup * 8;      // this warp's u, [token][column]
     pdl_wait();
-    auto stage = [&](uint32_t t0, uint32_t buf) {
-        float* dst = scan_smem + buf * kScanTokens * kToken;
-        constexpr uint32_t kWords = kPitch / 4, kRows = kDelta ? 3 : 2;
+    auto stage = [&](uint32_t group) {
+        float* dst = scan_smem + (group % kScanStages) * kStage;
+        const float* rec = p.records + (static_cast<size_t>(group) * p.heads + h) * kRecord;
 #pragma unroll 4
-        for (uint32_t i = threadIdx.x; i < kScanTokens * kRows * kWords; i += kScanThreads) {
-            const uint32_t t = i / (kRows * kWords), rest = i % (kRows * kWords), row = rest / kWords, word = rest % kWords;
-            float* d = dst + t * kToken + row * kPitch + word * 4;
-            if (t0 + t < p.tokens) {
-                const float* src = row == 0 ? p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch
-                                            : (row == 1 ? p.q : p.k) + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch;
-                cp_async_16(d, src + word * 4, 16);
-            } else {
-                const float fill = row == 0 ? 1.0f : 0.0f;
-                *reinterpret_cast<float4*>(d) = make_float4(fill, fill, fill, fill);
-            }
-        }
+        for (uint32_t i = threadIdx.x; i < kRecord / 4; i += kScanThreads) cp_async_16(dst + i * 4, rec + i * 4, 16);
 #pragma unroll
-        for (uint32_t i = threadIdx.x; i < kScanTokens * kScanColumns; i += kScanThreads) {
-            const uint32_t t = i / kScanColumns, c = i % kScanColumns;
-            float* d = dst + t * kToken + kV + c;
-            if (col_base + c < p.vdim && t0 + t < p.tokens) cp_async_4(d, p.v + static_cast<size_t>(t0 + t) * p.v_ld + h * p.vdim + col_base + c); else *d = 0.0f;
-        }
-        if (kDelta && threadIdx.x < kScanTokens) {
-            float* d = dst + threadIdx.x * kToken + kB;
-            if (t0 + threadIdx.x < p.tokens) cp_async_4(d, p.beta + static_cast<size_t>(t0 + threadIdx.x) * p.heads + h); else *d = 0.0f;
+        for (uint32_t i = threadIdx.x; i < kGroup * kScanColumns; i += kScanThreads) {
+            const uint32_t t = group * kGroup + i / kScanColumns, c = col_base + i % kScanColumns;
+            float* d = dst + kRecord + i;
+            if (c < p.vdim && t < p.tokens) cp_async_4(d, p.v + static_cast<size_t>(t) * p.v_ld + h * p.vdim + c); else *d = 0.0f;
         }
     };
     for (uint32_t i = 0; i < kScanStages - 1; ++i) {
-        if (i * kScanTokens < p.tokens) stage(i * kScanTokens, i);
+        if (i < groups) stage(i);
         cp_async_commit();
     }
-    uint64_t s[2][kQuads][2];
+    uint64_t s[kQuads][4];
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
-        const float* src = p.state + (static_cast<size_t>(h) * p.vdim + c0 + c) * kPitch + part * 4;
+    for (int j = 0; j < kQuads; ++j)
 #pragma unroll
-        for (int i = 0; i < kQuads; ++i) {
-            const float4 w = (c ? on1 : on0) ? __ldcg(reinterpret_cast<const float4*>(src + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
-            s[c][i][0] = pf_pack(w.x, w.y);
-            s[c][i][1] = pf_pack(w.z, w.w);
+        for (int c = 0; c < 4; ++c) {
+            const float* src = p.state + (static_cast<size_t>(h) * p.vdim + c0 + 2 * c) * kPitch + lane + 32 * j;
+            s[j][c] = pf_pack(c0 + 2 * c < p.vdim ? __ldcg(src) : 0.0f, c0 + 2 * c + 1 < p.vdim ? __ldcg(src + kPitch) : 0.0f);
         }
-    }
-    const uint64_t zero2 = pf_pack(0.0f, 0.0f);
-    uint32_t group = 0;
-    for (uint32_t t0 = 0; t0 < p.tokens; t0 += kScanTokens, ++group) {
+    const uint32_t my_t = lane >> 2, my_pair = lane & 3;
+    for (uint32_t group = 0; group < groups; ++group) {
         cp_async_wait<kScanStages - 2>();           // this group's copies have landed (this thread's; the barrier covers the others')
         __syncthreads();                            // ... and everybody is done with the buffer filled next
-        const uint32_t ahead = t0 + (kScanStages - 1) * kScanTokens;
-        if (ahead < p.tokens) stage(ahead, (group + kScanStages - 1) % kScanStages);
+        if (group + kScanStages - 1 < groups) stage(group + kScanStages - 1);
         cp_async_commit();
-        const float* tok = scan_smem + (group % kScanStages) * kScanTokens * kToken;
-        float out[2][kScanTokens];
+        const float* rec = scan_smem + (group % kScanStages) * kStage;
+        const float* v = rec + kRecord + warp * 8;
+        const uint64_t zero2 = pf_pack(0.0f, 0.0f);
+        auto with_state = [&](const float* rows) {  // rows [8][pitch] . S for this lane's token and pair of columns
+            uint64_t sum[kGroup][4];
 #pragma unroll
-        for (int t = 0; t < kScanTokens; ++t, tok += kToken) {
-            uint64_t g[kQuads][2], q[kQuads][2], k[kQuads][2];
+            for (int t = 0; t < kGroup; ++t)
 #pragma unroll
-            for (int i = 0; i < kQuads; ++i) {
-                const float4 a = reinterpret_cast<const float4*>(tok + kG)[i * 8 + part], b = reinterpret_cast<const float4*>(tok + kQ)[i * 8 + part];
-                g[i][0] = pf_pack(a.x, a.y); g[i][1] = pf_pack(a.z, a.w);
-                q[i][0] = pf_pack(b.x, b.y); q[i][1] = pf_pack(b.z, b.w);
-                if (kDelta) {
-                    const float4 c = reinterpret_cast<const float4*>(tok + kK)[i * 8 + part];
-                    k[i][0] = pf_pack(c.x, c.y); k[i][1] = pf_pack(c.z, c.w);
-                } else {
-                    k[i][0] = pf_pack(1.0f - a.x, 1.0f - a.y); k[i][1] = pf_pack(1.0f - a.z, 1.0f - a.w);
+                for (int j = 0; j < kQuads; ++j) {
+                    const float w = rows[t * kPitch + lane + 32 * j];
+                    const uint64_t ww = pf_pack(w, w);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) sum[t][c] = pf_fma(ww, s[j][c], j ? sum[t][c] : zero2);
                 }
-            }
-            const float2 v2 = *reinterpret_cast<const float2*>(tok + kV + local);
-            float u[2] = {v2.x, v2.y};
-            if (kDelta) {
-                const float beta = tok[kB];
-                float dot[2];
+            return warp_sum_pairs(sum, lane);
+        };
+        const float2 v_mine = *reinterpret_cast<const float2*>(v + my_t * kScanColumns + my_pair * 2);
+        uint64_t w_mine = pf_pack(v_mine.x, v_mine.y);
+        if (kDelta) w_mine = pf_fma(with_state(rec), pf_pack(-1.0f, -1.0f), w_mine);
+        uint64_t o = with_state(rec + kQ), u = zero2;
+        // this lane's rows of T and M times the w of all eight tokens (columns of this lane's pair)
 #pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    uint64_t d0 = zero2, d1 = zero2;
+        for (int t4 = 0; t4 < 2; ++t4) {
+            const float4 m4 = *reinterpret_cast<const float4*>(rec + kM + my_t * 8 + t4 * 4);
+            const float4 x4 = kDelta ? *reinterpret_cast<const float4*>(rec + kT + my_t * 8 + t4 * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float m[4] = {m4.x, m4.y, m4.z, m4.w}, x[4] = {x4.x, x4.y, x4.z, x4.w};
 #pragma unroll
-                    for (int i = 0; i < kQuads; ++i) {
-                        s[c][i][0] = pf_mul(s[c][i][0], g[i][0]);
-                        s[c][i][1] = pf_mul(s[c][i][1], g[i][1]);
-                        d0 = pf_fma(s[c][i][0], k[i][0], d0);
-                        d1 = pf_fma(s[c][i][1], k[i][1], d1);
-                    }
-                    float a, b, e, f;
-                    pf_unpack(d0, a, b);
-                    pf_unpack(d1, e, f);
-                    dot[c] = (a + b) + (e + f);
-                }
-#pragma unroll
-                for (int o = 1; o < 8; o <<= 1) {
-                    dot[0] += __shfl_xor_sync(0xffffffffu, dot[0], o);
-                    dot[1] += __shfl_xor_sync(0xffffffffu, dot[1], o);
-                }
-                u[0] = beta * (u[0] - dot[0]);
-                u[1] = beta * (u[1] - dot[1]);
-            }
-#pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const uint64_t uu = pf_pack(u[c], u[c]);
-                uint64_t d0 = zero2, d1 = zero2;
-#pragma unroll
-                for (int i = 0; i < kQuads; ++i) {
-                    if (kDelta) {
-                        s[c][i][0] = pf_fma(k[i][0], uu, s[c][i][0]);
-                        s[c][i][1] = pf_fma(k[i][1], uu, s[c][i][1]);
-                    } else {
-                        s[c][i][0] = pf_fma(k[i][0], uu, pf_mul(s[c][i][0], g[i][0]));
-                        s[c][i][1] = pf_fma(k[i][1], uu, pf_mul(s[c][i][1], g[i][1]));
-                    }
-                    d0 = pf_fma(s[c][i][0], q[i][0], d0);
-                    d1 = pf_fma(s[c][i][1], q[i][1], d1);
-                }
-                float a, b, e, f;
-                pf_unpack(d0, a, b);
-                pf_unpack(d1, e, f);
-                out[c][t] = (a + b) + (e + f);
+            for (int i = 0; i < 4; ++i) {
+                const uint64_t w = __shfl_sync(0xffffffffu, w_mine, (t4 * 4 + i) * 4 + static_cast<int>(my_pair));
+                o = pf_fma(pf_pack(m[i], m[i]), w, o);
+                if (kDelta) u = pf_fma(pf_pack(x[i], x[i]), w, u);
             }
         }
-        // eight partial read-outs per column over eight lanes: each exchange halves the tokens a lane carries
-        const bool b2 = part & 4, b1 = part & 2, b0 = part & 1;
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-            float r4[4], r2[2];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) r4[i] = (b2 ? out[c][i + 4] : out[c][i]) + __shfl_xor_sync(0xffffffffu, b2 ? out[c][i] : out[c][i + 4], 4);
-#pragma unroll
-            for (int i = 0; i < 2; ++i) r2[i] = (b1 ? r4[i + 2] : r4[i]) + __shfl_xor_sync(0xffffffffu, b1 ? r4[i] : r4[i + 2], 2);
-            const float o = (b0 ? r2[1] : r2[0]) + __shfl_xor_sync(0xffffffffu, b0 ? r2[0] : r2[1], 1);
-            if ((c ? on1 : on0) && t0 + part < p.tokens) p.out[(static_cast<size_t>(t0 + part) * p.heads + h) * p.vdim + c0 + c] = o;
+        const uint32_t t_mine = group * kGroup + my_t, c_mine = c0 + my_pair * 2;
+        if (t_mine < p.tokens) {
+            float o0, o1;
+            pf_unpack(o, o0, o1);
+            float* dst = p.out + (static_cast<size_t>(t_mine) * p.heads + h) * p.vdim + c_mine;
+            if (c_mine < p.vdim) dst[0] = o0;
+            if (c_mine + 1 < p.vdim) dst[1] = o1;
         }
+        const float* u_src = v;
+        uint32_t u_ld = kScanColumns;
+        if (kDelta) {
+            *reinterpret_cast<uint64_t*>(u_rows + my_t * 8 + my_pair * 2) = u;
+            __syncwarp();
+            u_src = u_rows;
+            u_ld = 8;
+        }
+#pragma unroll
+        for (int j = 0; j < kQuads; ++j) {
+            const float g = rec[kG + lane + 32 * j];
+            const uint64_t gg = pf_pack(g, g);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) s[j][c] = pf_mul(s[j][c], gg);
+        }
+#pragma unroll
+        for (int t = 0; t < kGroup; ++t) {
+            const float4 ua = *reinterpret_cast<const float4*>(u_src + t * u_ld), ub = *reinterpret_cast<const float4*>(u_src + t * u_ld + 4);
+            const uint64_t uu[4] = {pf_pack(ua.x, ua.y), pf_pack(ua.z, ua.w), pf_pack(ub.x, ub.y), pf_pack(ub.z, ub.w)};
+#pragma unroll
+            for (int j = 0; j < kQuads; ++j) {
+                const float k = rec[kK + t * kPitch + lane + 32 * j];
+                const uint64_t kk = pf_pack(k, k);
+#pragma unroll
+                for (int c = 0; c < 4; ++c) s[j][c] = pf_fma(kk, uu[c], s[j][c]);
+            }
+        }
+        if (kDelta) __syncwarp();                   // u_rows is read before the next group writes it
     }
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
-        float* dst = p.state + (static_cast<size_t>(h) * p.vdim + c0 + c) * kPitch + part * 4;
-        if (!(c ? on1 : on0)) continue;
+    for (int j = 0; j < kQuads; ++j)
 #pragma unroll
-        for (int i = 0; i < kQuads; ++i) {
-            float4 w;
-            pf_unpack(s[c][i][0], w.x, w.y);
-            pf_unpack(s[c][i][1], w.z, w.w);
-            *reinterpret_cast<float4*>(dst + i * 32) = w;
+        for (int c = 0; c < 4; ++c) {
+            float* dst = p.state + (static_cast<size_t>(h) * p.vdim + c0 + 2 * c) * kPitch + lane + 32 * j;
+            float a, b;
+            pf_unpack(s[j][c], a, b);
+            if (c0 + 2 * c < p.vdim) dst[0] = a;
+            if (c0 + 2 * c + 1 < p.vdim) dst[kPitch] = b;
         }
-    }
 }
 
 // ---- one token -------------------------------------------------------------------------------------------------------

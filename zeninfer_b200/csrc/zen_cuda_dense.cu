@@ -297,16 +297,29 @@ int zen_cuda_dev_gated_write_inputs_rows(const zen_cuda_linear_layer* l, const f
     return e.leave(launch(e, zk::gated_write_inputs_rows_kernel, dim3(u32(tokens)), dim3(256), 0, device_form(*l, 0), d_proj, u32(ld), d_q, d_f), "gated_write_inputs_rows");
 }
 
+size_t zen_cuda_state_scan_workspace_bytes(const zen_cuda_linear_layer* l, int delta, size_t tokens) {
+    if (!l) return 0;
+    return (tokens + zk::kGroup - 1) / zk::kGroup * l->heads * zk::scan_record_floats(pitch32(l->dim), delta != 0) * sizeof(float);
+}
+
 int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int delta, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld, const float* d_beta,
-                            size_t tokens, float* d_out, void* stream) {
+                            size_t tokens, void* d_workspace, size_t workspace_bytes, float* d_out, void* stream) {
     ZC_ENTER(stream, linear_ok(l, delta) && d_q && d_g && d_v && v_ld >= size_t(l->heads) * l->vdim && d_out && tokens && tokens <= 0x7fffffffu && l->heads <= 65535 &&
-                         (!delta || (d_k && d_beta)), "state_scan");
-    const zk::ScanParams p{d_q, d_k, d_g, d_v, d_beta, l->state, d_out, u32(tokens), l->heads, delta ? l->kv_heads : l->heads, l->vdim, u32(v_ld)};
+                         (!delta || (d_k && d_beta)) && d_workspace && !(reinterpret_cast<uintptr_t>(d_workspace) & 15) &&
+                         workspace_bytes >= zen_cuda_state_scan_workspace_bytes(l, delta, tokens), "state_scan");
+    const zk::ScanParams p{d_q, d_k, d_g, d_v, d_beta, static_cast<float*>(d_workspace), l->state, d_out, u32(tokens), l->heads, delta ? l->kv_heads : l->heads, l->vdim, u32(v_ld)};
     const dim3 grid((l->vdim + zk::kScanColumns - 1) / zk::kScanColumns, l->heads);
+    // A grid that fits the SMs one CTA each asks for more than half an SM's shared memory: launched while the groups kernel drains,
+    // its CTAs would otherwise pile up on the first SMs to come free, and each runs for the whole block of tokens.
+    const bool spread = static_cast<uint64_t>(grid.x) * grid.y <= static_cast<uint64_t>(e.sm_count);
+    auto alone = [&](size_t smem) { return spread ? std::max(smem, e.smem_optin / 2 + 1024) : smem; };
     auto go = [&](auto quads) {
         constexpr int kQ = decltype(quads)::value;
-        return delta ? launch(e, zk::state_scan_kernel<kQ, true>, grid, dim3(zk::kScanThreads), zk::scan_smem_bytes<kQ, true>(), p)
-                     : launch(e, zk::state_scan_kernel<kQ, false>, grid, dim3(zk::kScanThreads), zk::scan_smem_bytes<kQ, false>(), p);
+        const dim3 prepare(u32(((tokens + zk::kGroup - 1) / zk::kGroup * l->heads + 3) / 4));
+        const cudaError_t first = delta ? launch(e, zk::state_groups_kernel<kQ, true>, prepare, dim3(128), 0, p) : launch(e, zk::state_groups_kernel<kQ, false>, prepare, dim3(128), 0, p);
+        if (!e.leave(first, "state_scan: groups")) return first;
+        return delta ? launch(e, zk::state_scan_kernel<kQ, true>, grid, dim3(zk::kScanThreads), alone(zk::scan_smem_bytes<kQ, true>()), p)
+                     : launch(e, zk::state_scan_kernel<kQ, false>, grid, dim3(zk::kScanThreads), alone(zk::scan_smem_bytes<kQ, false>()), p);
     };
     cudaError_t r;
     switch (pitch32(l->dim) / 32) {

@@ -342,6 +342,8 @@ class KipiraxDecoder(Decoder):
                 # the right branch of a parallel mixer runs beside the left one
                 right_q=row(most(m.right.heads * pitch(m.right.dim) for m in pairs)), right_o=row(most(m.right.heads * m.right.vdim for m in pairs)),
                 right_mixed=torch.zeros((T, round_up(most(m.right.heads * m.right.vdim for m in pairs), 8)), **view))
+            space = lambda kind, delta: torch.zeros(most(self.be.state_scan_workspace_bytes(L[kind], delta, T) for L in self.layers if kind in L), dtype=torch.uint8, device=self.dev)
+            self._pf.update(scan=space("delta", True), right_scan=space("write", False))
             self.side = torch.cuda.Stream(device=self.dev)
             self._fork, self._join = torch.cuda.Event(), torch.cuda.Event()
         return self._pf
@@ -380,7 +382,7 @@ class KipiraxDecoder(Decoder):
                     be.dev_rows_view(at(n), N, rank, T, P(b["low"]), ld(rank), bf16, st)
                     gemm(handle, P(b["low"]), ld(rank), P(out), rows)
                 be.dev_delta_inputs_rows(L["delta"], P(b["proj"]), N, P(b["decay"]), m.heads * m.dim, T, P(self.pos), P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), P(b["beta"]), st)
-                be.dev_state_scan(L["delta"], True, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), width, P(b["beta"]), T, P(b["o"]), st)
+                be.dev_state_scan(L["delta"], True, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), width, P(b["beta"]), T, P(b["scan"]), b["scan"].numel(), P(b["o"]), st)
                 be.dev_head_outputs_rows(P(b["o"]), T, m.heads, m.vdim, m.vdim, P(b["mixed"]), ld(width), bf16, st, weight=L["delta"].norm, eps=cfg.eps,
                                          gate=P(b["gate"]), gate_ld=width, gate_mode=2)
                 gemm(L["o"][0], P(b["mixed"]), ld(width), P(b["y"][0]), W)
@@ -390,7 +392,7 @@ class KipiraxDecoder(Decoder):
                 self.side.wait_event(self._fork)
                 on_side = self.side.cuda_stream
                 be.dev_gated_write_inputs_rows(L["write"], at("right.q"), N, T, P(b["right_q"]), P(b["g"]), on_side)
-                be.dev_state_scan(L["write"], False, P(b["right_q"]), None, P(b["g"]), at("right.v"), N, None, T, P(b["right_o"]), on_side)
+                be.dev_state_scan(L["write"], False, P(b["right_q"]), None, P(b["g"]), at("right.v"), N, None, T, P(b["right_scan"]), b["right_scan"].numel(), P(b["right_o"]), on_side)
                 be.dev_head_outputs_rows(P(b["right_o"]), T, r.heads, r.vdim, r.vdim, P(b["right_mixed"]), ld(r.heads * r.vdim), bf16, on_side, weight=L["write"].norm, eps=cfg.eps)
                 self._join.record(self.side)
                 be.dev_window_attention_rows(L["window"], at("left.q"), at("left.k"), at("left.v"), N, T, P(self.pos), P(b["q"]), P(b["o"]), st)
