@@ -474,7 +474,7 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
     constexpr uint32_t kStepThreads = step_threads(kMaxQuads), kWarps = kStepThreads / 32;
     extern __shared__ __align__(16) float low[];                   // delta rule: a1 and g1 outputs, each padded with zeros to 64
     __shared__ __align__(16) float q[256], k[256], g[256];
-    __shared__ float v[256], o[256], gate[256];
+    __shared__ float v[256], o[256], gate[256], bias[256], norm[256];
     const uint32_t h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7, quads = l.pitch / 32;
     pdl_launch_dependents();
     // rows of the rank projections, eight lanes to a row (decays first, then the gate): weights, so their first kAhead words per
@@ -500,6 +500,11 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
             if (++word == words) { word = 0; r += kWarps * 4; }
         }
     }
+    // so are the small constants that would otherwise cost a round trip each in the middle of the step
+    for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) norm[i] = __ldg(l.norm + i);
+    if (kDelta)
+        for (uint32_t i = threadIdx.x; i < l.dim; i += kStepThreads) bias[i] = __ldg(l.dt_bias + h * l.dim + i);
+    const float a_scale = kDelta ? -expf(__ldg(l.a_log + h)) : 0.0f;
     pdl_wait();
     // the first columns' state words are on their way while the token's vectors are formed
     float* const state = l.state + static_cast<size_t>(h) * l.vdim * l.pitch + part * 4;
@@ -534,7 +539,6 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
         }
         __syncthreads();
         // decays and output gate
-        const float a_scale = -expf(l.a_log[h]);
         uint32_t r = warp * 4 + (lane >> 3), word = 0;
         float acc = 0.0f;
         auto take = [&](const uint4& w) {
@@ -552,7 +556,7 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
             for (int s = 1; s < 8; s <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, s);
             if (part == 0 && r < l.pitch + l.vdim) {
                 if (is_g) gate[r - l.pitch] = logistic(acc);
-                else g[r] = r < l.dim ? expf(a_scale * softplus_f(acc + l.dt_bias[h * l.dim + r])) : 0.0f;
+                else g[r] = r < l.dim ? expf(a_scale * softplus_f(acc + bias[r])) : 0.0f;
             }
             acc = 0.0f;
             word = 0;
@@ -629,7 +633,7 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
     float ss = 0.0f;
     for (uint32_t i = lane; i < l.vdim; i += 32) ss += o[i] * o[i];          // every warp forms the head's norm itself
     const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(l.vdim) + l.eps);
-    for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) out[h * l.vdim + i] = o[i] * inv * l.norm[i] * (kDelta ? gate[i] : 1.0f);
+    for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) out[h * l.vdim + i] = o[i] * inv * norm[i] * (kDelta ? gate[i] : 1.0f);
 }
 
 }  // namespace zk
