@@ -1276,6 +1276,8 @@ def run_kipirax(args) -> dict | None:
                     "gemm o": (mm(["attn_output"], ["tmp"], "att"), 2 * W * H * D + T * 4 * (W + H * D), 2 * T * W * H * D, 2 * tensor_peak),
                     "gemm gate|up": (mm(["ffn_gate", "ffn_up"], ["gate", "up"], "xn"), 4 * W * F + T * 4 * (W + 2 * F), 4 * T * W * F, 2 * tensor_peak),
                     "gemm down": (mm(["ffn_down"], ["tmp"], "hid"), 2 * W * F + T * 4 * (W + F), 2 * T * W * F, 2 * tensor_peak),
+                    "rope_kv_append rows": (lambda: be.dev_rope_kv_append_rows(P(b["q"]), P(b["k"]), P(b["v"]), T, P(lam.cos), P(lam.sin), P(zero), H, G, D, D // 2, True, P(lam.k_cache[0]),
+                                                                               P(lam.v_cache[0]), positions, st), T * D * 4 * (2 * H + 5 * G), 0, 1),
                     "silu_mul rows": (lambda: be.dev_silu_mul(P(b["gate"]), P(b["up"]), P(b["hid"]), T * F, st), T * F * 12, 0, 1),
                     "attention_prefill": (lambda: be.dev_attention_prefill(P(b["q"]), P(lam.k_cache[0]), P(lam.v_cache[0]), P(zero), P(b["att"]), T, H, G, D, positions, 0.0, 0, st),
                                           T * D * 4 * (2 * H + 2 * G), 2 * T * (T + 1) * H * D, tensor_peak),

@@ -57,7 +57,7 @@ __device__ __forceinline__ float conv_silu(const LinearLayer& l, const float* __
 // ---- inputs of the scan for a block of tokens -------------------------------------------------------------------------
 
 constexpr int kStrip = 8;          // tokens a warp takes at a time: a channel's inputs stay in registers while the taps slide over them
-constexpr int kMaxSlidingTaps = 8; // more taps than this are read again for every token
+constexpr int kMaxSlidingTaps = 4; // more taps than this are read again for every token
 
 // y[i] = silu(convolution) of channel c at tokens t0 .. t0 + n - 1 (n <= kStrip; the rest is not used).
 __device__ __forceinline__ void conv_silu_strip(const LinearLayer& l, const float* __restrict__ x, uint32_t ld, int t0, int n, int pos, uint32_t c,
@@ -69,7 +69,7 @@ __device__ __forceinline__ void conv_silu_strip(const LinearLayer& l, const floa
             if (i < n) y[i] = conv_silu(l, x, ld, t0 + i, pos, c, channels);
         return;
     }
-    float w[kMaxSlidingTaps], in[kMaxSlidingTaps - 1 + kStrip];       // w right-aligned: w[7] is the current token's; in[7 + i]: token t0 + i
+    float w[kMaxSlidingTaps], in[kMaxSlidingTaps - 1 + kStrip];       // w right-aligned: the last is the current token's; in[kMaxSlidingTaps - 1 + i]: token t0 + i
 #pragma unroll
     for (int j = 0; j < kMaxSlidingTaps; ++j) {
         const int tap = j - (kMaxSlidingTaps - taps);
@@ -110,24 +110,34 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
             const uint32_t head = is_q ? item : item - l.kv_heads, c0 = (is_q ? 0u : kd) + head * l.dim;
             float* dst = (is_q ? q : k) + (static_cast<size_t>(t0) * l.kv_heads + head) * l.pitch;
             const float scale = is_q ? 1.0f / sqrtf(static_cast<float>(l.dim)) : 1.0f;
-            float ss[kStrip];
+            float ss[kStrip], last[kStrip];      // last: the head's final 32 channels, which need not go out unscaled
 #pragma unroll
-            for (int i = 0; i < kStrip; ++i) ss[i] = 0.0f;
+            for (int i = 0; i < kStrip; ++i) ss[i] = last[i] = 0.0f;
             for (uint32_t d = lane; d < l.pitch; d += 32) {            // unscaled first: a lane reads back only what it wrote
+                const bool more = d + 32 < l.pitch;
 #pragma unroll
                 for (int i = 0; i < kStrip; ++i) y[i] = 0.0f;
                 if (d < l.dim) conv_silu_strip(l, proj, ld, t0, n, pos, c0 + d, channels, y);
 #pragma unroll
-                for (int i = 0; i < kStrip; ++i)
-                    if (i < n) { ss[i] += y[i] * y[i]; dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] = y[i]; }
+                for (int i = 0; i < kStrip; ++i) {
+                    ss[i] += y[i] * y[i];
+                    last[i] = y[i];
+                    if (more && i < n) dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] = y[i];
+                }
             }
 #pragma unroll
             for (int i = 0; i < kStrip; ++i) ss[i] = scale / sqrtf(warp_sum(ss[i]) + kUnitEps);
-            for (uint32_t d = lane; d < l.pitch; d += 32) {
+            for (uint32_t d = lane; d + 32 < l.pitch; d += 32) {
+                float back[kStrip];
+#pragma unroll
+                for (int i = 0; i < kStrip; ++i) back[i] = i < n ? dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] : 0.0f;
 #pragma unroll
                 for (int i = 0; i < kStrip; ++i)
-                    if (i < n) dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] *= ss[i];
+                    if (i < n) dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + d] = back[i] * ss[i];
             }
+#pragma unroll
+            for (int i = 0; i < kStrip; ++i)
+                if (i < n) dst[static_cast<size_t>(i) * l.kv_heads * l.pitch + l.pitch - 32 + lane] = last[i] * ss[i];
         } else if (item < qk_items + v_items) {
             const uint32_t c = (item - qk_items) * 32 + lane;
             if (c >= nv) continue;
@@ -139,12 +149,12 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
             const uint32_t h = item - qk_items - v_items;
             const float rate = -expf(l.a_log[h]);
             for (uint32_t d = lane; d < l.pitch; d += 32) {
-                const float bias = d < l.dim ? l.dt_bias[h * l.dim + d] : 0.0f;
+                const float bias = d < l.dim ? __ldg(l.dt_bias + h * l.dim + d) : 0.0f;
+#pragma unroll
+                for (int i = 0; i < kStrip; ++i) y[i] = d < l.dim && i < n ? __ldcg(decay + static_cast<size_t>(t0 + i) * decay_ld + h * l.dim + d) : 0.0f;
 #pragma unroll
                 for (int i = 0; i < kStrip; ++i)
-                    if (i < n)
-                        g[(static_cast<size_t>(t0 + i) * l.heads + h) * l.pitch + d] =
-                            d < l.dim ? expf(rate * softplus_f(__ldcg(decay + static_cast<size_t>(t0 + i) * decay_ld + h * l.dim + d) + bias)) : 0.0f;
+                    if (i < n) g[(static_cast<size_t>(t0 + i) * l.heads + h) * l.pitch + d] = d < l.dim ? expf(rate * softplus_f(y[i] + bias)) : 0.0f;
             }
             if (static_cast<int>(lane) < n) beta[static_cast<size_t>(t0 + lane) * l.heads + h] = logistic(__ldcg(proj + static_cast<size_t>(t0 + lane) * ld + channels + h));
         }
