@@ -1,6 +1,6 @@
 """A plain, slow Kipirax in numpy float64: one function per mechanism, token by token where the mechanism is a recurrence.
 
-Checker only: shares nothing with the product path.  Weights are a dict name -> array (any float dtype); `cfg` is the
+Used by tests only; shares nothing with the product path.  Weights are a dict name -> array (any float dtype); `cfg` is the
 model's config.json as a dict.
 """
 from __future__ import annotations
