@@ -486,7 +486,7 @@ int zen_cuda_dev_advance_position(int* d_pos, int delta, void* stream);
 
 /* The end of a sublayer, per row of n values: x_new = x_in + norm(y) (x_in alone when y_a is NULL).  y = y_a; with y_b,
  * y = (rms(y_a) * weight_a + rms(y_b) * weight_b) / 2.  norm: `groups` equal consecutive parts, each divided by
- * sqrt(mean(part^2) + eps), the whole times norm_weight.  The row's reader sees x_new + (before - x_new) * shift (before: the
+ * sqrt(mean(part^2) + eps), the whole times norm_weight; norm_weight NULL: x_new = x_in + y, for one y.  The row's reader sees x_new + (before - x_new) * shift (before: the
  * previous row's x_new; the block's first row reads `before`), or with out_norm the grouped norm of x_new times out_norm, or x_new.
  * x_out: where x_new goes (not x_in itself), or NULL.  keep: receives the last row of x_in, or NULL. */
 typedef struct zen_cuda_sublayer_end {
@@ -515,15 +515,25 @@ typedef struct zen_cuda_dense_task {
     float* d_y;                /* [rows] */
     int act;
     float cap;
+    const float* d_bias;       /* added to d_y before the activation, or NULL */
+    float* d_gated;            /* [gated_pairs] */
+    size_t gated_pairs;        /* the matrix begins with so many pairs of rows: d_gated[i] = silu(row 2 i) * (row 2 i + 1); d_y has the rows behind them */
 } zen_cuda_dense_task;
-/* One launch: d_y = act(W x) for every task, fp32 activations.  pre (or NULL): the input of the single task is what the sublayer
+typedef struct zen_cuda_dense_epilogue {   /* the same for a block of tokens */
+    int act;
+    float cap;
+    const float* d_bias;
+    void* d_gated;             /* [tokens][gated_ld], the type of the product's input rows */
+    size_t gated_ld, gated_pairs;
+} zen_cuda_dense_epilogue;
+/* One launch: d_y = act(W x + bias) for every task, fp32 activations; a task with pairs starts at an even row of the launch.  pre (or NULL): the input of the single task is what the sublayer
  * end's reader sees, formed inside the launch. */
 int zen_cuda_dev_dense_gemv(const zen_cuda_dense_task* tasks, size_t count, const zen_cuda_sublayer_end* pre, void* stream);
-/* d_out[t][r] = act(sum_k x[t][k] w[r][k]) for a block of tokens.  exact 0: x is bf16 (16-byte aligned, pitch a multiple of 8) and the
+/* d_out[t][r] = act(sum_k x[t][k] w[r][k] + bias[r]) for a block of tokens, rows counted behind the gated pairs (epilogue NULL: none of it).  exact 0: x is bf16 (16-byte aligned, pitch a multiple of 8) and the
  * product runs on the tensor cores with fp32 accumulation; exact 1: x is fp32 and so is every multiply-add.  out_bf16: d_out is
  * bf16 (exact 0 only). */
-int zen_cuda_dev_dense_gemm(const zen_cuda_weights* w, const void* d_x, size_t x_ld, size_t tokens, void* d_out, size_t out_ld, int out_bf16, int act,
-                            float cap, int exact, void* stream);
+int zen_cuda_dev_dense_gemm(const zen_cuda_weights* w, const void* d_x, size_t x_ld, size_t tokens, void* d_out, size_t out_ld, int out_bf16,
+                            const zen_cuda_dense_epilogue* epilogue, int exact, void* stream);
 
 /* d_out[t] = embed[tokens[t]] + positions[*d_pos + t]; positions NULL: the embedding alone. */
 int zen_cuda_dev_embed_rows_bf16(const zen_cuda_weights* embed, const zen_cuda_weights* positions, const int64_t* d_tokens, size_t tokens, const int* d_pos,
@@ -531,12 +541,17 @@ int zen_cuda_dev_embed_rows_bf16(const zen_cuda_weights* embed, const zen_cuda_w
 /* Columns [0, n) of rows of pitch src_ld as a product's input [rows][ld], zeros behind them. */
 int zen_cuda_dev_rows_view(const float* d_src, size_t src_ld, size_t n, size_t rows, void* d_dst, size_t ld, int bf16, void* stream);
 /* Heads of `width` values (pitch head_ld in d_o) -> a product's input: each head divided by its root mean square and times weight
- * (weight NULL: no norm), times sigmoid(gate): gate_mode 0 none, 1 one per head, 2 one per value (rows of pitch gate_ld). */
+ * (weight NULL: no norm), times a gate: gate_mode 0 none, 1 sigmoid, one per head, 2 sigmoid, 3 silu, one per value (rows of pitch gate_ld).
+ * Zeros are written behind the heads up to column `fill`. */
 int zen_cuda_dev_head_outputs_rows(const float* d_o, size_t rows, size_t heads, size_t width, size_t head_ld, const float* d_weight, float eps,
-                                   const float* d_gate, size_t gate_ld, int gate_mode, void* d_dst, size_t ld, int bf16, void* stream);
+                                   const float* d_gate, size_t gate_ld, int gate_mode, void* d_dst, size_t ld, size_t fill, int bf16, void* stream);
 
 /* Windowed attention with kept first tokens: position i sees j <= i when i - j < window or j < keep_first; bias != 0 takes
- * slope_h * (i - j) off the scores, slope_h = 2^(-8 (h + 1) / heads).  q and k are RMS-normed per head (q_weight, k_weight, eps).
+ * slope_h * (i - j) off the scores, slope_h = 2^(-8 (h + 1) / heads).  With q_weight and k_weight q and k are RMS-normed per head (eps).
+ * Without them q, k and v (consecutive columns) pass a causal convolution of `taps` taps per channel (taps 0: none; conv and ring
+ * [taps][(heads + kv_heads) qk_dim + kv_heads v_dim], slot = position mod taps), then dimension i and i + rot_pairs of every q and k head
+ * turn by the angle whose cosine and sine are entry i of row `position` of the host-built tables [max_positions][rot_pairs].  Values:
+ * v <- (1 - v_share) v + v_share v_first (v_first NULL: unchanged), then kept at v_keep (or NULL), both [tokens][kv_heads][v_dim].
  * Caches [max_positions][kv_heads][pitch], pitch = max(qk_dim, v_dim) rounded up to 32, at most 256. */
 typedef struct zen_cuda_window_attention {
     uint32_t heads, kv_heads, qk_dim, v_dim, pitch;
@@ -546,12 +561,21 @@ typedef struct zen_cuda_window_attention {
     const float* k_weight;
     float* k_cache;
     float* v_cache;
+    uint32_t rot_pairs, taps;
+    uint32_t gate_values;      /* 1: the step's gate is one value per output, [heads][v_dim] */
+    float v_share;
+    const float* rot_cos;
+    const float* rot_sin;
+    const float* conv;
+    float* ring;
+    const float* v_first;
+    float* v_keep;
 } zen_cuda_window_attention;
-/* A block of rows: q, k, v are columns of the projection rows (pitch ld).  Norms q and k, appends k and v at *d_pos .., and
+/* A block of rows: q, k, v are columns of the projection rows (pitch ld).  Finishes q and k, appends k and v at *d_pos .., and
  * attends; d_q and d_out are [tokens][heads][pitch]. */
 int zen_cuda_dev_window_attention_rows(const zen_cuda_window_attention* a, const float* d_proj_q, const float* d_proj_k, const float* d_proj_v, size_t ld,
                                        size_t tokens, const int* d_pos, float* d_q, float* d_out, void* stream);
-/* One token in one launch; d_out [heads][v_dim], times sigmoid(d_gate[h]) when d_gate is given. */
+/* One token in one launch; d_out [heads][v_dim], times the gate's sigmoid when d_gate is given. */
 int zen_cuda_dev_window_attention_step(const zen_cuda_window_attention* a, const float* d_q, const float* d_k, const float* d_v, const float* d_gate,
                                        const int* d_pos, float* d_out, void* stream);
 
@@ -560,6 +584,8 @@ int zen_cuda_dev_window_attention_step(const zen_cuda_window_attention* a, const
  *                channel (conv [taps][channels]) and silu (ring [taps][2 kv_heads dim + heads vdim], slot = position mod taps), q and k become unit vectors
  *                (q also times dim^-1/2), beta = sigmoid, g = exp(-exp(a_log) softplus(a2 a1 + dt_bias)); output gate sigmoid(g2 g1).
  *   gated write  S <- f * S + (1 - f) v^T; o = S^T q; q = silu, f = lower + (1 - lower) sigmoid(. + f_bias).
+ *   decayed write S <- g * S + k v^T; o = S^T q; q and k rotated as for attention above (rot_pairs 0: not), q times dim^-1/2;
+ *                g = decay[h], or decay NULL: sigmoid(a2 a1 + dt_bias)^inv_tau per channel; output gate silu, one per value.
  * norm [vdim]: weight of the output's RMS norm per head.  dim and vdim at most 256. */
 typedef struct zen_cuda_linear_layer {
     uint32_t heads, kv_heads, dim, vdim, taps;
@@ -574,10 +600,16 @@ typedef struct zen_cuda_linear_layer {
     const float* norm;
     float* ring;
     float* state;
+    const float* decay;
+    float inv_tau;
+    uint32_t rot_pairs, max_positions;
+    const float* rot_cos;
+    const float* rot_sin;
 } zen_cuda_linear_layer;
+enum { ZEN_CUDA_STATE_GATED_WRITE = 0, ZEN_CUDA_STATE_DELTA_RULE = 1, ZEN_CUDA_STATE_DECAYED_WRITE = 2 };
 /* One token, from the projections to the output projection's input [heads * vdim], in one launch.
- * d_proj: q | k | v | b | a1 | g1 (delta) or q | f | v (gated write). */
-int zen_cuda_dev_state_step(const zen_cuda_linear_layer* l, int delta, const float* d_proj, const int* d_pos, float* d_out, void* stream);
+ * d_proj: q | k | v | b | a1 | g1 (delta), q | f | v (gated write) or q | k | v | gate | a1 (decayed write; no a1 with constant decays). */
+int zen_cuda_dev_state_step(const zen_cuda_linear_layer* l, int rule, const float* d_proj, const int* d_pos, float* d_out, void* stream);
 /* A block: the scan's inputs from the projection rows.  Delta rule: d_q, d_k [tokens][kv_heads][pitch], d_g [tokens][heads][pitch],
  * d_v [tokens][heads * vdim], d_beta [tokens][heads]; d_decay [tokens][decay_ld] = a2 a1 without the bias; the ring is brought up to date. */
 int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, const float* d_decay, size_t decay_ld, size_t tokens,
@@ -586,9 +618,12 @@ int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* 
 int zen_cuda_dev_gated_write_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, size_t tokens, float* d_q, float* d_f, void* stream);
 /* The recurrence over the block: d_out [tokens][heads][vdim].  d_v: rows of pitch v_ld.  d_k and d_beta: delta rule only.  The
  * workspace (16-byte aligned) holds what is formed for every eight tokens before the recurrence runs. */
-size_t zen_cuda_state_scan_workspace_bytes(const zen_cuda_linear_layer* l, int delta, size_t tokens);
-int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int delta, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld,
+size_t zen_cuda_state_scan_workspace_bytes(const zen_cuda_linear_layer* l, int rule, size_t tokens);
+int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int rule, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld,
                             const float* d_beta, size_t tokens, void* d_workspace, size_t workspace_bytes, float* d_out, void* stream);
+/* The decayed write over the block, from the projection rows (the step's columns, pitch ld); d_out [tokens][heads][vdim] before norm and gate. */
+int zen_cuda_dev_decayed_write_scan(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, size_t tokens, const int* d_pos, void* d_workspace,
+                                    size_t workspace_bytes, float* d_out, void* stream);
 
 /* The device-side error channel.  Synchronises `stream` (NULL: the backend's own), then reads and clears the error word
  * the kernels set.  Returns

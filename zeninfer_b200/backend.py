@@ -48,7 +48,8 @@ ABI_SYMBOLS = (
     "zen_cuda_dev_embed_rows_q8_0", "zen_cuda_dev_rope_kv_append_rows", "zen_cuda_dev_attention_prefill",
     "zen_cuda_dev_sublayer_end_rows", "zen_cuda_dev_dense_gemv", "zen_cuda_dev_dense_gemm", "zen_cuda_dev_embed_rows_bf16", "zen_cuda_dev_rows_view",
     "zen_cuda_dev_head_outputs_rows", "zen_cuda_dev_window_attention_rows", "zen_cuda_dev_window_attention_step", "zen_cuda_dev_state_step",
-    "zen_cuda_dev_delta_inputs_rows", "zen_cuda_dev_gated_write_inputs_rows", "zen_cuda_dev_state_scan", "zen_cuda_state_scan_workspace_bytes",
+    "zen_cuda_dev_delta_inputs_rows", "zen_cuda_dev_gated_write_inputs_rows", "zen_cuda_dev_state_scan", "zen_cuda_dev_decayed_write_scan",
+    "zen_cuda_state_scan_workspace_bytes",
 )
 
 
@@ -92,6 +93,7 @@ class PickSegment(C.Structure):
 
 
 DENSE_PLAIN, DENSE_SQUARED_RELU, DENSE_SOFTCAP = 0, 1, 2
+GATED_WRITE, DELTA_RULE, DECAYED_WRITE = 0, 1, 2        # rules of a mixer with a matrix state
 
 
 class SublayerEnd(C.Structure):
@@ -100,17 +102,25 @@ class SublayerEnd(C.Structure):
 
 
 class DenseTask(C.Structure):
-    _fields_ = [("w", C.c_void_p), ("d_x", C.c_void_p), ("d_y", C.c_void_p), ("act", C.c_int), ("cap", C.c_float)]
+    _fields_ = [("w", C.c_void_p), ("d_x", C.c_void_p), ("d_y", C.c_void_p), ("act", C.c_int), ("cap", C.c_float), ("d_bias", C.c_void_p),
+                ("d_gated", C.c_void_p), ("gated_pairs", C.c_size_t)]
+
+
+class DenseEpilogue(C.Structure):
+    _fields_ = [("act", C.c_int), ("cap", C.c_float), ("d_bias", C.c_void_p), ("d_gated", C.c_void_p), ("gated_ld", C.c_size_t), ("gated_pairs", C.c_size_t)]
 
 
 class WindowAttention(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "qk_dim", "v_dim", "pitch", "window", "keep_first", "bias", "max_positions")] + [
-        ("scale", C.c_float), ("eps", C.c_float)] + [(n, C.c_void_p) for n in ("q_weight", "k_weight", "k_cache", "v_cache")]
+        ("scale", C.c_float), ("eps", C.c_float)] + [(n, C.c_void_p) for n in ("q_weight", "k_weight", "k_cache", "v_cache")] + [
+        (n, C.c_uint32) for n in ("rot_pairs", "taps", "gate_values")] + [("v_share", C.c_float)] + [
+        (n, C.c_void_p) for n in ("rot_cos", "rot_sin", "conv", "ring", "v_first", "v_keep")]
 
 
 class LinearLayer(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "taps")] + [("eps", C.c_float)] + [
-        (n, C.c_void_p) for n in ("conv", "a_log", "dt_bias", "a2", "g2", "f_bias", "lower", "norm", "ring", "state")]
+        (n, C.c_void_p) for n in ("conv", "a_log", "dt_bias", "a2", "g2", "f_bias", "lower", "norm", "ring", "state", "decay")] + [
+        ("inv_tau", C.c_float), ("rot_pairs", C.c_uint32), ("max_positions", C.c_uint32), ("rot_cos", C.c_void_p), ("rot_sin", C.c_void_p)]
 
 
 def load_library(path: str | None = None) -> C.CDLL:
@@ -211,16 +221,17 @@ def load_library(path: str | None = None) -> C.CDLL:
     lib.zen_cuda_dev_advance_position.argtypes = [vp, i, vp]
     lib.zen_cuda_dev_sublayer_end_rows.argtypes = [C.POINTER(SublayerEnd), sz, vp, sz, i, vp]
     lib.zen_cuda_dev_dense_gemv.argtypes = [C.POINTER(DenseTask), sz, C.POINTER(SublayerEnd), vp]
-    lib.zen_cuda_dev_dense_gemm.argtypes = [vp, vp, sz, sz, vp, sz, i, i, C.c_float, i, vp]
+    lib.zen_cuda_dev_dense_gemm.argtypes = [vp, vp, sz, sz, vp, sz, i, C.POINTER(DenseEpilogue), i, vp]
     lib.zen_cuda_dev_embed_rows_bf16.argtypes = [vp, vp, vp, sz, vp, vp, vp]
     lib.zen_cuda_dev_rows_view.argtypes = [vp, sz, sz, sz, vp, sz, i, vp]
-    lib.zen_cuda_dev_head_outputs_rows.argtypes = [vp, sz, sz, sz, sz, vp, C.c_float, vp, sz, i, vp, sz, i, vp]
+    lib.zen_cuda_dev_head_outputs_rows.argtypes = [vp, sz, sz, sz, sz, vp, C.c_float, vp, sz, i, vp, sz, sz, i, vp]
     lib.zen_cuda_dev_window_attention_rows.argtypes = [C.POINTER(WindowAttention), vp, vp, vp, sz, sz, vp, vp, vp, vp]
     lib.zen_cuda_dev_window_attention_step.argtypes = [C.POINTER(WindowAttention), vp, vp, vp, vp, vp, vp, vp]
     lib.zen_cuda_dev_state_step.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp]
     lib.zen_cuda_dev_delta_inputs_rows.argtypes = [C.POINTER(LinearLayer), vp, sz, vp, sz, sz, vp, vp, vp, vp, vp, vp, vp]
     lib.zen_cuda_dev_gated_write_inputs_rows.argtypes = [C.POINTER(LinearLayer), vp, sz, sz, vp, vp, vp]
     lib.zen_cuda_dev_state_scan.argtypes = [C.POINTER(LinearLayer), i, vp, vp, vp, vp, sz, vp, sz, vp, sz, vp, vp]
+    lib.zen_cuda_dev_decayed_write_scan.argtypes = [C.POINTER(LinearLayer), vp, sz, sz, vp, vp, sz, vp, vp]
     lib.zen_cuda_state_scan_workspace_bytes.argtypes = [C.POINTER(LinearLayer), i, sz]
     lib.zen_cuda_state_scan_workspace_bytes.restype = sz
     return lib
@@ -629,17 +640,21 @@ class Backend:
         if not self.lib.zen_cuda_dev_sublayer_end_rows(C.byref(end), rows, d_view, view_ld, int(view_bf16), stream):
             self._fail("dev_sublayer_end_rows")
 
-    def dev_dense_gemv(self, tasks: Sequence[tuple[int, int | None, int]], stream: int = 0, *, pre: SublayerEnd | None = None, act: int = DENSE_PLAIN,
-                       cap: float = 0.0) -> None:
-        """One launch of bf16 products with single fp32 vectors: (handle, d_x, d_y) each; pre: the input is formed inside."""
-        arr = (DenseTask * len(tasks))(*[DenseTask(h, x, y, act, cap) for h, x, y in tasks])
+    def dev_dense_gemv(self, tasks: Sequence[tuple[int, int | None, int | None]], stream: int = 0, *, pre: SublayerEnd | None = None, act: int = DENSE_PLAIN,
+                       cap: float = 0.0, bias: int | None = None, gated: int | None = None, gated_pairs: int = 0) -> None:
+        """One launch of bf16 products with single fp32 vectors: (handle, d_x, d_y) each; pre: the input is formed inside.  bias is added
+        to d_y; a matrix that begins with gated_pairs pairs of rows leaves silu(first) * second of each at `gated`."""
+        arr = (DenseTask * len(tasks))(*[DenseTask(h, x, y, act, cap, bias, gated, gated_pairs) for h, x, y in tasks])
         if not self.lib.zen_cuda_dev_dense_gemv(arr, len(tasks), C.byref(pre) if pre is not None else None, stream):
             self._fail("dev_dense_gemv")
 
     def dev_dense_gemm(self, handle: int, d_x: int, x_ld: int, tokens: int, d_out: int, out_ld: int, stream: int = 0, *, out_bf16: bool = False,
-                       act: int = DENSE_PLAIN, cap: float = 0.0, exact: bool = False) -> None:
-        """A bf16 matrix times a block of tokens: bf16 rows on the tensor cores, or (exact) fp32 rows in fp32 multiply-adds."""
-        if not self.lib.zen_cuda_dev_dense_gemm(handle, d_x, x_ld, tokens, d_out, out_ld, int(out_bf16), act, cap, int(exact), stream):
+                       act: int = DENSE_PLAIN, cap: float = 0.0, exact: bool = False, bias: int | None = None, gated: int | None = None, gated_ld: int = 0,
+                       gated_pairs: int = 0) -> None:
+        """A bf16 matrix times a block of tokens: bf16 rows on the tensor cores, or (exact) fp32 rows in fp32 multiply-adds.  bias and
+        gated pairs as in dev_dense_gemv."""
+        epilogue = DenseEpilogue(act, cap, bias, gated, gated_ld, gated_pairs)
+        if not self.lib.zen_cuda_dev_dense_gemm(handle, d_x, x_ld, tokens, d_out, out_ld, int(out_bf16), C.byref(epilogue), int(exact), stream):
             self._fail("dev_dense_gemm")
 
     def dev_embed_rows_bf16(self, embed: int, positions: int | None, d_tokens: int, tokens: int, d_pos: int, d_out: int, stream: int = 0) -> None:
@@ -651,8 +666,10 @@ class Backend:
             self._fail("dev_rows_view")
 
     def dev_head_outputs_rows(self, d_o: int, rows: int, heads: int, width: int, head_ld: int, d_dst: int, ld: int, bf16: bool, stream: int = 0, *,
-                              weight: int | None = None, eps: float = 0.0, gate: int | None = None, gate_ld: int = 0, gate_mode: int = 0) -> None:
-        if not self.lib.zen_cuda_dev_head_outputs_rows(d_o, rows, heads, width, head_ld, weight, eps, gate, gate_ld, gate_mode, d_dst, ld, int(bf16), stream):
+                              weight: int | None = None, eps: float = 0.0, gate: int | None = None, gate_ld: int = 0, gate_mode: int = 0, fill: int | None = None) -> None:
+        """fill: columns written, zeros behind the heads (default: the whole row)."""
+        if not self.lib.zen_cuda_dev_head_outputs_rows(d_o, rows, heads, width, head_ld, weight, eps, gate, gate_ld, gate_mode, d_dst, ld, ld if fill is None else fill,
+                                                           int(bf16), stream):
             self._fail("dev_head_outputs_rows")
 
     def dev_window_attention_rows(self, a: WindowAttention, d_q: int, d_k: int, d_v: int, ld: int, tokens: int, d_pos: int, d_q_normed: int, d_out: int,
@@ -664,9 +681,9 @@ class Backend:
         if not self.lib.zen_cuda_dev_window_attention_step(C.byref(a), d_q, d_k, d_v, d_gate, d_pos, d_out, stream):
             self._fail("dev_window_attention_step")
 
-    def dev_state_step(self, layer: LinearLayer, delta: bool, d_proj: int, d_pos: int, d_out: int, stream: int = 0) -> None:
+    def dev_state_step(self, layer: LinearLayer, rule: int, d_proj: int, d_pos: int, d_out: int, stream: int = 0) -> None:
         """One token through a mixer with a matrix state: from its projections to its output projection's input."""
-        if not self.lib.zen_cuda_dev_state_step(C.byref(layer), int(delta), d_proj, d_pos, d_out, stream):
+        if not self.lib.zen_cuda_dev_state_step(C.byref(layer), int(rule), d_proj, d_pos, d_out, stream):
             self._fail("dev_state_step")
 
     def dev_delta_inputs_rows(self, layer: LinearLayer, d_proj: int, ld: int, d_decay: int, decay_ld: int, tokens: int, d_pos: int, d_q: int, d_k: int,
@@ -678,13 +695,19 @@ class Backend:
         if not self.lib.zen_cuda_dev_gated_write_inputs_rows(C.byref(layer), d_proj, ld, tokens, d_q, d_f, stream):
             self._fail("dev_gated_write_inputs_rows")
 
-    def state_scan_workspace_bytes(self, layer: LinearLayer, delta: bool, tokens: int) -> int:
-        return int(self.lib.zen_cuda_state_scan_workspace_bytes(C.byref(layer), int(delta), tokens))
+    def state_scan_workspace_bytes(self, layer: LinearLayer, rule: int, tokens: int) -> int:
+        return int(self.lib.zen_cuda_state_scan_workspace_bytes(C.byref(layer), int(rule), tokens))
 
-    def dev_state_scan(self, layer: LinearLayer, delta: bool, d_q: int, d_k: int | None, d_g: int, d_v: int, v_ld: int, d_beta: int | None, tokens: int,
+    def dev_state_scan(self, layer: LinearLayer, rule: int, d_q: int, d_k: int | None, d_g: int, d_v: int, v_ld: int, d_beta: int | None, tokens: int,
                        d_workspace: int, workspace_bytes: int, d_out: int, stream: int = 0) -> None:
-        if not self.lib.zen_cuda_dev_state_scan(C.byref(layer), int(delta), d_q, d_k, d_g, d_v, v_ld, d_beta, tokens, d_workspace, workspace_bytes, d_out, stream):
+        if not self.lib.zen_cuda_dev_state_scan(C.byref(layer), int(rule), d_q, d_k, d_g, d_v, v_ld, d_beta, tokens, d_workspace, workspace_bytes, d_out, stream):
             self._fail("dev_state_scan")
+
+    def dev_decayed_write_scan(self, layer: LinearLayer, d_proj: int, ld: int, tokens: int, d_pos: int, d_workspace: int, workspace_bytes: int, d_out: int,
+                               stream: int = 0) -> None:
+        """The decayed write over a block, straight from its projection rows."""
+        if not self.lib.zen_cuda_dev_decayed_write_scan(C.byref(layer), d_proj, ld, tokens, d_pos, d_workspace, workspace_bytes, d_out, stream):
+            self._fail("dev_decayed_write_scan")
 
     def dev_check(self, stream: int = 0) -> None:
         """Synchronises `stream` and raises if a kernel reported through the device-side error word (a bounded wait that

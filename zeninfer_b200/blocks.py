@@ -203,10 +203,10 @@ def dequantize(fmt: int, packed: np.ndarray, rows: int, columns: int) -> np.ndar
 
 def to_bf16(w: np.ndarray) -> np.ndarray:
     """fp32 -> bfloat16 bit patterns (uint16), round to nearest even; finite values only."""
-    u = np.ascontiguousarray(w, np.float32).view(np.uint32)
+    u = np.ascontiguousarray(w, np.float32).reshape(np.shape(w)).view(np.uint32)
     return ((u + np.uint32(0x7FFF) + ((u >> 16) & 1)) >> 16).astype(np.uint16)
 
 
 def from_bf16(bits: np.ndarray) -> np.ndarray:
     """bfloat16 bit patterns (uint16) -> fp32, exact."""
-    return (np.ascontiguousarray(bits, np.uint16).astype(np.uint32) << 16).view(np.float32)
+    return (np.ascontiguousarray(bits, np.uint16).reshape(np.shape(bits)).astype(np.uint32) << 16).view(np.float32)

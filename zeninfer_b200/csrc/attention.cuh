@@ -6,28 +6,45 @@
 
 #include <cstdint>
 
+#include "token_mixing.cuh"
 #include "zk_ptx.cuh"
 
 namespace zk {
+
+// What forms q, k and v where they are convolved and rotated: channels q | k | v in the convolution's numbering, the rotation of
+// q and k, and values mixed with those of an earlier layer: v <- (1 - share) v + share v_first.
+struct AttnRotary {
+    ShortConv conv;
+    HalfRotation turn;
+    const float* v_first;     // [tokens][kv_heads][v_dim]: the earlier layer's values of the same tokens; null: no mixing
+    float* v_keep;            // where this layer's values go for later layers, or null
+    float share;
+};
+
+// How attention_decode_kernel<kFused = true> finds q and k_new: to be rotated in adjacent pairs by the tables passed beside them, to be
+// RMS-normed per head, or to be convolved and rotated by halves.
+enum AttnInput : int { kAttnAdjacentPairs = 0, kAttnNormed = 1, kAttnConvRotary = 2 };
 
 // What a windowed attention with a distance bias adds to the plain one.  Query position i sees key position j <= i when
 // i - j < window or j < keep_first; the score is (q . k) * scale - slope_h * (i - j), slope_h = 2^(-8 (h + 1) / heads).
 struct AttnWindow {
     uint32_t keep_first;      // kept tokens at the start of the sequence (0: none)
     uint32_t biased;          // 1: the distance bias is taken off the scores
-    // attention_decode_kernel<..., kNormed = true> only: q and k arrive as raw projections and are RMS-normed per head here,
-    // value heads may be narrower than the cache's head pitch, and every head's output is scaled by a gate.
-    const float* q_weight;    // [qk_dim]
-    const float* k_weight;    // [qk_dim]
-    const float* gate;        // [heads]: the output is multiplied by sigmoid(gate[h]); null: no gate
+    // kAttnNormed and kAttnConvRotary: q, k and v arrive as raw projections and are finished here, value heads may be narrower
+    // than the cache's head pitch, and the output is scaled by a gate.
+    const float* q_weight;    // kAttnNormed: [qk_dim]
+    const float* k_weight;    // kAttnNormed: [qk_dim]
+    const float* gate;        // [heads], or [heads][v_dim] with gate_values: the output is multiplied by its sigmoid; null: no gate
     float eps;
     uint32_t qk_dim, v_dim;   // real sizes of a query/key and a value head; the cache's pitch D covers both, zero-padded
+    uint32_t gate_values;
+    AttnRotary rotary;        // kAttnConvRotary
 };
 
 __device__ __forceinline__ float attn_slope(uint32_t h, uint32_t heads) {
     return static_cast<float>(exp2(-8.0 * static_cast<double>(h + 1) / static_cast<double>(heads)));
 }
-__device__ __forceinline__ float logistic(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float mixed_value(float v, float first, float share) { return fmaf(share, first, (1.0f - share) * v); }
 
 // Grouped-query attention for one new token.  A cluster of kAttnSplit CTAs serves one query head: CTA `rank` takes
 // positions first + rank, first + rank + kAttnSplit, ...; inside a CTA a warp takes a position at a time, four dimensions
@@ -76,17 +93,18 @@ __device__ __forceinline__ void rope_quad(float4& v, uint32_t base, uint32_t pai
 // (include/zen/d3d12_backend.h:247).  Other clusters never read the cache at the current position, so the append
 // races with nothing.
 //
-// kNormed (with kFused): instead of the rotation, q and k_new are RMS-normed per head with AttnWindow's weights; the kept first
-// tokens and the distance bias of AttnWindow apply; out is [heads][v_dim], gated.  The cache's head pitch is D for keys and values
-// alike, zero beyond qk_dim / v_dim.
-template <bool kFused, bool kWide, bool kNormed = false>
+// kInput (with kFused): kAttnNormed norms q and k_new per head with AttnWindow's weights instead of the rotation; kAttnConvRotary
+// convolves all three, rotates q and k_new by halves and mixes v_new.  In both the kept first tokens and the distance bias of
+// AttnWindow apply; out is [heads][v_dim], gated.  The cache's head pitch is D for keys and values alike, zero beyond qk_dim / v_dim.
+template <bool kFused, bool kWide, int kInput = kAttnAdjacentPairs>
 __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThreads, kWide ? 2 : 3)
     attention_decode_kernel(const float* __restrict__ q, const float* __restrict__ k_cache_in, const float* __restrict__ v_cache_in,
                             const int* __restrict__ pos_ptr, float* __restrict__ out, uint32_t heads, uint32_t kv_heads, uint32_t D, float scale,
                             uint32_t window, uint32_t max_positions, int* error_word, const float* __restrict__ k_new, const float* __restrict__ v_new,
                             const float* __restrict__ cos_t, const float* __restrict__ sin_t, uint32_t pairs, float* k_cache_out, float* v_cache_out,
                             AttnWindow win) {
-    static_assert(kFused || !kNormed, "the normed form appends its own key");
+    constexpr bool kNormed = kInput == kAttnNormed, kOwn = kInput != kAttnAdjacentPairs;    // kOwn: finishes and appends its own key
+    static_assert(kFused || !kOwn, "the token in flight is formed here");
     const float* k_cache = kFused ? k_cache_out : k_cache_in;   // fused: the caches are also written here, so no read-only promise
     const float* v_cache = kFused ? v_cache_out : v_cache_in;
     namespace cg = cooperative_groups;
@@ -104,7 +122,7 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
     pdl_wait();
     // the first round trip: the position, and beside it everything whose address does not depend on it
     const int pos = *pos_ptr;
-    const uint32_t d_q = kNormed ? win.qk_dim : D, d_v = kNormed ? win.v_dim : D;
+    const uint32_t d_q = kOwn ? win.qk_dim : D, d_v = kOwn ? win.v_dim : D;
     const float* qh = q + static_cast<size_t>(h) * d_q;
     float4 q0 = make_float4(0.f, 0.f, 0.f, 0.f), q1 = q0;
     // real head sizes need not be a multiple of four floats, nor their start in the projection row aligned
@@ -117,13 +135,16 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
         return r;
     };
     float gate_value = 1.0f;
+    if (kOwn && win.gate) {
+        if (!win.gate_values) gate_value = logistic(__ldcg(win.gate + h));
+        else if (threadIdx.x < d_v) gate_value = logistic(__ldcg(win.gate + static_cast<size_t>(h) * d_v + threadIdx.x));
+    }
     if (kNormed) {
         q0 = ragged(qh, 4 * lane, d_q);
         if (kWide) q1 = ragged(qh, 128 + 4 * lane, d_q);
-        if (win.gate) gate_value = logistic(__ldcg(win.gate + h));
     }
-    if (!kNormed && lo_on) q0 = __ldcg(reinterpret_cast<const float4*>(qh + 4 * lane));      // q, k_new, v_new: written by the launch before this one
-    if (!kNormed && hi_on) q1 = __ldcg(reinterpret_cast<const float4*>(qh + 128 + 4 * lane));
+    if (!kOwn && lo_on) q0 = __ldcg(reinterpret_cast<const float4*>(qh + 4 * lane));      // q, k_new, v_new: written by the launch before this one
+    if (!kOwn && hi_on) q1 = __ldcg(reinterpret_cast<const float4*>(qh + 128 + 4 * lane));
     const float* knew = kFused ? k_new + static_cast<size_t>(kh) * d_q : nullptr;
     const float* vnew = kFused ? v_new + static_cast<size_t>(kh) * d_v : nullptr;
     float4 kn0 = make_float4(0.f, 0.f, 0.f, 0.f), kn1 = kn0, vn0 = kn0, vn1 = kn0;   // the token in flight, every warp's copy
@@ -147,15 +168,55 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
         normed(q0, q1, win.q_weight);
         normed(kn0, kn1, win.k_weight);
     }
-    if (kFused && !kNormed) {
+    if (kFused && !kOwn) {
         if (lo_on) { kn0 = __ldcg(reinterpret_cast<const float4*>(knew + 4 * lane)); vn0 = __ldcg(reinterpret_cast<const float4*>(vnew + 4 * lane)); }
         if (hi_on) { kn1 = __ldcg(reinterpret_cast<const float4*>(knew + 128 + 4 * lane)); vn1 = __ldcg(reinterpret_cast<const float4*>(vnew + 128 + 4 * lane)); }
     }
     const bool bad = pos < 0 || static_cast<uint32_t>(pos) >= max_positions;
+    if constexpr (kInput == kAttnConvRotary) {
+        __shared__ __align__(16) float head[3][kAttnMaxD];        // q, k, v of this head, convolved; zero beyond their sizes
+        const AttnRotary& ro = win.rotary;
+        const uint32_t i = threadIdx.x, cq = h * d_q + i, ck = (heads + kh) * d_q + i, cv = (heads + kv_heads) * d_q + kh * d_v + i;
+        const bool on = !bad, owner = rank == 0 && h % (heads / kv_heads) == 0;
+        const int at = bad ? 0 : pos;
+        float* slot = ro.conv.taps ? ro.conv.ring + static_cast<size_t>(static_cast<uint32_t>(at) % ro.conv.taps) * ro.conv.channels : nullptr;
+        float yq = 0.0f, yk = 0.0f, yv = 0.0f;
+        if (on && i < d_q) {
+            yq = conv_sum(ro.conv, qh + i, 0, 0, at, cq);
+            yk = conv_sum(ro.conv, knew + i, 0, 0, at, ck);
+            if (slot && rank == 0) slot[cq] = __ldcg(qh + i);
+            if (slot && owner) slot[ck] = __ldcg(knew + i);
+        }
+        if (on && i < d_v) {
+            yv = conv_sum(ro.conv, vnew + i, 0, 0, at, cv);
+            if (ro.v_first) yv = mixed_value(yv, __ldcg(ro.v_first + kh * d_v + i), ro.share);
+            if (ro.v_keep && owner) ro.v_keep[kh * d_v + i] = yv;
+            if (slot && owner) slot[cv] = __ldcg(vnew + i);
+        }
+        head[0][i] = yq;
+        head[1][i] = yk;
+        head[2][i] = yv;
+        __syncthreads();
+        const size_t row = rotation_row(ro.turn, at);
+        yq = rotated(ro.turn, [&](uint32_t d) { return head[0][d]; }, i, row);
+        yk = rotated(ro.turn, [&](uint32_t d) { return head[1][d]; }, i, row);
+        __syncthreads();
+        head[0][i] = yq;
+        head[1][i] = yk;
+        __syncthreads();
+        q0 = *reinterpret_cast<const float4*>(&head[0][4 * lane]);
+        kn0 = *reinterpret_cast<const float4*>(&head[1][4 * lane]);
+        vn0 = *reinterpret_cast<const float4*>(&head[2][4 * lane]);
+        if (kWide) {
+            q1 = *reinterpret_cast<const float4*>(&head[0][128 + 4 * lane]);
+            kn1 = *reinterpret_cast<const float4*>(&head[1][128 + 4 * lane]);
+            vn1 = *reinterpret_cast<const float4*>(&head[2][128 + 4 * lane]);
+        }
+    }
     if (bad && threadIdx.x == 0 && blockIdx.x == 0 && blockIdx.y == 0) atomicExch(error_word, kErrBadPosition);
     const uint32_t first = (window && static_cast<uint32_t>(pos) + 1 > window) ? static_cast<uint32_t>(pos) + 1 - window : 0u;
     uint32_t kept = 0;                                                                        // kept tokens the window has left behind
-    if (kNormed) kept = min(win.keep_first, first);
+    if (kOwn) kept = min(win.keep_first, first);
     const uint32_t count = bad ? 0u : static_cast<uint32_t>(pos) + 1 - first + kept;          // positions attended by the head
     const uint32_t mine = count > rank ? (count - rank + kAttnSplit - 1) / kAttnSplit : 0u;   // ... by this CTA
     const float* kbase = k_cache + static_cast<size_t>(first + rank) * kw + static_cast<size_t>(kh) * D;
@@ -164,12 +225,12 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
     const uint32_t last = count ? count - 1 : 0;                  // index of the current position among the attended ones
     const uint32_t skipped = first - kept;                        // positions between the kept tokens and the window
     auto position_of = [&](uint32_t index) { return index < kept ? index : index + skipped; };
-    const float slope = kNormed && win.biased ? attn_slope(h, heads) : 0.0f;
+    const float slope = kOwn && win.biased ? attn_slope(h, heads) : 0.0f;
 
     float run_max = -INFINITY;
     double run_sum = 0.0;
     float4 a0 = make_float4(0.f, 0.f, 0.f, 0.f), a1 = a0;
-    bool rotated = false;
+    bool turned = false;
     for (uint32_t i0 = warp; i0 < mine; i0 += kWarps * kAttnUnroll) {
         // the second round trip: keys and values of this round's positions together (and, the first time, the cos/sin row)
         float4 ka[kAttnUnroll], kb[kAttnUnroll], va[kAttnUnroll], vb[kAttnUnroll];
@@ -182,7 +243,7 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
             if (i < mine && !fresh[u]) {
                 const float* kt = kbase + static_cast<size_t>(i) * step;
                 const float* vt = vbase + static_cast<size_t>(i) * step;
-                if (kNormed) {
+                if (kOwn) {
                     const size_t row = static_cast<size_t>(position_of(rank + i * kAttnSplit)) * kw + static_cast<size_t>(kh) * D;
                     kt = k_cache + row;
                     vt = v_cache + row;
@@ -191,12 +252,12 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
                 if (hi_on) { kb[u] = __ldcg(reinterpret_cast<const float4*>(kt + 128 + 4 * lane)); vb[u] = __ldcg(reinterpret_cast<const float4*>(vt + 128 + 4 * lane)); }
             }
         }
-        if (kFused && !kNormed && !rotated && !bad) {   // rotate q and the new key once (table rows of the current position)
+        if (kFused && !kOwn && !turned && !bad) {   // rotate q and the new key once (table rows of the current position)
             const float* cs = cos_t + static_cast<size_t>(pos) * pairs;
             const float* sn = sin_t + static_cast<size_t>(pos) * pairs;
             if (lo_on) { rope_quad(q0, 4u * lane, pairs, cs, sn); rope_quad(kn0, 4u * lane, pairs, cs, sn); }
             if (hi_on) { rope_quad(q1, 128u + 4u * lane, pairs, cs, sn); rope_quad(kn1, 128u + 4u * lane, pairs, cs, sn); }
-            rotated = true;
+            turned = true;
         }
         float sc[kAttnUnroll];
 #pragma unroll
@@ -206,7 +267,7 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
             sc[u] = i0 + u * kWarps < mine ? acc * scale : -INFINITY;
-            if (kNormed && i0 + u * kWarps < mine) sc[u] -= slope * static_cast<float>(static_cast<uint32_t>(pos) - position_of(rank + (i0 + u * kWarps) * kAttnSplit));
+            if (kOwn && i0 + u * kWarps < mine) sc[u] -= slope * static_cast<float>(static_cast<uint32_t>(pos) - position_of(rank + (i0 + u * kWarps) * kAttnSplit));
         }
         float new_max = run_max;
 #pragma unroll
@@ -227,13 +288,13 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
         run_max = new_max;
     }
     // append: the cluster of the KV group's first query head, the CTA that owns the current position
-    if (kNormed && !bad && h % (heads / kv_heads) == 0 && rank == last % kAttnSplit && warp == 0) {
+    if (kOwn && !bad && h % (heads / kv_heads) == 0 && rank == last % kAttnSplit && warp == 0) {
         float* kr = k_cache_out + static_cast<size_t>(pos) * kw + static_cast<size_t>(kh) * D;
         float* vr = v_cache_out + static_cast<size_t>(pos) * kw + static_cast<size_t>(kh) * D;
         if (lo_on) { *reinterpret_cast<float4*>(kr + 4 * lane) = kn0; *reinterpret_cast<float4*>(vr + 4 * lane) = vn0; }
         if (hi_on) { *reinterpret_cast<float4*>(kr + 128 + 4 * lane) = kn1; *reinterpret_cast<float4*>(vr + 128 + 4 * lane) = vn1; }
     }
-    if (kFused && !kNormed && !bad && h % (heads / kv_heads) == 0 && rank == last % kAttnSplit && threadIdx.x < D) {
+    if (kFused && !kOwn && !bad && h % (heads / kv_heads) == 0 && rank == last % kAttnSplit && threadIdx.x < D) {
         const float* cs = cos_t + static_cast<size_t>(pos) * pairs;
         const float* sn = sin_t + static_cast<size_t>(pos) * pairs;
         const uint32_t dd = threadIdx.x, pr = dd >> 1;
@@ -283,7 +344,7 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
             const float inv = 1.0f / static_cast<float>(denom);
             float total = 0.0f;
             for (uint32_t r = 0; r < kAttnSplit; ++r) total += w[r] * cluster.map_shared_rank(&share, r)->out[threadIdx.x];
-            out[static_cast<size_t>(h) * d_v + threadIdx.x] = kNormed ? total * inv * gate_value : total * inv;
+            out[static_cast<size_t>(h) * d_v + threadIdx.x] = kOwn ? total * inv * gate_value : total * inv;
         }
     }
     cluster.sync();                                   // nobody leaves while rank 0 still reads its shared memory

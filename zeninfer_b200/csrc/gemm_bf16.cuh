@@ -4,7 +4,8 @@
 // a TMEM lane is a weight row and consecutive lanes store consecutive outputs of one token.  One persistent CTA per SM, six warps:
 // TMA producer (64 columns of K per stage: 128 x 128 B of weights and kNTile x 128 B of activations, 128-byte swizzle), MMA issuer,
 // four epilogue warps; two accumulators in TMEM, so the epilogue of a tile runs under the next tile's products.  K and rows that
-// do not fill a tile arrive as zeros from the tensor maps.
+// do not fill a tile arrive as zeros from the tensor maps.  The first 2 pairs rows may be (gate, up) pairs that leave as
+// silu(gate) * up: neighbouring TMEM lanes, exchanged between lanes of the epilogue warp.
 //
 // gemm_bf16_exact_kernel: fp32 activations times bf16 weights in fp32 FMAs, for the 32-bit mode.
 #pragma once
@@ -22,9 +23,11 @@ constexpr uint32_t kBgABytes = kBgM * kBgK * 2;
 struct GemmBf16Params {
     CUtensorMap map_w;        // [rows][ld] bf16, box 64 x 128
     CUtensorMap map_x;        // [tokens][ld] bf16, box 64 x kNTile
-    float* out;               // [tokens][out_ld] fp32, or null
+    float* out;               // [tokens][out_ld] fp32, or null; row r of the matrix is column r - 2 pairs
     __nv_bfloat16* out_bf16;  // [tokens][out_ld] bf16 when out is null
-    uint32_t out_ld, rows, tokens, k_tiles, m_tiles, n_tiles;
+    __nv_bfloat16* gated;     // [tokens][gated_ld]: column i from rows 2 i and 2 i + 1
+    const float* bias;        // [rows - 2 pairs], or null
+    uint32_t out_ld, gated_ld, pairs, rows, tokens, k_tiles, m_tiles, n_tiles;
     int act;
     float cap;
     int* error_word;
@@ -134,7 +137,8 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const __grid_c
         uint32_t count = 0;
         pdl_wait();                                                // the outputs may still be read by an earlier launch
         for (uint32_t tile = blockIdx.x; tile < tiles; tile += gridDim.x, ++count) {
-            const uint32_t set = count & 1, n0 = (tile % p.n_tiles) * kNTile, r = (tile / p.n_tiles) * kBgM + quad * 32 + lane;
+            const uint32_t set = count & 1, n0 = (tile % p.n_tiles) * kNTile, r = (tile / p.n_tiles) * kBgM + quad * 32 + lane, paired = 2 * p.pairs;
+            const float bias = p.bias && r >= paired && r < p.rows ? __ldg(p.bias + r - paired) : 0.0f;
             if (*abort_word || !mbar_wait(&tmem_full[set], (count >> 1) & 1)) {
                 if (lane == 0 && !*abort_word) { *abort_word = 1; atomicExch(p.error_word, kErrTmemWaitTimeout); }
                 break;
@@ -152,13 +156,23 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const __grid_c
                     __syncwarp();
                     if (lane == 0) mbar_arrive(&tmem_empty[set]);
                 }
-                if (r < p.rows) {
+                if (r - lane < paired) {                           // some of the warp's rows are pairs: an even lane takes one token, its partner the next
+                    const bool odd = lane & 1;
+#pragma unroll
+                    for (int c = 0; c < kChunk; c += 2) {
+                        const float keep = __uint_as_float(odd ? v[c + 1] : v[c]);
+                        const float other = __shfl_xor_sync(0xffffffffu, __uint_as_float(odd ? v[c] : v[c + 1]), 1);
+                        const uint32_t t = n0 + c0 + c + (odd ? 1u : 0u);
+                        if (r < paired && t < p.tokens) p.gated[static_cast<size_t>(t) * p.gated_ld + r / 2] = __float2bfloat16_rn(odd ? silu_f(other) * keep : silu_f(keep) * other);
+                    }
+                }
+                if (r >= paired && r < p.rows) {
 #pragma unroll
                     for (int c = 0; c < kChunk; ++c) {
                         const uint32_t t = n0 + c0 + c;
                         if (t < p.tokens) {
-                            const float y = dense_activation(__uint_as_float(v[c]), p.act, p.cap);
-                            const size_t at = static_cast<size_t>(t) * p.out_ld + r;
+                            const float y = dense_activation(__uint_as_float(v[c]) + bias, p.act, p.cap);
+                            const size_t at = static_cast<size_t>(t) * p.out_ld + (r - paired);
                             if (p.out) p.out[at] = y; else p.out_bf16[at] = __float2bfloat16_rn(y);
                         }
                     }
@@ -174,11 +188,12 @@ __global__ void __launch_bounds__(kBgThreads, 1) gemm_bf16_kernel(const __grid_c
     }
 }
 
-// out[t][r] = act(sum_k x[t][k] w[r][k]), 64 x 64 outputs per CTA, four by four per thread.
+// out[t][r - 2 pairs] = act(sum_k x[t][k] w[r][k] + bias[r - 2 pairs]) and gated[t][i] = silu(row 2 i) * (row 2 i + 1), 64 x 64 sums per
+// CTA, four by four per thread.
 constexpr int kExactTile = 64, kExactK = 16;
 __global__ void __launch_bounds__(256) gemm_bf16_exact_kernel(const __nv_bfloat16* __restrict__ w, uint32_t w_ld, const float* __restrict__ x, uint32_t x_ld,
                                                               float* __restrict__ out, uint32_t out_ld, uint32_t rows, uint32_t tokens, uint32_t K, int act,
-                                                              float cap) {
+                                                              float cap, const float* __restrict__ bias, float* __restrict__ gated, uint32_t gated_ld, uint32_t pairs) {
     __shared__ float ws[kExactK][kExactTile + 4], xs[kExactK][kExactTile + 4];
     pdl_launch_dependents();
     pdl_wait();
@@ -210,7 +225,11 @@ __global__ void __launch_bounds__(256) gemm_bf16_exact_kernel(const __nv_bfloat1
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const uint32_t r = r0 + tx * 4 + i;
-            if (r < rows) out[static_cast<size_t>(t) * out_ld + r] = dense_activation(acc[i][j], act, cap);
+            if (r < 2 * pairs) {
+                if (!(i & 1)) gated[static_cast<size_t>(t) * gated_ld + r / 2] = silu_f(acc[i][j]) * acc[i + 1 < 4 ? i + 1 : i][j];
+            } else if (r < rows) {
+                out[static_cast<size_t>(t) * out_ld + (r - 2 * pairs)] = dense_activation(acc[i][j] + (bias ? __ldg(bias + r - 2 * pairs) : 0.0f), act, cap);
+            }
         }
     }
 }

@@ -6,7 +6,8 @@
 //   * weights are constants: the first two steps' loads go out before the previous grid has finished (griddepcontrol);
 //   * the prologue can finish the sublayer before it (row_ops.cuh: grouped norm, residual add, token shift or output norm), so
 //     a decode step needs no launches for them: every CTA forms the input vector itself, CTA 0 stores the residual stream;
-//   * the epilogue applies the product's activation (squared ReLU, or the logits' soft cap) in fp32.
+//   * the epilogue adds a bias and applies the product's activation (squared ReLU, or the logits' soft cap) in fp32; a matrix may
+//     begin with pairs of rows (gate, up) that leave the launch as silu(gate) * up.
 // Activations are fp32 throughout: the product is exact up to fp32 accumulation.
 #pragma once
 #include "row_ops.cuh"
@@ -23,9 +24,12 @@ enum : int { kActNone = 0, kActSquaredRelu = 1, kActSoftcap = 2 };
 struct DenseTask {
     const __nv_bfloat16* w;   // [rows][ld], zero beyond the real columns
     const float* x;           // [K]; ignored when the launch carries a prologue
-    float* y;                 // [rows]
+    float* y;                 // [rows - 2 pairs]
+    const float* bias;        // [rows - 2 pairs], or null
+    float* gated;             // [pairs]
     uint32_t rows, K, ld;
     uint32_t first_row;       // index of its first row in the launch's row space
+    uint32_t pairs;           // rows 2 i and 2 i + 1 (i < pairs) give gated[i]; first_row is even then
     int act;
     float cap;
 };
@@ -34,6 +38,7 @@ struct DenseGemvParams {
     DenseTask task[kDenseMaxTasks];
     uint32_t tasks, total_rows;
     uint32_t k_split;         // warps that share a row group: a power of two, at most kDenseWarps
+    uint32_t row_unit;        // a CTA's slice begins at a multiple of this many rows: 2 where a task has pairs
     uint32_t has_prologue;    // 1: one task, whose input is the prologue's view
     uint32_t scratch_floats;
     SublayerEnd pre;
@@ -58,8 +63,9 @@ __device__ __forceinline__ void dense_fma8(const uint4& w, const float (&x)[8], 
 __global__ void __launch_bounds__(kDenseThreads, 1) gemv_bf16_kernel(const __grid_constant__ DenseGemvParams p) {
     extern __shared__ __align__(16) float dense_smem[];
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t slice0 = static_cast<uint32_t>(static_cast<uint64_t>(p.total_rows) * blockIdx.x / gridDim.x);
-    const uint32_t slice1 = static_cast<uint32_t>(static_cast<uint64_t>(p.total_rows) * (blockIdx.x + 1) / gridDim.x);
+    const uint64_t row_units = (p.total_rows + p.row_unit - 1) / p.row_unit;
+    const uint32_t slice0 = static_cast<uint32_t>(row_units * blockIdx.x / gridDim.x) * p.row_unit;
+    const uint32_t slice1 = min(static_cast<uint32_t>(row_units * (blockIdx.x + 1) / gridDim.x) * p.row_unit, p.total_rows);
     const uint32_t team = warp / p.k_split, part = warp % p.k_split, teams = kDenseWarps / p.k_split;
     pdl_launch_dependents();
 
@@ -187,9 +193,17 @@ __global__ void __launch_bounds__(kDenseThreads, 1) gemv_bf16_kernel(const __gri
         while (row >= p.task[ti].first_row + p.task[ti].rows) ++ti;
         const DenseTask& t = p.task[ti];
         const uint32_t parts = min(p.k_split, dense_units(t.ld));
-        float v = 0.0f;
-        for (uint32_t s = 0; s < parts; ++s) v += sums[static_cast<size_t>(i) * p.k_split + s];
-        t.y[row - t.first_row] = dense_activation(v, t.act, t.cap);
+        auto total = [&](uint32_t at) {
+            float v = 0.0f;
+            for (uint32_t s = 0; s < parts; ++s) v += sums[static_cast<size_t>(at) * p.k_split + s];
+            return v;
+        };
+        const uint32_t r = row - t.first_row, paired = 2 * t.pairs;
+        if (r < paired) {
+            if (!(r & 1)) t.gated[r / 2] = silu_f(total(i)) * total(i + 1);
+        } else {
+            t.y[r - paired] = dense_activation(total(i) + (t.bias ? __ldg(t.bias + r - paired) : 0.0f), t.act, t.cap);
+        }
     }
 }
 

@@ -2,94 +2,46 @@
 //
 //   delta rule    S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q      (g per key channel)
 //   gated write   S <- f * S + (1 - f) v^T;           o = S^T q                       (f per key channel, no key)
+//   decayed write S <- g * S + k v^T;                 o = S^T q                       (g per key channel of the token, or one constant
+//                                                                                      per head; q and k may be rotated by position)
 //
 // state_scan_kernel walks a block of tokens, eight at a time, with the state in registers; state_step_kernel takes one token and
 // does everything between the layer's input projections and its output projection.  The kernels around the scan form its inputs (short causal
 // convolution, unit norms, decays, gates) for all tokens at once.
 //
 // Device layout of a state: [heads][vdim][pitch], pitch = dim rounded up to 32 and zero beyond dim, so that eight lanes read a
-// column's rows as consecutive 16-byte words.  The convolution keeps the inputs of the last `taps` tokens in a ring
-// [taps][channels] whose slot is the position modulo taps: a token reads the taps - 1 slots before its own and nobody else
-// writes those, so it needs no second buffer.
+// column's rows as consecutive 16-byte words.
 #pragma once
 #include "gemv_bf16.cuh"
+#include "token_mixing.cuh"
 
 namespace zk {
 
-__device__ __forceinline__ float silu_f(float z) { return z * logistic(z); }
-__device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z + log1pf(expf(-z)) : log1pf(expf(z)); }
 constexpr float kUnitEps = 1e-6f;
+enum StateRule : int { kGatedWrite = 0, kDeltaRule = 1, kDecayedWrite = 2 };
 
 struct LinearLayer {
     uint32_t heads, kv_heads, dim, vdim, pitch;
-    uint32_t taps;                 // delta rule: convolution taps
-    uint32_t rank_a, rank_g;       // delta rule: ranks of the decay's and the output gate's projections
+    uint32_t rank_a, rank_g;       // ranks of the decay's (delta rule, decayed write) and the output gate's (delta rule) projections
     uint32_t a2_ld, g2_ld;
-    const float* conv;             // [taps][channels]: q, k, v channels
-    const float* a_log;            // [heads]
-    const float* dt_bias;          // [heads][dim]
+    ShortConv conv;                // delta rule: q, k, v channels
+    const float* a_log;            // delta rule: [heads]
+    const float* dt_bias;          // [heads][dim], added to the decay's projection
     const __nv_bfloat16* a2;       // [heads dim][a2_ld]
     const __nv_bfloat16* g2;       // [heads vdim][g2_ld]
+    const float* decay;            // decayed write: [heads] constants, or null: g = sigmoid(a2 a1 + dt_bias)^inv_tau
+    float inv_tau;
+    HalfRotation turn;             // decayed write: of q and k
     const float* f_bias;           // gated write: [heads][dim]
     const float* lower;            // gated write: [heads][dim]
     const float* norm;             // [vdim]
-    float* ring;                   // [taps][channels]
     float* state;                  // [heads][vdim][pitch]
     float eps;
 };
 __host__ __device__ inline uint32_t linear_channels(const LinearLayer& l) { return 2 * l.kv_heads * l.dim + l.heads * l.vdim; }
-
-// Convolution of channel c at block row t (position pos + t), then silu.  x: projection rows of pitch ld, channel c at column c;
-// rows before the block come from the ring, tokens before the sequence's start are zeros.
-__device__ __forceinline__ float conv_silu(const LinearLayer& l, const float* __restrict__ x, uint32_t ld, int t, int pos, uint32_t c, uint32_t channels) {
-    float y = 0.0f;
-    const int taps = static_cast<int>(l.taps);
-#pragma unroll 4
-    for (int j = 0; j < taps; ++j) {
-        const int s = t - (taps - 1 - j), at = pos + s;
-        const float* src = s >= 0 ? x + static_cast<size_t>(s) * ld + c : l.ring + static_cast<size_t>(static_cast<uint32_t>(max(at, 0)) % l.taps) * channels + c;
-        const float v = at >= 0 ? __ldcg(src) : 0.0f;
-        y = fmaf(__ldg(l.conv + static_cast<size_t>(j) * channels + c), v, y);
-    }
-    return silu_f(y);
-}
+__device__ __forceinline__ float channel_decay(float z, float inv_tau) { return expf(-softplus_f(-z) * inv_tau); }     // sigmoid(z)^inv_tau
 
 // ---- inputs of the scan for a block of tokens -------------------------------------------------------------------------
-
-constexpr int kStrip = 8;          // tokens a warp takes at a time: a channel's inputs stay in registers while the taps slide over them
-constexpr int kMaxSlidingTaps = 4; // more taps than this are read again for every token
-
-// y[i] = silu(convolution) of channel c at tokens t0 .. t0 + n - 1 (n <= kStrip; the rest is not used).
-__device__ __forceinline__ void conv_silu_strip(const LinearLayer& l, const float* __restrict__ x, uint32_t ld, int t0, int n, int pos, uint32_t c,
-                                                uint32_t channels, float (&y)[kStrip]) {
-    const int taps = static_cast<int>(l.taps);
-    if (taps > kMaxSlidingTaps) {
-#pragma unroll
-        for (int i = 0; i < kStrip; ++i)
-            if (i < n) y[i] = conv_silu(l, x, ld, t0 + i, pos, c, channels);
-        return;
-    }
-    float w[kMaxSlidingTaps], in[kMaxSlidingTaps - 1 + kStrip];       // w right-aligned: the last is the current token's; in[kMaxSlidingTaps - 1 + i]: token t0 + i
-#pragma unroll
-    for (int j = 0; j < kMaxSlidingTaps; ++j) {
-        const int tap = j - (kMaxSlidingTaps - taps);
-        w[j] = tap >= 0 ? __ldg(l.conv + static_cast<size_t>(tap) * channels + c) : 0.0f;
-    }
-#pragma unroll
-    for (int i = 0; i < kMaxSlidingTaps - 1 + kStrip; ++i) {
-        const int s = t0 + i - (kMaxSlidingTaps - 1), at = pos + s;   // block row, position
-        in[i] = 0.0f;
-        if (at >= 0 && s >= t0 - (taps - 1) && s < t0 + n)
-            in[i] = s >= 0 ? __ldcg(x + static_cast<size_t>(s) * ld + c) : l.ring[static_cast<size_t>(static_cast<uint32_t>(at) % l.taps) * channels + c];
-    }
-#pragma unroll
-    for (int i = 0; i < kStrip; ++i) {
-        float sum = 0.0f;
-#pragma unroll
-        for (int j = 0; j < kMaxSlidingTaps; ++j) sum = fmaf(w[j], in[i + j], sum);
-        y[i] = silu_f(sum);
-    }
-}
 
 // Delta rule.  proj [T][ld]: q | k | v | b columns; decay [T][heads dim] = W_a2 W_a1 h.
 //   q, k [T][kv_heads][pitch] unit vectors (q also times dim^-1/2), g [T][heads][pitch], v [T][heads vdim], beta [T][heads].
@@ -102,6 +54,11 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
     pdl_wait();
     const int t0 = static_cast<int>(blockIdx.x) * kStrip, n = min(kStrip, static_cast<int>(tokens) - t0), pos = *pos_ptr;
     const uint32_t lane = threadIdx.x & 31, channels = linear_channels(l), kd = l.kv_heads * l.dim, nv = l.heads * l.vdim;
+    auto silu_strip = [&](uint32_t c, float (&y)[kStrip]) {
+        conv_sum_strip(l.conv, proj + c, ld, t0, n, pos, c, y);
+#pragma unroll
+        for (int i = 0; i < kStrip; ++i) y[i] = silu_f(y[i]);
+    };
     const uint32_t qk_items = 2 * l.kv_heads, v_items = (nv + 31) / 32, items = qk_items + v_items + l.heads;
     for (uint32_t item = blockIdx.y * 8 + (threadIdx.x >> 5); item < items; item += gridDim.y * 8) {
         float y[kStrip];
@@ -117,7 +74,7 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
                 const bool more = d + 32 < l.pitch;
 #pragma unroll
                 for (int i = 0; i < kStrip; ++i) y[i] = 0.0f;
-                if (d < l.dim) conv_silu_strip(l, proj, ld, t0, n, pos, c0 + d, channels, y);
+                if (d < l.dim) silu_strip(c0 + d, y);
 #pragma unroll
                 for (int i = 0; i < kStrip; ++i) {
                     ss[i] += y[i] * y[i];
@@ -141,7 +98,7 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
         } else if (item < qk_items + v_items) {
             const uint32_t c = (item - qk_items) * 32 + lane;
             if (c >= nv) continue;
-            conv_silu_strip(l, proj, ld, t0, n, pos, 2 * kd + c, channels, y);
+            silu_strip(2 * kd + c, y);
 #pragma unroll
             for (int i = 0; i < kStrip; ++i)
                 if (i < n) v[static_cast<size_t>(t0 + i) * nv + c] = y[i];
@@ -159,17 +116,6 @@ __global__ void __launch_bounds__(256) delta_inputs_rows_kernel(const __grid_con
             if (static_cast<int>(lane) < n) beta[static_cast<size_t>(t0 + lane) * l.heads + h] = logistic(__ldcg(proj + static_cast<size_t>(t0 + lane) * ld + channels + h));
         }
     }
-}
-
-// The ring after a block of T tokens: the inputs of its last min(T, taps) tokens.  Runs after the kernel above.
-__global__ void __launch_bounds__(256) conv_ring_update_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj, uint32_t ld, uint32_t tokens,
-                                                               const int* __restrict__ pos_ptr) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const uint32_t channels = linear_channels(l), c = blockIdx.x * 256 + threadIdx.x, pos = static_cast<uint32_t>(*pos_ptr);
-    if (c >= channels) return;
-    for (uint32_t t = tokens > l.taps ? tokens - l.taps : 0; t < tokens; ++t)
-        l.ring[static_cast<size_t>((pos + t) % l.taps) * channels + c] = proj[static_cast<size_t>(t) * ld + c];
 }
 
 // Gated write.  proj [T][ld]: q | f columns.  q, f [T][heads][pitch]; f = 1 beyond dim (the padding neither decays nor writes).
@@ -202,17 +148,20 @@ __global__ void __launch_bounds__(256) gated_write_inputs_rows_kernel(const __gr
 // u = T (v - (k G) . S) with T = (1 + diag(beta) A)^-1 diag(beta).  Only products of decays appear, never a quotient, so nothing
 // overflows however strong they are.  state_groups_kernel forms, for every group and head at once, the scaled vectors and the
 // small matrices T and M (o_t = (q_t G_t) . S + sum_s M_ts w_s with w = v - (k G) . S, M = B T); state_scan_kernel walks the groups.
-// The gated write has u = v and k = 1 - f: no T, and M = B.
+// The gated write has u = v and k = 1 - f, the decayed write u = v: no T, and M = B.  For the decayed write q and k are columns of the
+// projection rows (pitch v_ld, heads of `dim`), and this kernel rotates them and forms the decays.
 //
 // A group's record, fp32: [k G: 8 x pitch, delta rule only] [q G: 8 x pitch] [k g...: 8 x pitch] [G_8: pitch] [T: 8 x 8, delta only]
 // [M: 8 x 8].  Missing tokens at the end of a block have g = 1, k = q = beta = 0 and leave the state as it is.
 
 struct ScanParams {
-    const float* q;        // [T][q_heads][pitch]
-    const float* k;        // [T][q_heads][pitch]; delta rule only
-    const float* g;        // [T][heads][pitch]
+    const float* q;        // [T][q_heads][pitch]; decayed write: [T][v_ld]
+    const float* k;        // [T][q_heads][pitch], delta rule; [T][v_ld], decayed write
+    const float* g;        // [T][heads][pitch]; not for the decayed write
     const float* v;        // [T][v_ld], head h's values at column h * vdim
     const float* beta;     // [T][heads]; delta rule only
+    const float* low;      // decayed write without constant decays: [T][v_ld], the decay's low-rank inputs
+    const int* pos;        // decayed write with a rotation
     float* records;        // [groups][heads][record]
     float* state;          // [heads][vdim][pitch]
     float* out;            // [T][heads][vdim]
@@ -238,10 +187,12 @@ __device__ __forceinline__ void warp_sum64(float (&v)[64], int lane) {
 }
 
 // One warp per (group, head); a lane takes channels lane, lane + 32, ...  Grid: ceil(groups * heads / 4).
-template <int kQuads, bool kDelta>
-__global__ void __launch_bounds__(128) state_groups_kernel(const __grid_constant__ ScanParams p) {
+template <int kQuads, int kRule>
+__global__ void __launch_bounds__(128) state_groups_kernel(const __grid_constant__ ScanParams p, const __grid_constant__ LinearLayer l) {
+    constexpr bool kDelta = kRule == kDeltaRule;
     constexpr uint32_t kPitch = kQuads * 32, kRecord = scan_record_floats(kPitch, kDelta);
     __shared__ float sums[4][64], t_matrix[4][64];
+    extern __shared__ __align__(16) float group_low[];          // decayed write: [warp][token][rank rounded up to 8]
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -252,6 +203,18 @@ __global__ void __launch_bounds__(128) state_groups_kernel(const __grid_constant
     float* const q_out = rec + (kDelta ? 8 * kPitch : 0);
     float* const k_out = q_out + 8 * kPitch;
     float* const g_out = k_out + 8 * kPitch;
+    const uint32_t low_ld = (l.rank_a + 7) & ~7u;
+    float* const low = group_low + warp * kGroup * low_ld;
+    const bool ranked = kRule == kDecayedWrite && !l.decay;
+    const float fixed = kRule == kDecayedWrite && l.decay ? __ldg(l.decay + h) : 0.0f, q_scale = 1.0f / sqrtf(static_cast<float>(l.dim));
+    const int pos = kRule == kDecayedWrite && l.turn.half ? *p.pos : 0;
+    if (ranked) {
+        for (uint32_t i = lane; i < kGroup * low_ld; i += 32) {
+            const uint32_t t = i / low_ld, c = i % low_ld;
+            low[i] = t0 + t < p.tokens && c < l.rank_a ? __ldcg(p.low + static_cast<size_t>(t0 + t) * p.v_ld + c) : 0.0f;
+        }
+        __syncwarp();
+    }
     // entry of (t, s): A's at t (t - 1) / 2 + s for s < t, B's at 28 + t (t + 1) / 2 + s for s <= t
     float acc[64];
 #pragma unroll
@@ -260,12 +223,40 @@ __global__ void __launch_bounds__(128) state_groups_kernel(const __grid_constant
     for (int j = 0; j < kQuads; ++j) {
         const uint32_t d = lane + 32 * j;
         float g[kGroup], k[kGroup], q[kGroup];
+        if constexpr (kRule == kDecayedWrite) {
+            const bool real = d < l.dim;
+            if (ranked) {
+                const float bias = real ? __ldg(l.dt_bias + h * l.dim + d) : 0.0f;
 #pragma unroll
-        for (int t = 0; t < kGroup; ++t) {
-            const bool on = t0 + t < p.tokens;
-            g[t] = on ? __ldcg(p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch + d) : 1.0f;
-            q[t] = on ? __ldcg(p.q + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch + d) : 0.0f;
-            k[t] = !kDelta ? 1.0f - g[t] : on ? __ldcg(p.k + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch + d) : 0.0f;
+                for (int t = 0; t < kGroup; ++t) g[t] = bias;
+                const __nv_bfloat16* w = l.a2 + static_cast<size_t>(h * l.dim + d) * l.a2_ld;
+                for (uint32_t c = 0; c < low_ld; c += 8) {      // a2_ld is the rank rounded up to 8 as well
+                    const uint4 w8 = real ? __ldg(reinterpret_cast<const uint4*>(w + c)) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+                    for (int t = 0; t < kGroup; ++t) {
+                        const float4 x0 = *reinterpret_cast<const float4*>(low + t * low_ld + c), x1 = *reinterpret_cast<const float4*>(low + t * low_ld + c + 4);
+                        const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+                        dense_fma8(w8, x, g[t]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < kGroup; ++t) {
+                const bool on = t0 + t < p.tokens;
+                const size_t at = static_cast<size_t>(t0 + t) * p.v_ld + h * l.dim, row = l.turn.half ? rotation_row(l.turn, pos + static_cast<int>(t0 + t)) : 0;
+                auto turned = [&](const float* x) { return on && real ? rotated(l.turn, [&](uint32_t i) { return __ldcg(x + at + i); }, d, row) : 0.0f; };
+                g[t] = !on ? 1.0f : ranked ? channel_decay(g[t], l.inv_tau) : fixed;
+                q[t] = q_scale * turned(p.q);
+                k[t] = turned(p.k);
+            }
+        } else {
+#pragma unroll
+            for (int t = 0; t < kGroup; ++t) {
+                const bool on = t0 + t < p.tokens;
+                g[t] = on ? __ldcg(p.g + (static_cast<size_t>(t0 + t) * p.heads + h) * kPitch + d) : 1.0f;
+                q[t] = on ? __ldcg(p.q + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch + d) : 0.0f;
+                k[t] = !kDelta ? 1.0f - g[t] : on ? __ldcg(p.k + (static_cast<size_t>(t0 + t) * p.q_heads + qh) * kPitch + d) : 0.0f;
+            }
         }
         float run = 1.0f;
 #pragma unroll
@@ -474,15 +465,16 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const __grid_c
 // ---- one token -------------------------------------------------------------------------------------------------------
 
 // One CTA per head: everything from the projections of one token to the output projection's input.  proj: delta rule
-// q | k | v | b | a1 | g1, gated write q | f | v.  out [heads][vdim].
+// q | k | v | b | a1 | g1, gated write q | f | v, decayed write q | k | v | g | a1 (a1 without constant decays).  out [heads][vdim].
 // kMaxQuads: most 16-byte words a lane holds of a column (pitch / 32): up to four, a CTA of 1024 threads takes 128 columns at a time.
 __host__ __device__ constexpr int step_threads(int max_quads) { return max_quads <= 4 ? 1024 : 512; }
 __host__ __device__ inline uint32_t step_low_floats(const LinearLayer& l) { return ((l.rank_a + 63) & ~63u) + ((l.rank_g + 63) & ~63u); }
-template <bool kDelta, int kMaxQuads>
+template <int kRule, int kMaxQuads>
 __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(const __grid_constant__ LinearLayer l, const float* __restrict__ proj,
                                                                   const int* __restrict__ pos_ptr, float* __restrict__ out) {
+    constexpr bool kDelta = kRule == kDeltaRule;
     constexpr uint32_t kStepThreads = step_threads(kMaxQuads), kWarps = kStepThreads / 32;
-    extern __shared__ __align__(16) float low[];                   // delta rule: a1 and g1 outputs, each padded with zeros to 64
+    extern __shared__ __align__(16) float low[];                   // a1 and (delta rule) g1 outputs, each padded with zeros to 64
     __shared__ __align__(16) float q[256], k[256], g[256];
     __shared__ float v[256], o[256], gate[256], bias[256], norm[256];
     const uint32_t h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & 7, quads = l.pitch / 32;
@@ -491,19 +483,22 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
     // lane are fetched while the previous launch is still running
     constexpr uint32_t kAhead = kMaxQuads <= 4 ? 4 : 8;
     uint4 ahead[kAhead];
-    const uint32_t words = kDelta ? (max(l.a2_ld, l.g2_ld) + 63) / 64 : 0;      // 16-byte words per lane and row
+    const bool ranked = kDelta || (kRule == kDecayedWrite && !l.decay);
+    const uint32_t words = ranked ? (max(l.a2_ld, l.g2_ld) + 63) / 64 : 0;      // 16-byte words per lane and row
+    uint32_t rank_rows = ranked ? l.pitch : 0;
+    if (kDelta) rank_rows += l.vdim;
     auto rank_row = [&](uint32_t r, uint32_t& ld) -> const __nv_bfloat16* {     // null: padding
         const bool is_g = r >= l.pitch;
         const uint32_t d = is_g ? r - l.pitch : r;
         ld = is_g ? l.g2_ld : l.a2_ld;
-        if (d >= (is_g ? l.vdim : l.dim)) return nullptr;
+        if (r >= rank_rows || d >= (is_g ? l.vdim : l.dim)) return nullptr;
         return is_g ? l.g2 + static_cast<size_t>(h * l.vdim + d) * ld : l.a2 + static_cast<size_t>(h * l.dim + d) * ld;
     };
-    if (kDelta) {
+    if (ranked) {
         uint32_t r = warp * 4 + (lane >> 3), word = 0;
 #pragma unroll
         for (uint32_t i = 0; i < kAhead; ++i) {
-            uint32_t ld;
+            uint32_t ld = 0;
             const __nv_bfloat16* w = rank_row(r, ld);
             const uint32_t c = (word * 8 + part) * 8;
             ahead[i] = w && c < ld ? __ldg(reinterpret_cast<const uint4*>(w + c)) : make_uint4(0, 0, 0, 0);
@@ -512,9 +507,9 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
     }
     // so are the small constants that would otherwise cost a round trip each in the middle of the step
     for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) norm[i] = __ldg(l.norm + i);
-    if (kDelta)
+    if (ranked)
         for (uint32_t i = threadIdx.x; i < l.dim; i += kStepThreads) bias[i] = __ldg(l.dt_bias + h * l.dim + i);
-    const float a_scale = kDelta ? -expf(__ldg(l.a_log + h)) : 0.0f;
+    const float a_scale = kDelta ? -expf(__ldg(l.a_log + h)) : 0.0f, fixed = kRule == kDecayedWrite && l.decay ? __ldg(l.decay + h) : 0.0f;
     pdl_wait();
     // the first columns' state words are on their way while the token's vectors are formed
     float* const state = l.state + static_cast<size_t>(h) * l.vdim * l.pitch + part * 4;
@@ -524,31 +519,16 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
     for (uint32_t i = 0; i < kMaxQuads; ++i)
         pre[i] = (i < quads && col < l.vdim) ? __ldcg(reinterpret_cast<const float4*>(state + static_cast<size_t>(col) * l.pitch + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
     float beta = 0.0f;
-    if (kDelta) {
-        const int pos = *pos_ptr;
-        const uint32_t channels = linear_channels(l), kd = l.kv_heads * l.dim, qh = h / (l.heads / l.kv_heads);
-        const uint32_t pad_a = (l.rank_a + 63) & ~63u;
+    // the decays, and the delta rule's output gate, from the low-rank inputs
+    const uint32_t pad_a = (l.rank_a + 63) & ~63u;
+    auto stage_low = [&](const float* a1, const float* g1) {
         for (uint32_t i = threadIdx.x; i < step_low_floats(l); i += kStepThreads) {
             const bool is_g = i >= pad_a;
             const uint32_t c = is_g ? i - pad_a : i;
-            low[i] = c < (is_g ? l.rank_g : l.rank_a) ? __ldcg(proj + channels + l.heads + (is_g ? l.rank_a : 0u) + c) : 0.0f;
+            low[i] = c < (is_g ? l.rank_g : l.rank_a) ? __ldcg((is_g ? g1 : a1) + c) : 0.0f;
         }
-        beta = logistic(__ldcg(proj + channels + h));
-        const bool owner = h % (l.heads / l.kv_heads) == 0;        // one CTA per q/k head keeps its ring
-        float* slot = l.ring + static_cast<size_t>(static_cast<uint32_t>(pos) % l.taps) * channels;
-        for (uint32_t i = threadIdx.x; i < 2 * l.pitch + l.vdim; i += kStepThreads) {
-            const bool is_v = i >= 2 * l.pitch, is_k = !is_v && i >= l.pitch;
-            const uint32_t d = is_v ? i - 2 * l.pitch : is_k ? i - l.pitch : i;
-            float y = 0.0f;
-            if (is_v || d < l.dim) {
-                const uint32_t c = is_v ? 2 * kd + h * l.vdim + d : (is_k ? kd : 0u) + qh * l.dim + d;
-                y = conv_silu(l, proj, 0, 0, pos, c, channels);
-                if (is_v || owner) slot[c] = __ldcg(proj + c);
-            }
-            (is_v ? v : is_k ? k : q)[d] = y;
-        }
-        __syncthreads();
-        // decays and output gate
+    };
+    auto low_rank = [&] {
         uint32_t r = warp * 4 + (lane >> 3), word = 0;
         float acc = 0.0f;
         auto take = [&](const uint4& w) {
@@ -564,9 +544,10 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
             if (word != words) return;
 #pragma unroll
             for (int s = 1; s < 8; s <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, s);
-            if (part == 0 && r < l.pitch + l.vdim) {
+            if (part == 0 && r < rank_rows) {
                 if (is_g) gate[r - l.pitch] = logistic(acc);
-                else g[r] = r < l.dim ? expf(a_scale * softplus_f(acc + bias[r])) : 0.0f;
+                else if (kDelta) g[r] = r < l.dim ? expf(a_scale * softplus_f(acc + bias[r])) : 0.0f;
+                else g[r] = r < l.dim ? channel_decay(acc + bias[r], l.inv_tau) : 0.0f;
             }
             acc = 0.0f;
             word = 0;
@@ -575,13 +556,34 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
         // r - lane / 8 and word are the same in all lanes of a warp, so the loops below do not diverge around the shuffles
 #pragma unroll
         for (uint32_t i = 0; i < kAhead; ++i)
-            if (r - (lane >> 3) < l.pitch + l.vdim) take(ahead[i]);
-        while (r - (lane >> 3) < l.pitch + l.vdim) {
-            uint32_t ld;
+            if (r - (lane >> 3) < rank_rows) take(ahead[i]);
+        while (r - (lane >> 3) < rank_rows) {
+            uint32_t ld = 0;
             const __nv_bfloat16* w = rank_row(r, ld);
             const uint32_t c = (word * 8 + part) * 8;
             take(w && c < ld ? __ldg(reinterpret_cast<const uint4*>(w + c)) : make_uint4(0, 0, 0, 0));
         }
+    };
+    if (kDelta) {
+        const int pos = *pos_ptr;
+        const uint32_t channels = linear_channels(l), kd = l.kv_heads * l.dim, qh = h / (l.heads / l.kv_heads);
+        stage_low(proj + channels + l.heads, proj + channels + l.heads + l.rank_a);
+        beta = logistic(__ldcg(proj + channels + h));
+        const bool owner = h % (l.heads / l.kv_heads) == 0;        // one CTA per q/k head keeps its ring
+        float* slot = l.conv.ring + static_cast<size_t>(static_cast<uint32_t>(pos) % l.conv.taps) * channels;
+        for (uint32_t i = threadIdx.x; i < 2 * l.pitch + l.vdim; i += kStepThreads) {
+            const bool is_v = i >= 2 * l.pitch, is_k = !is_v && i >= l.pitch;
+            const uint32_t d = is_v ? i - 2 * l.pitch : is_k ? i - l.pitch : i;
+            float y = 0.0f;
+            if (is_v || d < l.dim) {
+                const uint32_t c = is_v ? 2 * kd + h * l.vdim + d : (is_k ? kd : 0u) + qh * l.dim + d;
+                y = silu_f(conv_sum(l.conv, proj + c, 0, 0, pos, c));
+                if (is_v || owner) slot[c] = __ldcg(proj + c);
+            }
+            (is_v ? v : is_k ? k : q)[d] = y;
+        }
+        __syncthreads();
+        low_rank();
         __syncthreads();
         if (warp < 2) {                                            // unit norms: warp 0 takes q, warp 1 k
             float* x = warp ? k : q;
@@ -590,6 +592,30 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
             float inv = 1.0f / sqrtf(warp_sum(ss) + kUnitEps);
             if (!warp) inv *= 1.0f / sqrtf(static_cast<float>(l.dim));
             for (uint32_t d = lane; d < l.pitch; d += 32) x[d] *= inv;
+        }
+    } else if (kRule == kDecayedWrite) {
+        const uint32_t kd = l.heads * l.dim, nv = l.heads * l.vdim;
+        const size_t row = l.turn.half ? rotation_row(l.turn, *pos_ptr) : 0;
+        const float q_scale = 1.0f / sqrtf(static_cast<float>(l.dim));
+        if (ranked) stage_low(proj + 2 * kd + 2 * nv, nullptr);
+        for (uint32_t i = threadIdx.x; i < 2 * (l.pitch + l.vdim); i += kStepThreads) {
+            if (i < 2 * l.pitch) {
+                const bool is_k = i >= l.pitch;
+                const uint32_t d = is_k ? i - l.pitch : i;
+                const float* x = proj + (is_k ? kd : 0u) + h * l.dim;
+                const float y = d < l.dim ? rotated(l.turn, [&](uint32_t j) { return __ldcg(x + j); }, d, row) : 0.0f;
+                if (is_k) k[d] = y; else q[d] = y * q_scale;
+                if (!ranked && !is_k) g[d] = fixed;
+            } else {
+                const bool is_g = i >= 2 * l.pitch + l.vdim;
+                const uint32_t d = i - 2 * l.pitch - (is_g ? l.vdim : 0u);
+                const float y = __ldcg(proj + 2 * kd + (is_g ? nv : 0u) + h * l.vdim + d);
+                if (is_g) gate[d] = silu_f(y); else v[d] = y;
+            }
+        }
+        if (ranked) {
+            __syncthreads();
+            low_rank();
         }
     } else {
         for (uint32_t d = threadIdx.x; d < l.pitch; d += kStepThreads) {
@@ -643,7 +669,7 @@ __global__ void __launch_bounds__(step_threads(kMaxQuads)) state_step_kernel(con
     float ss = 0.0f;
     for (uint32_t i = lane; i < l.vdim; i += 32) ss += o[i] * o[i];          // every warp forms the head's norm itself
     const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(l.vdim) + l.eps);
-    for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) out[h * l.vdim + i] = o[i] * inv * norm[i] * (kDelta ? gate[i] : 1.0f);
+    for (uint32_t i = threadIdx.x; i < l.vdim; i += kStepThreads) out[h * l.vdim + i] = o[i] * inv * norm[i] * (kRule == kGatedWrite ? 1.0f : gate[i]);
 }
 
 }  // namespace zk

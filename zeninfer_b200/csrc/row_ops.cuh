@@ -1,6 +1,6 @@
 // Row-wise operators of the bfloat16 decoders, all in fp32: embedding rows with learned positions, the end of a sublayer
 // (grouped RMS norm of its output, residual add, token shift or output norm for whatever reads the stream next), per-head norms
-// with a gate, query/key norms with the KV append, and the logit soft cap.
+// with a gate, and query/key norms or convolution and rotation with the KV append.
 //
 // The end of a sublayer is a device function, because it runs in two places: as a kernel over the rows of a block
 // (sublayer_end_rows_kernel) and in the prologue of the decode product that consumes its result (gemv_bf16.cuh).
@@ -19,7 +19,8 @@ namespace zk {
 // x_new = x_in + norm(y), or x_in alone without y_a; per row of n values.
 //   y         = y_a, or with y_b half the sum of both after each is divided by its root mean square and multiplied by
 //               weight_a / weight_b
-//   norm      = groups equal consecutive parts, each divided by its own root mean square, times norm_weight
+//   norm      = groups equal consecutive parts, each divided by its own root mean square, times norm_weight; without norm_weight
+//               the residual add is plain: x_new = x_in + y
 // The row's consumer gets h = x_new + (before - x_new) * shift (before: the previous token's x_new), or the grouped norm of x_new
 // with out_norm, or x_new itself.  keep receives the block's last row of x_in: the sublayer's own input, which the sequence's next
 // token reads as `before`.
@@ -86,6 +87,11 @@ __device__ __forceinline__ void sublayer_row(const SublayerEnd& p, size_t r, flo
         return;
     }
     const float* a = p.y_a + r * p.n;
+    if (!p.norm_weight) {
+        for (uint32_t i = threadIdx.x; i < p.n; i += kThreads) row[i] = __ldcg(x + i) + __ldcg(a + i);
+        __syncthreads();
+        return;
+    }
     if (p.y_b) {
         constexpr uint32_t kWarps = kThreads / 32;
         const float* b = p.y_b + r * p.n;
@@ -195,12 +201,13 @@ __global__ void __launch_bounds__(256) rows_view_kernel(const float* __restrict_
 }
 
 // Per head of `width` values (input pitch head_ld): o, divided by its root mean square and times weight when weight is given,
-// times sigmoid(gate).  gate_mode 0: none; 1: one value per head, gate [rows][gate_ld]; 2: one per value, [rows][gate_ld], laid
-// out heads x width.  dst [rows][ld] packs the heads without padding, zeros behind them.  A warp takes a head; grid: rows.
+// times a gate.  gate_mode 0: none; 1: sigmoid, one value per head, gate [rows][gate_ld]; 2 and 3: sigmoid or silu, one per value,
+// [rows][gate_ld], laid out heads x width.  dst [rows][ld] packs the heads without padding, zeros behind them up to column `fill`.
+// A warp takes a head; grid: rows.
 template <typename TView>
 __global__ void __launch_bounds__(256) head_outputs_rows_kernel(const float* __restrict__ o, uint32_t heads, uint32_t width, uint32_t head_ld,
                                                                 const float* __restrict__ weight, float eps, const float* __restrict__ gate, uint32_t gate_ld,
-                                                                int gate_mode, TView* __restrict__ dst, uint32_t ld) {
+                                                                int gate_mode, TView* __restrict__ dst, uint32_t ld, uint32_t fill) {
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -217,11 +224,14 @@ __global__ void __launch_bounds__(256) head_outputs_rows_kernel(const float* __r
         for (uint32_t i = lane; i < width; i += 32) {
             float y = v[i] * inv * head_gate;
             if (weight) y *= weight[i];
-            if (gate_mode == 2) y *= logistic(gate[r * gate_ld + h * width + i]);
+            if (gate_mode >= 2) {
+                const float z = gate[r * gate_ld + h * width + i];
+                y *= gate_mode == 2 ? logistic(z) : silu_f(z);
+            }
             store_as(dst + r * ld + h * width + i, y);
         }
     }
-    for (uint32_t i = heads * width + threadIdx.x; i < ld; i += 256) store_as(dst + r * ld + i, 0.0f);
+    for (uint32_t i = heads * width + threadIdx.x; i < fill; i += 256) store_as(dst + r * ld + i, 0.0f);
 }
 
 // Query and key norms of a block of rows and the append of its keys and values at positions *pos ..: q, k, v are columns of the
@@ -253,6 +263,78 @@ __global__ void __launch_bounds__(256) qk_norm_append_rows_kernel(const float* _
         }
         const float* w = is_q ? win.q_weight : win.k_weight;
         for (uint32_t i = lane; i < pitch; i += 32) dst[i] = i < n ? ((is_q || is_k) ? src[i] * inv * w[i] : src[i]) : 0.0f;
+    }
+}
+
+// The ring after a block of T tokens: the inputs of its last min(T, taps) tokens.  Runs after every reader of the ring; x: the
+// channels' columns of the projection rows.
+__global__ void __launch_bounds__(256) conv_ring_update_kernel(const __grid_constant__ ShortConv conv, const float* __restrict__ x, uint32_t ld, uint32_t tokens,
+                                                               const int* __restrict__ pos_ptr) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t c = blockIdx.x * 256 + threadIdx.x, pos = static_cast<uint32_t>(*pos_ptr);
+    if (c >= conv.channels) return;
+    for (uint32_t t = tokens > conv.taps ? tokens - conv.taps : 0; t < tokens; ++t)
+        conv.ring[static_cast<size_t>((pos + t) % conv.taps) * conv.channels + c] = x[static_cast<size_t>(t) * ld + c];
+}
+
+// The rotary form of the norm-and-append kernel: per channel of q, k and v the short convolution, then the rotation of q and k, the mixing of v
+// with the values of an earlier layer (or their keeping for later layers), and the append.  A warp takes (strip of kStrip tokens,
+// head); grid: (strips, CTAs that share one).  The ring is brought up to date afterwards (conv_ring_update_kernel).
+__global__ void __launch_bounds__(256) conv_rotary_append_rows_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, uint32_t ld,
+                                                                      const __grid_constant__ AttnWindow win, uint32_t heads, uint32_t kv_heads, uint32_t pitch,
+                                                                      uint32_t tokens, const int* __restrict__ pos_ptr, float* __restrict__ q_out,
+                                                                      float* __restrict__ k_cache, float* __restrict__ v_cache, uint32_t max_positions,
+                                                                      int* error_word) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const AttnRotary& ro = win.rotary;
+    const int t0 = static_cast<int>(blockIdx.x) * kStrip, n = min(kStrip, static_cast<int>(tokens) - t0), pos = *pos_ptr;
+    if (pos < 0 || static_cast<long long>(pos) + tokens > static_cast<long long>(max_positions)) {
+        if (threadIdx.x == 0) atomicExch(error_word, kErrBadPosition);
+        return;
+    }
+    const uint32_t lane = threadIdx.x & 31, half = ro.turn.half, items = heads + 2 * kv_heads;
+    for (uint32_t item = blockIdx.y * 8 + (threadIdx.x >> 5); item < items; item += gridDim.y * 8) {
+        const bool is_q = item < heads, is_k = !is_q && item < heads + kv_heads, is_v = !is_q && !is_k;
+        const uint32_t g = is_q ? item : is_k ? item - heads : item - heads - kv_heads, size = is_v ? win.v_dim : win.qk_dim;
+        const uint32_t first = is_q ? 0u : is_k ? heads * win.qk_dim : (heads + kv_heads) * win.qk_dim;      // the convolution's channel of the part's first column
+        const float* src = (is_q ? q : is_k ? k : v) + g * size;
+        const uint32_t c0 = first + g * size, step = (is_q ? heads : kv_heads) * pitch;
+        float* dst = is_q ? q_out + (static_cast<size_t>(t0) * heads + g) * pitch : (is_k ? k_cache : v_cache) + (static_cast<size_t>(pos + t0) * kv_heads + g) * pitch;
+        float a[kStrip], b[kStrip];
+        const uint32_t turned = is_v ? 0u : 2 * half;
+        for (uint32_t i = lane; i < turned / 2; i += 32) {
+            conv_sum_strip(ro.conv, src + i, ld, t0, n, pos, c0 + i, a);
+            conv_sum_strip(ro.conv, src + half + i, ld, t0, n, pos, c0 + half + i, b);
+#pragma unroll
+            for (int j = 0; j < kStrip; ++j) {
+                if (j >= n) break;
+                const size_t row = rotation_row(ro.turn, pos + t0 + j) + i;
+                const float c = __ldg(ro.turn.cos_t + row), s = __ldg(ro.turn.sin_t + row);
+                dst[static_cast<size_t>(j) * step + i] = rotated_low(a[j], b[j], c, s);
+                dst[static_cast<size_t>(j) * step + half + i] = rotated_high(a[j], b[j], c, s);
+            }
+        }
+        for (uint32_t i = turned + lane; i < pitch; i += 32) {
+#pragma unroll
+            for (int j = 0; j < kStrip; ++j) a[j] = 0.0f;
+            if (i < size) {
+                conv_sum_strip(ro.conv, src + i, ld, t0, n, pos, c0 + i, a);
+                if (is_v && (ro.v_first || ro.v_keep)) {
+#pragma unroll
+                    for (int j = 0; j < kStrip; ++j) {
+                        if (j >= n) break;
+                        const size_t at = static_cast<size_t>(t0 + j) * kv_heads * size + g * size + i;
+                        if (ro.v_first) a[j] = mixed_value(a[j], __ldcg(ro.v_first + at), ro.share);
+                        if (ro.v_keep) ro.v_keep[at] = a[j];
+                    }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < kStrip; ++j)
+                if (j < n) dst[static_cast<size_t>(j) * step + i] = a[j];
+        }
     }
 }
 

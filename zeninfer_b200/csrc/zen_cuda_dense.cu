@@ -49,7 +49,7 @@ uint32_t pitch32(uint32_t n) { return (n + 31u) & ~31u; }
 
 bool sublayer_ok(const zen_cuda_sublayer_end* s) {
     if (!s || !s->x_in || !s->n || !s->groups || s->n % s->groups || s->groups > 4096) return false;
-    if (s->x_out == s->x_in || (s->y_a && !s->norm_weight) || (s->y_b && (!s->y_a || !s->weight_a || !s->weight_b))) return false;
+    if (s->x_out == s->x_in || (s->y_b && (!s->y_a || !s->norm_weight || !s->weight_a || !s->weight_b))) return false;
     return !(s->shift && (!s->before || s->out_norm || s->before == s->keep));
 }
 zk::SublayerEnd device_form(const zen_cuda_sublayer_end& s) {
@@ -76,29 +76,79 @@ cudaError_t launch_gemm(const Entry& e, zk::GemmBf16Params& p) {
 
 bool window_ok(const zen_cuda_window_attention* a) {
     return a && a->heads && a->kv_heads && a->heads % a->kv_heads == 0 && a->qk_dim && a->v_dim && a->pitch == pitch32(std::max(a->qk_dim, a->v_dim)) &&
-           a->pitch <= 256 && a->window && a->max_positions && a->q_weight && a->k_weight && a->k_cache && a->v_cache;
+           a->pitch <= 256 && a->window && a->max_positions && a->k_cache && a->v_cache && !a->q_weight == !a->k_weight &&
+           (a->q_weight ? !a->taps && !a->rot_pairs && !a->v_first && !a->v_keep
+                        : 2 * a->rot_pairs <= a->qk_dim && (!a->rot_pairs || (a->rot_cos && a->rot_sin)) && (!a->taps || (a->conv && a->ring)));
 }
+bool is_rotary(const zen_cuda_window_attention& a) { return !a.q_weight; }
 zk::AttnWindow device_form(const zen_cuda_window_attention& a, const float* gate) {
-    return zk::AttnWindow{a.keep_first, a.bias ? 1u : 0u, a.q_weight, a.k_weight, gate, a.eps, a.qk_dim, a.v_dim};
+    zk::AttnWindow w{a.keep_first, a.bias ? 1u : 0u, a.q_weight, a.k_weight, gate, a.eps, a.qk_dim, a.v_dim, a.gate_values ? 1u : 0u, {}};
+    w.rotary.conv = zk::ShortConv{a.conv, a.ring, a.taps, (a.heads + a.kv_heads) * a.qk_dim + a.kv_heads * a.v_dim};
+    w.rotary.turn = zk::HalfRotation{a.rot_cos, a.rot_sin, a.rot_pairs, a.max_positions};
+    w.rotary.v_first = a.v_first;
+    w.rotary.v_keep = a.v_keep;
+    w.rotary.share = a.v_share;
+    return w;
 }
 
-bool linear_ok(const zen_cuda_linear_layer* l, int delta) {
-    if (!l || !l->heads || !l->dim || !l->vdim || l->dim > 256 || l->vdim > 256 || !l->state || !l->norm) return false;
-    if (!delta) return l->kv_heads == l->heads && l->f_bias && l->lower;
+bool linear_ok(const zen_cuda_linear_layer* l, int rule) {
+    if (!l || rule < ZEN_CUDA_STATE_GATED_WRITE || rule > ZEN_CUDA_STATE_DECAYED_WRITE || !l->heads || !l->dim || !l->vdim || l->dim > 256 || l->vdim > 256 || !l->state || !l->norm) return false;
+    if (rule == ZEN_CUDA_STATE_GATED_WRITE) return l->kv_heads == l->heads && l->f_bias && l->lower;
+    if (rule == ZEN_CUDA_STATE_DECAYED_WRITE)
+        return l->kv_heads == l->heads && 2 * l->rot_pairs <= l->dim && (!l->rot_pairs || (l->rot_cos && l->rot_sin && l->max_positions)) &&
+               (l->decay || (l->dt_bias && l->inv_tau > 0.0f && is_bf16(l->a2) && l->a2->rows == size_t(l->heads) * l->dim && l->a2->cols <= 512));
     return l->kv_heads && l->heads % l->kv_heads == 0 && l->taps && l->conv && l->a_log && l->dt_bias && l->ring && is_bf16(l->a2) && is_bf16(l->g2) &&
            l->a2->rows == size_t(l->heads) * l->dim && l->g2->rows == size_t(l->heads) * l->vdim;
 }
-zk::LinearLayer device_form(const zen_cuda_linear_layer& l, int delta) {
+zk::LinearLayer device_form(const zen_cuda_linear_layer& l, int rule) {
     zk::LinearLayer d{};
     d.heads = l.heads; d.kv_heads = l.kv_heads; d.dim = l.dim; d.vdim = l.vdim; d.pitch = pitch32(l.dim);
-    d.taps = delta ? l.taps : 0; d.eps = l.eps; d.norm = l.norm; d.state = l.state;
-    if (delta) {
+    d.eps = l.eps; d.norm = l.norm; d.state = l.state;
+    if (rule == ZEN_CUDA_STATE_DELTA_RULE) {
+        d.conv = zk::ShortConv{l.conv, l.ring, l.taps, zk::linear_channels(d)};
         d.rank_a = u32(l.a2->cols); d.rank_g = u32(l.g2->cols); d.a2_ld = l.a2->nbp; d.g2_ld = l.g2->nbp;
-        d.conv = l.conv; d.a_log = l.a_log; d.dt_bias = l.dt_bias; d.a2 = plane(l.a2); d.g2 = plane(l.g2); d.ring = l.ring;
+        d.a_log = l.a_log; d.dt_bias = l.dt_bias; d.a2 = plane(l.a2); d.g2 = plane(l.g2);
+    } else if (rule == ZEN_CUDA_STATE_DECAYED_WRITE) {
+        d.turn = zk::HalfRotation{l.rot_cos, l.rot_sin, l.rot_pairs, l.max_positions};
+        d.decay = l.decay;
+        if (!l.decay) { d.rank_a = u32(l.a2->cols); d.a2_ld = l.a2->nbp; d.dt_bias = l.dt_bias; d.a2 = plane(l.a2); d.inv_tau = l.inv_tau; }
     } else {
         d.f_bias = l.f_bias; d.lower = l.lower;
     }
     return d;
+}
+
+// The groups' records, then the walk over them.
+cudaError_t run_scan(Entry& e, int rule, uint32_t dim, const zk::ScanParams& p, const zk::LinearLayer& l) {
+    const dim3 grid((p.vdim + zk::kScanColumns - 1) / zk::kScanColumns, p.heads);
+    // A grid that fits the SMs one CTA each asks for more than half an SM's shared memory: launched while the groups kernel drains,
+    // its CTAs would otherwise pile up on the first SMs to come free, and each runs for the whole block of tokens.
+    const bool spread = static_cast<uint64_t>(grid.x) * grid.y <= static_cast<uint64_t>(e.sm_count);
+    auto alone = [&](size_t smem) { return spread ? std::max(smem, e.smem_optin / 2 + 1024) : smem; };
+    auto go = [&](auto quads, auto which) {
+        constexpr int kQ = decltype(quads)::value, kRule = decltype(which)::value;
+        constexpr bool kDelta = kRule == zk::kDeltaRule;
+        const dim3 prepare(u32(((p.tokens + zk::kGroup - 1) / zk::kGroup * p.heads + 3) / 4));
+        const size_t low = rule == ZEN_CUDA_STATE_DECAYED_WRITE ? size_t(4) * zk::kGroup * ((l.rank_a + 7) & ~7u) * sizeof(float) : 0;
+        const cudaError_t first = launch(e, zk::state_groups_kernel<kQ, kRule>, prepare, dim3(128), low, p, l);
+        if (!e.leave(first, "state_scan: groups")) return first;
+        return launch(e, zk::state_scan_kernel<kQ, kDelta>, grid, dim3(zk::kScanThreads), alone(zk::scan_smem_bytes<kQ, kDelta>()), p);
+    };
+    auto by_rule = [&](auto quads) {
+        return rule == ZEN_CUDA_STATE_DELTA_RULE      ? go(quads, std::integral_constant<int, zk::kDeltaRule>{})
+               : rule == ZEN_CUDA_STATE_DECAYED_WRITE ? go(quads, std::integral_constant<int, zk::kDecayedWrite>{})
+                                                      : go(quads, std::integral_constant<int, zk::kGatedWrite>{});
+    };
+    switch (pitch32(dim) / 32) {
+    case 1: return by_rule(std::integral_constant<int, 1>{});
+    case 2: return by_rule(std::integral_constant<int, 2>{});
+    case 3: return by_rule(std::integral_constant<int, 3>{});
+    case 4: return by_rule(std::integral_constant<int, 4>{});
+    case 5: return by_rule(std::integral_constant<int, 5>{});
+    case 6: return by_rule(std::integral_constant<int, 6>{});
+    case 7: return by_rule(std::integral_constant<int, 7>{});
+    default: return by_rule(std::integral_constant<int, 8>{});
+    }
 }
 
 }  // namespace
@@ -129,11 +179,14 @@ int zen_cuda_dev_dense_gemv(const zen_cuda_dense_task* tasks, size_t count, cons
     uint64_t rows = 0;
     size_t x_floats = 0;
     uint32_t units = 1;
+    p.row_unit = 1;
     for (size_t i = 0; i < count; ++i) {
         const zen_cuda_dense_task& t = tasks[i];
-        if (!is_bf16(t.w) || !t.d_y || (!pre && !t.d_x) || (pre && t.w->cols != pre->n) || (t.act == ZEN_CUDA_DENSE_SOFTCAP && !(t.cap > 0.0f)))
+        if (!is_bf16(t.w) || (!pre && !t.d_x) || (pre && t.w->cols != pre->n) || (t.act == ZEN_CUDA_DENSE_SOFTCAP && !(t.cap > 0.0f)) ||
+            t.gated_pairs > t.w->rows / 2 || (t.gated_pairs && (!t.d_gated || rows % 2)) || (t.w->rows > 2 * t.gated_pairs && !t.d_y))
             return e.fail("dense_gemv: bad task");
-        p.task[i] = zk::DenseTask{plane(t.w), t.d_x, t.d_y, u32(t.w->rows), u32(t.w->cols), t.w->nbp, u32(rows), t.act, t.cap};
+        p.task[i] = zk::DenseTask{plane(t.w), t.d_x, t.d_y, t.d_bias, t.d_gated, u32(t.w->rows), u32(t.w->cols), t.w->nbp, u32(rows), u32(t.gated_pairs), t.act, t.cap};
+        if (t.gated_pairs) p.row_unit = 2;
         rows += t.w->rows;
         units = std::max(units, zk::dense_units(t.w->nbp));
         x_floats += static_cast<size_t>(zk::dense_units(t.w->nbp)) * zk::kDenseUnit;
@@ -148,22 +201,26 @@ int zen_cuda_dev_dense_gemv(const zen_cuda_dense_task* tasks, size_t count, cons
         p.pre = device_form(*pre);
         p.scratch_floats = (zk::row_scratch_floats(zk::kDenseThreads, pre->groups) + 3u) & ~3u;
     }
-    const uint32_t grid = std::min<uint32_t>(u32(e.sm_count), u32(rows));
-    const size_t slice = (rows + grid - 1) / grid;
+    const uint32_t row_units = u32((rows + p.row_unit - 1) / p.row_unit), grid = std::min<uint32_t>(u32(e.sm_count), row_units);
+    const size_t slice = static_cast<size_t>((row_units + grid - 1) / grid) * p.row_unit;
     const size_t smem = (x_floats + p.scratch_floats + slice * p.k_split) * sizeof(float);
     if (smem > e.smem_optin) return e.fail("dense_gemv: the input vector and a slice's sums do not fit shared memory");
     return e.leave(launch(e, zk::gemv_bf16_kernel, dim3(grid), dim3(zk::kDenseThreads), smem, p), "dense_gemv");
 }
 
-int zen_cuda_dev_dense_gemm(const zen_cuda_weights* w, const void* d_x, size_t x_ld, size_t tokens, void* d_out, size_t out_ld, int out_bf16, int act, float cap,
-                            int exact, void* stream) {
-    ZC_ENTER(stream, is_bf16(w) && d_x && d_out && tokens && tokens <= 0x7fffffffu && x_ld >= w->cols && out_ld >= w->rows && !(exact && out_bf16) &&
-                         !(act == ZEN_CUDA_DENSE_SOFTCAP && !(cap > 0.0f)), "dense_gemm");
+int zen_cuda_dev_dense_gemm(const zen_cuda_weights* w, const void* d_x, size_t x_ld, size_t tokens, void* d_out, size_t out_ld, int out_bf16,
+                            const zen_cuda_dense_epilogue* epilogue, int exact, void* stream) {
+    const zen_cuda_dense_epilogue ep = epilogue ? *epilogue : zen_cuda_dense_epilogue{};
+    ZC_ENTER(stream, is_bf16(w) && d_x && tokens && tokens <= 0x7fffffffu && x_ld >= w->cols && ep.gated_pairs <= w->rows / 2 &&
+                         (w->rows == 2 * ep.gated_pairs || (d_out && out_ld >= w->rows - 2 * ep.gated_pairs)) &&
+                         (!ep.gated_pairs || (ep.d_gated && ep.gated_ld >= ep.gated_pairs)) && !(exact && out_bf16) &&
+                         !(ep.act == ZEN_CUDA_DENSE_SOFTCAP && !(ep.cap > 0.0f)), "dense_gemm");
     if (exact) {
         const size_t ty = (tokens + zk::kExactTile - 1) / zk::kExactTile;
         if (ty > 65535) return e.fail("dense_gemm: too many tokens");
         return e.leave(launch(e, zk::gemm_bf16_exact_kernel, dim3(u32((w->rows + zk::kExactTile - 1) / zk::kExactTile), u32(ty)), dim3(256), 0, plane(w), w->nbp,
-                              static_cast<const float*>(d_x), u32(x_ld), static_cast<float*>(d_out), u32(out_ld), u32(w->rows), u32(tokens), u32(w->cols), act, cap),
+                              static_cast<const float*>(d_x), u32(x_ld), static_cast<float*>(d_out), u32(out_ld), u32(w->rows), u32(tokens), u32(w->cols), ep.act, ep.cap, ep.d_bias,
+                              static_cast<float*>(ep.d_gated), u32(ep.gated_ld), u32(ep.gated_pairs)),
                        "dense_gemm");
     }
     if (x_ld % 8 || (reinterpret_cast<uintptr_t>(d_x) & 15)) return e.fail("dense_gemm: bf16 rows must be 16-byte aligned");
@@ -174,7 +231,8 @@ int zen_cuda_dev_dense_gemm(const zen_cuda_weights* w, const void* d_x, size_t x
     p.out_ld = u32(out_ld); p.rows = u32(w->rows); p.tokens = u32(tokens);
     p.k_tiles = u32((w->cols + zk::kBgK - 1) / zk::kBgK);
     p.m_tiles = u32((w->rows + zk::kBgM - 1) / zk::kBgM);
-    p.act = act; p.cap = cap; p.error_word = e.d_error;
+    p.act = ep.act; p.cap = ep.cap; p.bias = ep.d_bias; p.error_word = e.d_error;
+    p.gated = static_cast<__nv_bfloat16*>(ep.d_gated); p.gated_ld = u32(ep.gated_ld); p.pairs = u32(ep.gated_pairs);
     // the tile width that moves the fewest operand bytes through the busiest SM
     int best = 0;
     uint64_t best_cost = ~0ull;
@@ -210,13 +268,13 @@ int zen_cuda_dev_rows_view(const float* d_src, size_t src_ld, size_t n, size_t r
 }
 
 int zen_cuda_dev_head_outputs_rows(const float* d_o, size_t rows, size_t heads, size_t width, size_t head_ld, const float* d_weight, float eps, const float* d_gate,
-                                   size_t gate_ld, int gate_mode, void* d_dst, size_t ld, int bf16, void* stream) {
-    ZC_ENTER(stream, d_o && rows && rows <= 0x7fffffffu && heads && width && head_ld >= width && gate_mode >= 0 && gate_mode <= 2 && (!gate_mode || d_gate) && d_dst &&
-                         ld >= heads * width, "head_outputs_rows");
+                                   size_t gate_ld, int gate_mode, void* d_dst, size_t ld, size_t fill, int bf16, void* stream) {
+    ZC_ENTER(stream, d_o && rows && rows <= 0x7fffffffu && heads && width && head_ld >= width && gate_mode >= 0 && gate_mode <= 3 && (!gate_mode || d_gate) && d_dst &&
+                         fill >= heads * width && ld >= fill, "head_outputs_rows");
     auto go = [&](auto* dst) {
         using T = std::remove_pointer_t<decltype(dst)>;
         return launch(e, zk::head_outputs_rows_kernel<T>, dim3(u32(rows)), dim3(256), 0, d_o, u32(heads), u32(width), u32(head_ld), d_weight, eps, d_gate, u32(gate_ld),
-                      gate_mode, dst, u32(ld));
+                      gate_mode, dst, u32(ld), u32(fill));
     };
     return e.leave(bf16 ? go(static_cast<__nv_bfloat16*>(d_dst)) : go(static_cast<float*>(d_dst)), "head_outputs_rows");
 }
@@ -225,9 +283,23 @@ int zen_cuda_dev_window_attention_rows(const zen_cuda_window_attention* a, const
                                        size_t tokens, const int* d_pos, float* d_q, float* d_out, void* stream) {
     ZC_ENTER(stream, window_ok(a) && d_proj_q && d_proj_k && d_proj_v && tokens && tokens <= 65535 && d_pos && d_q && d_out, "window_attention_rows");
     const zk::AttnWindow win = device_form(*a, nullptr);
-    cudaError_t r = launch(e, zk::qk_norm_append_rows_kernel, dim3(u32(tokens)), dim3(256), 0, d_proj_q, d_proj_k, d_proj_v, u32(ld), win, a->heads, a->kv_heads, a->pitch,
-                           d_pos, d_q, a->k_cache, a->v_cache, a->max_positions, e.d_error);
-    if (!e.leave(r, "window_attention_rows: append")) return 0;
+    cudaError_t r;
+    if (is_rotary(*a)) {
+        const uint32_t items = a->heads + 2 * a->kv_heads, share = std::max(1u, std::min(64u, (items + 7) / 8));
+        r = launch(e, zk::conv_rotary_append_rows_kernel, dim3(u32((tokens + zk::kStrip - 1) / zk::kStrip), share), dim3(256), 0, d_proj_q, d_proj_k, d_proj_v, u32(ld), win,
+                   a->heads, a->kv_heads, a->pitch, u32(tokens), d_pos, d_q, a->k_cache, a->v_cache, a->max_positions, e.d_error);
+        if (!e.leave(r, "window_attention_rows: append")) return 0;
+        if (a->taps) {
+            if (d_proj_k != d_proj_q + size_t(a->heads) * a->qk_dim || d_proj_v != d_proj_k + size_t(a->kv_heads) * a->qk_dim)
+                return e.fail("window_attention_rows: the convolved q, k and v are consecutive columns");
+            r = launch(e, zk::conv_ring_update_kernel, dim3((win.rotary.conv.channels + 255) / 256), dim3(256), 0, win.rotary.conv, d_proj_q, u32(ld), u32(tokens), d_pos);
+            if (!e.leave(r, "window_attention_rows: ring")) return 0;
+        }
+    } else {
+        r = launch(e, zk::qk_norm_append_rows_kernel, dim3(u32(tokens)), dim3(256), 0, d_proj_q, d_proj_k, d_proj_v, u32(ld), win, a->heads, a->kv_heads, a->pitch,
+                   d_pos, d_q, a->k_cache, a->v_cache, a->max_positions, e.d_error);
+        if (!e.leave(r, "window_attention_rows: append")) return 0;
+    }
     const uint32_t group = a->heads / a->kv_heads;
     const int cap = a->pitch > 128 ? 2 : 4, r_heads = (cap >= 4 && group % 4 == 0) ? 4 : group % 2 == 0 ? 2 : 1;
     const size_t ctas = (tokens + zk::kPfTokens - 1) / zk::kPfTokens * a->kv_heads * (group / r_heads);
@@ -265,74 +337,75 @@ int zen_cuda_dev_window_attention_step(const zen_cuda_window_attention* a, const
                       d_out, a->heads, a->kv_heads, a->pitch, a->scale, a->window, a->max_positions, e.d_error, d_k, d_v, static_cast<const float*>(nullptr),
                       static_cast<const float*>(nullptr), 0u, a->k_cache, a->v_cache, device_form(*a, d_gate));
     };
-    return e.leave(a->pitch > 128 ? go(zk::attention_decode_kernel<true, true, true>) : go(zk::attention_decode_kernel<true, false, true>), "window_attention_step");
+    const bool wide = a->pitch > 128;
+    const cudaError_t r = is_rotary(*a) ? (wide ? go(zk::attention_decode_kernel<true, true, zk::kAttnConvRotary>) : go(zk::attention_decode_kernel<true, false, zk::kAttnConvRotary>))
+                                        : (wide ? go(zk::attention_decode_kernel<true, true, zk::kAttnNormed>) : go(zk::attention_decode_kernel<true, false, zk::kAttnNormed>));
+    return e.leave(r, "window_attention_step");
 }
 
-int zen_cuda_dev_state_step(const zen_cuda_linear_layer* l, int delta, const float* d_proj, const int* d_pos, float* d_out, void* stream) {
-    ZC_ENTER(stream, linear_ok(l, delta) && d_proj && d_pos && d_out, "state_step");
-    const zk::LinearLayer d = device_form(*l, delta);
+int zen_cuda_dev_state_step(const zen_cuda_linear_layer* l, int rule, const float* d_proj, const int* d_pos, float* d_out, void* stream) {
+    ZC_ENTER(stream, linear_ok(l, rule) && d_proj && d_pos && d_out, "state_step");
+    const zk::LinearLayer d = device_form(*l, rule);
     const bool small = d.pitch <= 128;
     auto go = [&](auto kernel, size_t smem) { return launch(e, kernel, dim3(l->heads), dim3(zk::step_threads(small ? 4 : 8)), smem, d, d_proj, d_pos, d_out); };
-    const size_t low = delta ? zk::step_low_floats(d) * sizeof(float) : 0;
-    const cudaError_t r = delta ? (small ? go(zk::state_step_kernel<true, 4>, low) : go(zk::state_step_kernel<true, 8>, low))
-                                : (small ? go(zk::state_step_kernel<false, 4>, 0) : go(zk::state_step_kernel<false, 8>, 0));
+    const size_t low = zk::step_low_floats(d) * sizeof(float);
+    auto by_size = [&](auto which) {
+        constexpr int kRule = decltype(which)::value;
+        return small ? go(zk::state_step_kernel<kRule, 4>, low) : go(zk::state_step_kernel<kRule, 8>, low);
+    };
+    const cudaError_t r = rule == ZEN_CUDA_STATE_DELTA_RULE      ? by_size(std::integral_constant<int, zk::kDeltaRule>{})
+                          : rule == ZEN_CUDA_STATE_DECAYED_WRITE ? by_size(std::integral_constant<int, zk::kDecayedWrite>{})
+                                                                 : by_size(std::integral_constant<int, zk::kGatedWrite>{});
     return e.leave(r, "state_step");
 }
 
 int zen_cuda_dev_delta_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, const float* d_decay, size_t decay_ld, size_t tokens, const int* d_pos,
                                    float* d_q, float* d_k, float* d_g, float* d_v, float* d_beta, void* stream) {
-    ZC_ENTER(stream, linear_ok(l, 1) && d_proj && d_decay && decay_ld >= size_t(l->heads) * l->dim && tokens && tokens <= 0x7fffffffu && d_pos && d_q && d_k && d_g && d_v &&
+    ZC_ENTER(stream, linear_ok(l, ZEN_CUDA_STATE_DELTA_RULE) && d_proj && d_decay && decay_ld >= size_t(l->heads) * l->dim && tokens && tokens <= 0x7fffffffu && d_pos && d_q && d_k && d_g && d_v &&
                          d_beta, "delta_inputs_rows");
-    const zk::LinearLayer d = device_form(*l, 1);
+    const zk::LinearLayer d = device_form(*l, ZEN_CUDA_STATE_DELTA_RULE);
     const uint32_t items = 2 * l->kv_heads + (l->heads * l->vdim + 31) / 32 + l->heads, share = std::max(1u, std::min(64u, (items + 15) / 16));
     const cudaError_t r = launch(e, zk::delta_inputs_rows_kernel, dim3(u32((tokens + zk::kStrip - 1) / zk::kStrip), share), dim3(256), 0, d, d_proj, u32(ld), u32(tokens),
                                  d_decay, u32(decay_ld), d_pos, d_q, d_k, d_g, d_v, d_beta);
     if (!e.leave(r, "delta_inputs_rows")) return 0;
-    return e.leave(launch(e, zk::conv_ring_update_kernel, dim3((zk::linear_channels(d) + 255) / 256), dim3(256), 0, d, d_proj, u32(ld), u32(tokens), d_pos),
+    return e.leave(launch(e, zk::conv_ring_update_kernel, dim3((d.conv.channels + 255) / 256), dim3(256), 0, d.conv, d_proj, u32(ld), u32(tokens), d_pos),
                    "delta_inputs_rows: ring");
 }
 
 int zen_cuda_dev_gated_write_inputs_rows(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, size_t tokens, float* d_q, float* d_f, void* stream) {
-    ZC_ENTER(stream, linear_ok(l, 0) && d_proj && tokens && tokens <= 0x7fffffffu && d_q && d_f, "gated_write_inputs_rows");
-    return e.leave(launch(e, zk::gated_write_inputs_rows_kernel, dim3(u32(tokens)), dim3(256), 0, device_form(*l, 0), d_proj, u32(ld), d_q, d_f), "gated_write_inputs_rows");
+    ZC_ENTER(stream, linear_ok(l, ZEN_CUDA_STATE_GATED_WRITE) && d_proj && tokens && tokens <= 0x7fffffffu && d_q && d_f, "gated_write_inputs_rows");
+    return e.leave(launch(e, zk::gated_write_inputs_rows_kernel, dim3(u32(tokens)), dim3(256), 0, device_form(*l, ZEN_CUDA_STATE_GATED_WRITE), d_proj, u32(ld), d_q, d_f), "gated_write_inputs_rows");
 }
 
-size_t zen_cuda_state_scan_workspace_bytes(const zen_cuda_linear_layer* l, int delta, size_t tokens) {
+size_t zen_cuda_state_scan_workspace_bytes(const zen_cuda_linear_layer* l, int rule, size_t tokens) {
     if (!l) return 0;
-    return (tokens + zk::kGroup - 1) / zk::kGroup * l->heads * zk::scan_record_floats(pitch32(l->dim), delta != 0) * sizeof(float);
+    return (tokens + zk::kGroup - 1) / zk::kGroup * l->heads * zk::scan_record_floats(pitch32(l->dim), rule == ZEN_CUDA_STATE_DELTA_RULE) * sizeof(float);
 }
 
-int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int delta, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld, const float* d_beta,
+int zen_cuda_dev_state_scan(const zen_cuda_linear_layer* l, int rule, const float* d_q, const float* d_k, const float* d_g, const float* d_v, size_t v_ld, const float* d_beta,
                             size_t tokens, void* d_workspace, size_t workspace_bytes, float* d_out, void* stream) {
-    ZC_ENTER(stream, linear_ok(l, delta) && d_q && d_g && d_v && v_ld >= size_t(l->heads) * l->vdim && d_out && tokens && tokens <= 0x7fffffffu && l->heads <= 65535 &&
-                         (!delta || (d_k && d_beta)) && d_workspace && !(reinterpret_cast<uintptr_t>(d_workspace) & 15) &&
-                         workspace_bytes >= zen_cuda_state_scan_workspace_bytes(l, delta, tokens), "state_scan");
-    const zk::ScanParams p{d_q, d_k, d_g, d_v, d_beta, static_cast<float*>(d_workspace), l->state, d_out, u32(tokens), l->heads, delta ? l->kv_heads : l->heads, l->vdim, u32(v_ld)};
-    const dim3 grid((l->vdim + zk::kScanColumns - 1) / zk::kScanColumns, l->heads);
-    // A grid that fits the SMs one CTA each asks for more than half an SM's shared memory: launched while the groups kernel drains,
-    // its CTAs would otherwise pile up on the first SMs to come free, and each runs for the whole block of tokens.
-    const bool spread = static_cast<uint64_t>(grid.x) * grid.y <= static_cast<uint64_t>(e.sm_count);
-    auto alone = [&](size_t smem) { return spread ? std::max(smem, e.smem_optin / 2 + 1024) : smem; };
-    auto go = [&](auto quads) {
-        constexpr int kQ = decltype(quads)::value;
-        const dim3 prepare(u32(((tokens + zk::kGroup - 1) / zk::kGroup * l->heads + 3) / 4));
-        const cudaError_t first = delta ? launch(e, zk::state_groups_kernel<kQ, true>, prepare, dim3(128), 0, p) : launch(e, zk::state_groups_kernel<kQ, false>, prepare, dim3(128), 0, p);
-        if (!e.leave(first, "state_scan: groups")) return first;
-        return delta ? launch(e, zk::state_scan_kernel<kQ, true>, grid, dim3(zk::kScanThreads), alone(zk::scan_smem_bytes<kQ, true>()), p)
-                     : launch(e, zk::state_scan_kernel<kQ, false>, grid, dim3(zk::kScanThreads), alone(zk::scan_smem_bytes<kQ, false>()), p);
-    };
-    cudaError_t r;
-    switch (pitch32(l->dim) / 32) {
-    case 1: r = go(std::integral_constant<int, 1>{}); break;
-    case 2: r = go(std::integral_constant<int, 2>{}); break;
-    case 3: r = go(std::integral_constant<int, 3>{}); break;
-    case 4: r = go(std::integral_constant<int, 4>{}); break;
-    case 5: r = go(std::integral_constant<int, 5>{}); break;
-    case 6: r = go(std::integral_constant<int, 6>{}); break;
-    case 7: r = go(std::integral_constant<int, 7>{}); break;
-    default: r = go(std::integral_constant<int, 8>{}); break;
-    }
-    return e.leave(r, "state_scan");
+    const bool delta = rule == ZEN_CUDA_STATE_DELTA_RULE;
+    ZC_ENTER(stream, linear_ok(l, rule) && rule != ZEN_CUDA_STATE_DECAYED_WRITE && d_q && d_g && d_v && v_ld >= size_t(l->heads) * l->vdim && d_out && tokens &&
+                         tokens <= 0x7fffffffu && l->heads <= 65535 && (!delta || (d_k && d_beta)) && d_workspace && !(reinterpret_cast<uintptr_t>(d_workspace) & 15) &&
+                         workspace_bytes >= zen_cuda_state_scan_workspace_bytes(l, rule, tokens), "state_scan");
+    zk::ScanParams p{};
+    p.q = d_q; p.k = d_k; p.g = d_g; p.v = d_v; p.beta = d_beta; p.records = static_cast<float*>(d_workspace); p.state = l->state; p.out = d_out;
+    p.tokens = u32(tokens); p.heads = l->heads; p.q_heads = delta ? l->kv_heads : l->heads; p.vdim = l->vdim; p.v_ld = u32(v_ld);
+    return e.leave(run_scan(e, rule, l->dim, p, device_form(*l, rule)), "state_scan");
+}
+
+int zen_cuda_dev_decayed_write_scan(const zen_cuda_linear_layer* l, const float* d_proj, size_t ld, size_t tokens, const int* d_pos, void* d_workspace,
+                                    size_t workspace_bytes, float* d_out, void* stream) {
+    constexpr int rule = ZEN_CUDA_STATE_DECAYED_WRITE;
+    ZC_ENTER(stream, linear_ok(l, rule) && d_proj && tokens && tokens <= 0x7fffffffu && l->heads <= 65535 && d_pos && d_out && d_workspace &&
+                         !(reinterpret_cast<uintptr_t>(d_workspace) & 15) && workspace_bytes >= zen_cuda_state_scan_workspace_bytes(l, rule, tokens) &&
+                         ld >= 2 * size_t(l->heads) * (l->dim + l->vdim) + (l->decay ? 0 : l->a2->cols), "decayed_write_scan");
+    const size_t nq = size_t(l->heads) * l->dim, nv = size_t(l->heads) * l->vdim;
+    zk::ScanParams p{};
+    p.q = d_proj; p.k = d_proj + nq; p.v = d_proj + 2 * nq; p.low = d_proj + 2 * nq + 2 * nv; p.pos = d_pos;
+    p.records = static_cast<float*>(d_workspace); p.state = l->state; p.out = d_out;
+    p.tokens = u32(tokens); p.heads = p.q_heads = l->heads; p.vdim = l->vdim; p.v_ld = u32(ld);
+    return e.leave(run_scan(e, rule, l->dim, p, device_form(*l, rule)), "decayed_write_scan");
 }
 
 }  // extern "C"

@@ -24,16 +24,13 @@ activation and every multiply-add is fp32 (the weights are bf16 in the file, whi
 """
 from __future__ import annotations
 
-import json
-import os
 from dataclasses import dataclass
 
 import numpy as np
 
 from . import blocks
-from .backend import DENSE_PLAIN, DENSE_SOFTCAP, DENSE_SQUARED_RELU, Backend, LinearLayer, SublayerEnd, WindowAttention
-from .decoder import Decoder
-from .safetensors import SafetensorsFile
+from .backend import (DELTA_RULE, DENSE_PLAIN, DENSE_SOFTCAP, DENSE_SQUARED_RELU, GATED_WRITE, Backend, LinearLayer, SublayerEnd, WindowAttention)
+from .dense_decoder import DenseDecoder, round_up
 
 CHANNEL_DELTA, PARALLEL = "channel_delta", "parallel"
 
@@ -123,10 +120,6 @@ class KipiraxConfig:
         return cfg
 
 
-def round_up(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
-
-
 # The rows of a mixer's input projection matrix, in order: (tensor, rows).
 def delta_rows(m: DeltaConfig, rank_a: int, rank_g: int) -> list[tuple[str, int]]:
     return [("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim), ("b", m.heads), ("a1", rank_a), ("g1", rank_g)]
@@ -162,42 +155,13 @@ def tensor_plan(cfg: KipiraxConfig, rank_a: int, rank_g: int) -> list[tuple[str,
     return plan + [("final.norm", (W,)), ("head", (cfg.vocab, W))]
 
 
-class KipiraxDecoder(Decoder):
-    """`tensor(name)` returns a tensor of the model: uint16 bfloat16 bit patterns or fp32, in its own shape."""
-
-    PREFILL_MIN = 2
+class KipiraxDecoder(DenseDecoder):
+    Config = KipiraxConfig
 
     def __init__(self, backend: Backend, cfg: KipiraxConfig, tensor, dtype: str = "bfloat16", max_positions: int | None = None, device=None) -> None:
-        if dtype not in ("bfloat16", "float32"):
-            raise ValueError(f"dtype {dtype!r}")
-        self.cfg, self.exact = cfg, dtype == "float32"
-        self._init_runtime(backend, cfg.vocab, min(max_positions or cfg.max_positions, cfg.max_positions), device)
-        self.handles: list[int] = []
-        self.layers: list[dict] = []
-        self._pf = None
+        self._init_dense(backend, cfg, tensor, dtype, min(max_positions or cfg.max_positions, cfg.max_positions), device)
+        fetch, matrix, vector = self._fetch, self._matrix, self._vector
         W, add, f32 = cfg.width, self.sequence.add, dict(dtype=self.torch.float32, device=self.dev)
-
-        def fetch(name: str, shape: tuple[int, ...] | None = None) -> np.ndarray:
-            a = tensor(name)
-            if shape is not None and tuple(a.shape) != shape:
-                raise ValueError(f"{name}: shape {tuple(a.shape)}, expected {shape}")
-            return a
-
-        def matrix(*parts: tuple[str, int], columns: int | None = None) -> int:
-            """The named tensors' rows, stacked, as one resident bf16 matrix."""
-            arrays = []
-            for name, rows in parts:
-                a = fetch(name, (rows, columns if columns is not None else W))
-                arrays.append(a if a.dtype == np.uint16 else blocks.to_bf16(a))
-            stacked = np.ascontiguousarray(arrays[0] if len(arrays) == 1 else np.concatenate(arrays))
-            h = backend.dev_upload("BF16", stacked.view(np.uint8), stacked.shape[0], stacked.shape[1])
-            self.handles.append(h)
-            return h
-
-        def vector(name: str, shape: tuple[int, ...]):
-            a = fetch(name, shape)
-            a = blocks.from_bf16(a) if a.dtype == np.uint16 else np.asarray(a, np.float32)
-            return self.torch.from_numpy(np.array(a, np.float32)).to(self.dev)
 
         self.embed = matrix(("embed", cfg.vocab))
         self.positions = matrix(("pos", cfg.max_positions))
@@ -251,14 +215,6 @@ class KipiraxDecoder(Decoder):
         self.mixed = [self.torch.zeros(mixed, **f32) for _ in range(2)]
         self.hidden = self.torch.zeros(max([L["ff"] or 1 for L in self.layers]), **f32)
 
-    @classmethod
-    def load(cls, backend: Backend, path: str, **kwargs) -> "KipiraxDecoder":
-        """A folder with config.json and model.safetensors."""
-        with open(os.path.join(path, "config.json")) as f:
-            cfg = KipiraxConfig.from_dict(json.load(f))
-        with SafetensorsFile(os.path.join(path, "model.safetensors")) as st:
-            return cls(backend, cfg, st.array, **kwargs)      # uploads complete before the mapping closes
-
     # ---- the end of a sublayer: what the next launch that reads the residual stream still has to do ----
     def _end(self, pending: dict, x_out=None, shift_of: dict | None = None, out_norm=None) -> SublayerEnd:
         P = lambda t: None if t is None else t.data_ptr()
@@ -291,10 +247,10 @@ class KipiraxDecoder(Decoder):
         for L in self.layers:
             product(L["proj"], self.proj, end=dict(shift_of=L))
             if "delta" in L:
-                be.dev_state_step(L["delta"], True, P(self.proj), P(self.pos), P(self.mixed[0]), st)
+                be.dev_state_step(L["delta"], DELTA_RULE, P(self.proj), P(self.pos), P(self.mixed[0]), st)
             else:
                 be.dev_window_attention_step(L["window"], at(L, "left.q"), at(L, "left.k"), at(L, "left.v"), at(L, "left.g"), P(self.pos), P(self.mixed[0]), st)
-                be.dev_state_step(L["write"], False, at(L, "right.q"), P(self.pos), P(self.mixed[1]), st)
+                be.dev_state_step(L["write"], GATED_WRITE, at(L, "right.q"), P(self.pos), P(self.mixed[1]), st)
             y = self.y[:len(L["o"])]
             be.dev_dense_gemv([(h, P(m), P(out)) for h, m, out in zip(L["o"], self.mixed, y)], st)
             pending = self._after_mixer(L, self.x[cur], y)
@@ -342,8 +298,8 @@ class KipiraxDecoder(Decoder):
                 # the right branch of a parallel mixer runs beside the left one
                 right_q=row(most(m.right.heads * pitch(m.right.dim) for m in pairs)), right_o=row(most(m.right.heads * m.right.vdim for m in pairs)),
                 right_mixed=torch.zeros((T, round_up(most(m.right.heads * m.right.vdim for m in pairs), 8)), **view))
-            space = lambda kind, delta: torch.zeros(most(self.be.state_scan_workspace_bytes(L[kind], delta, T) for L in self.layers if kind in L), dtype=torch.uint8, device=self.dev)
-            self._pf.update(scan=space("delta", True), right_scan=space("write", False))
+            space = lambda kind, rule: torch.zeros(most(self.be.state_scan_workspace_bytes(L[kind], rule, T) for L in self.layers if kind in L), dtype=torch.uint8, device=self.dev)
+            self._pf.update(scan=space("delta", DELTA_RULE), right_scan=space("write", GATED_WRITE))
             self.side = torch.cuda.Stream(device=self.dev)
             self._fork, self._join = torch.cuda.Event(), torch.cuda.Event()
         return self._pf
@@ -382,7 +338,7 @@ class KipiraxDecoder(Decoder):
                     be.dev_rows_view(at(n), N, rank, T, P(b["low"]), ld(rank), bf16, st)
                     gemm(handle, P(b["low"]), ld(rank), P(out), rows)
                 be.dev_delta_inputs_rows(L["delta"], P(b["proj"]), N, P(b["decay"]), m.heads * m.dim, T, P(self.pos), P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), P(b["beta"]), st)
-                be.dev_state_scan(L["delta"], True, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), width, P(b["beta"]), T, P(b["scan"]), b["scan"].numel(), P(b["o"]), st)
+                be.dev_state_scan(L["delta"], DELTA_RULE, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), width, P(b["beta"]), T, P(b["scan"]), b["scan"].numel(), P(b["o"]), st)
                 be.dev_head_outputs_rows(P(b["o"]), T, m.heads, m.vdim, m.vdim, P(b["mixed"]), ld(width), bf16, st, weight=L["delta"].norm, eps=cfg.eps,
                                          gate=P(b["gate"]), gate_ld=width, gate_mode=2)
                 gemm(L["o"][0], P(b["mixed"]), ld(width), P(b["y"][0]), W)
@@ -392,7 +348,7 @@ class KipiraxDecoder(Decoder):
                 self.side.wait_event(self._fork)
                 on_side = self.side.cuda_stream
                 be.dev_gated_write_inputs_rows(L["write"], at("right.q"), N, T, P(b["right_q"]), P(b["g"]), on_side)
-                be.dev_state_scan(L["write"], False, P(b["right_q"]), None, P(b["g"]), at("right.v"), N, None, T, P(b["right_scan"]), b["right_scan"].numel(), P(b["right_o"]), on_side)
+                be.dev_state_scan(L["write"], GATED_WRITE, P(b["right_q"]), None, P(b["g"]), at("right.v"), N, None, T, P(b["right_scan"]), b["right_scan"].numel(), P(b["right_o"]), on_side)
                 be.dev_head_outputs_rows(P(b["right_o"]), T, r.heads, r.vdim, r.vdim, P(b["right_mixed"]), ld(r.heads * r.vdim), bf16, on_side, weight=L["write"].norm, eps=cfg.eps)
                 self._join.record(self.side)
                 be.dev_window_attention_rows(L["window"], at("left.q"), at("left.k"), at("left.v"), N, T, P(self.pos), P(b["q"]), P(b["o"]), st)
@@ -415,23 +371,6 @@ class KipiraxDecoder(Decoder):
         with self.torch.cuda.stream(self.stream):      # what the head reads after a block: the last token's stream, nothing left to add
             self.x[0].copy_(b["last"][T - 1])
         self.pending = dict(x=self.x[0])
-
-    def _block_logits(self, rows: list[int]):
-        torch, st, W = self.torch, self.stream.cuda_stream, self.cfg.width
-        ld = round_up(W, 8)
-        x = self._prefill_buffers()["last"][torch.tensor(rows, device=self.dev)]
-        view = torch.zeros((len(rows), ld), dtype=torch.float32 if self.exact else torch.bfloat16, device=self.dev)
-        out = torch.zeros((len(rows), self.vocab), dtype=torch.float32, device=self.dev)
-        self.be.dev_sublayer_end_rows(self._end(dict(x=x), out_norm=self.final_norm), len(rows), view.data_ptr(), ld, not self.exact, st)
-        self.be.dev_dense_gemm(self.head, view.data_ptr(), ld, len(rows), out.data_ptr(), self.vocab, st, exact=self.exact, **self._logit_act())
-        self.stream.synchronize()      # x and view may go once the launches that read them have run
-        return out
-
-    def close(self) -> None:
-        super().close()
-        for h in self.handles:
-            self.be.dev_free(h)
-        self.handles.clear()
 
 
 def random_tensor(name: str, shape: tuple[int, ...], rng: np.random.Generator) -> np.ndarray:

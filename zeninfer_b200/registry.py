@@ -34,7 +34,12 @@ def _kipirax(backend: Backend, path: str, dtype: str, max_positions: int | None)
     return KipiraxDecoder.load(backend, path, dtype=dtype, max_positions=max_positions)
 
 
-MODELS: dict[str, Callable[[Backend, str, str, "int | None"], Decoder]] = {"llama": _llama, "Kipirax": _kipirax}
+def _sikivik(backend: Backend, path: str, dtype: str, max_positions: int | None) -> Decoder:
+    from .sikivik import SikivikDecoder
+    return SikivikDecoder.load(backend, path, dtype=dtype, max_positions=max_positions)
+
+
+MODELS: dict[str, Callable[[Backend, str, str, "int | None"], Decoder]] = {"llama": _llama, "Kipirax": _kipirax, "Sikivik": _sikivik}
 
 
 def architecture_of(path: str) -> str:
