@@ -4,6 +4,7 @@ from __future__ import annotations
 
 import numpy as np
 
+from dense_helpers import logit_error, selectors, tokens_for  # noqa: F401
 from zeninfer_b200 import blocks
 from zeninfer_b200.kipirax import KipiraxConfig, random_tensors
 
@@ -39,20 +40,6 @@ def model(name: str, seed: int = 0):
     return c, cfg, bits, {n: blocks.from_bf16(a) for n, a in bits.items()}
 
 
-def tokens_for(c: dict, n: int, seed: int = 1) -> list[int]:
-    return np.random.default_rng(seed).integers(0, c["vocab"], n).tolist()
-
-
-def selectors(rows: list[tuple[str, int]]) -> dict[str, np.ndarray]:
-    """Matrices that pick a tensor's columns out of a projection row: with them a mixer of the oracle reads the same projections
-    a kernel is given."""
-    total, at, out = sum(n for _, n in rows), 0, {}
-    for name, n in rows:
-        out[name] = np.eye(total)[at:at + n]
-        at += n
-    return out
-
-
 def standout_attention(T: int, heads: int, kv_heads: int, dim: int, vdim: int, planted: list[int], seed: int):
     """q, k, v rows in which the keys at `planted` positions match every query so well that, wherever one is visible, it decides
     the output: a mask that is one position off cannot hide.  Norm weights come with it."""
@@ -66,11 +53,3 @@ def standout_attention(T: int, heads: int, kv_heads: int, dim: int, vdim: int, p
         v[j] += 3.0 + n
     return (q.astype(np.float32), k.astype(np.float32), v.astype(np.float32),
             (1.0 + 0.1 * rng.standard_normal(dim)).astype(np.float32), (1.0 + 0.1 * rng.standard_normal(dim)).astype(np.float32))
-
-
-def logit_error(got, ref) -> float:
-    """Largest over the positions of rms(got - ref) / rms(ref), mean over the vocabulary taken off."""
-    got, ref = np.asarray(got, np.float64), np.asarray(ref, np.float64)
-    d = (got - ref) - (got - ref).mean(axis=-1, keepdims=True)
-    r = ref - ref.mean(axis=-1, keepdims=True)
-    return float((np.sqrt((d * d).mean(axis=-1)) / np.sqrt((r * r).mean())).max())

@@ -9,10 +9,12 @@ import numpy as np
 import pytest
 
 import kipirax_cases as cases
+from dense_helpers import bf16_matrix, close, dev, feed_in, host, zeros
 from oracle import kipirax as ref
 from zeninfer_b200 import blocks, safetensors
-from zeninfer_b200.backend import (DENSE_PLAIN, DENSE_SOFTCAP, DENSE_SQUARED_RELU, BackendError, LinearLayer, SublayerEnd, WindowAttention)
-from zeninfer_b200.kipirax import KipiraxDecoder, delta_rows, round_up
+from zeninfer_b200.backend import (DELTA_RULE, DENSE_PLAIN, DENSE_SOFTCAP, DENSE_SQUARED_RELU, GATED_WRITE, BackendError, LinearLayer, SublayerEnd, WindowAttention)
+from zeninfer_b200.dense_decoder import round_up
+from zeninfer_b200.kipirax import KipiraxDecoder, delta_rows
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -23,34 +25,6 @@ F32_BAR, BF16_BAR = 5e-5, 4e-2       # logit_error of a whole model in either pr
 def be():
     from zeninfer_b200 import Backend
     return Backend()
-
-
-def dev(a, dtype=np.float32):
-    import torch
-    return torch.from_numpy(np.ascontiguousarray(np.asarray(a, dtype))).cuda()
-
-
-def zeros(*shape):
-    import torch
-    return torch.zeros(shape, device="cuda")
-
-
-def host(t):
-    import torch
-    torch.cuda.synchronize()
-    return t.float().cpu().numpy()
-
-
-def bf16_matrix(be, rows, cols, seed):
-    bits = blocks.to_bf16(np.random.default_rng(seed).standard_normal((rows, cols), dtype=np.float32) * np.float32(cols ** -0.5))
-    return be.dev_upload("BF16", bits.view(np.uint8), rows, cols), blocks.from_bf16(bits).astype(np.float64)
-
-
-def close(got, want, tol=2e-5):
-    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
-    assert got.shape == want.shape and np.isfinite(got).all()
-    err = np.abs(got - want).max() / max(np.abs(want).max(), 1e-30)
-    assert err <= tol, err
 
 
 ACTS = {DENSE_PLAIN: lambda z, cap: z, DENSE_SQUARED_RELU: lambda z, cap: np.maximum(z, 0) ** 2, DENSE_SOFTCAP: lambda z, cap: cap * np.tanh(z / cap)}
@@ -248,6 +222,7 @@ def test_attention_reports_a_position_past_the_cache(be):
 
 
 # ---- mixers with a matrix state ----
+RULES = {"delta": DELTA_RULE, "write": GATED_WRITE}
 CUTS = [[75], [2, 3, 40, 7, 9], [1, 8, 16, 17], [33]]
 
 
@@ -288,7 +263,7 @@ def run_linear(be, kind, m, case, cuts):
     pitch, N = round_up(dim, 32), proj.shape[1]
     P = lambda t: t.data_ptr()
     dp, pos, got, done = dev(proj), dev([0], np.int32), np.zeros_like(want), 0
-    ws = zeros(be.state_scan_workspace_bytes(layer, kind == "delta", T) // 4)
+    ws = zeros(be.state_scan_workspace_bytes(layer, RULES[kind], T) // 4)
     q, k, gd, v, beta, o = zeros(T, g, pitch), zeros(T, g, pitch), zeros(T, h, pitch), zeros(T, h * vdim), zeros(T, h), zeros(T, h, vdim)
     y, at = zeros(T, h * vdim), {}
     col = 0
@@ -302,18 +277,18 @@ def run_linear(be, kind, m, case, cuts):
             be.dev_dense_gemm(extra["a2"], P(row) + 4 * at["a1"], N, n, P(decay), h * dim, exact=True)
             be.dev_dense_gemm(extra["g2"], P(row) + 4 * at["g1"], N, n, P(gate), h * vdim, exact=True)
             be.dev_delta_inputs_rows(layer, P(row), N, P(decay), h * dim, n, P(pos), P(q), P(k), P(gd), P(v), P(beta))
-            be.dev_state_scan(layer, True, P(q), P(k), P(gd), P(v), h * vdim, P(beta), n, P(ws), 4 * ws.numel(), P(o))
+            be.dev_state_scan(layer, DELTA_RULE, P(q), P(k), P(gd), P(v), h * vdim, P(beta), n, P(ws), 4 * ws.numel(), P(o))
             be.dev_head_outputs_rows(P(o), n, h, vdim, vdim, P(y), h * vdim, False, weight=layer.norm, eps=layer.eps, gate=P(gate), gate_ld=h * vdim, gate_mode=2)
         else:
             be.dev_gated_write_inputs_rows(layer, P(row), N, n, P(q), P(gd))
-            be.dev_state_scan(layer, False, P(q), None, P(gd), P(row) + 4 * at["v"], N, None, n, P(ws), 4 * ws.numel(), P(o))
+            be.dev_state_scan(layer, GATED_WRITE, P(q), None, P(gd), P(row) + 4 * at["v"], N, None, n, P(ws), 4 * ws.numel(), P(o))
             be.dev_head_outputs_rows(P(o), n, h, vdim, vdim, P(y), h * vdim, False, weight=layer.norm, eps=layer.eps)
         got[done:done + n] = host(y)[:n]
         done += n
         pos.fill_(done)
     one = zeros(h * vdim)
     while done < T:
-        be.dev_state_step(layer, kind == "delta", P(dp[done]), P(pos), P(one))
+        be.dev_state_step(layer, RULES[kind], P(dp[done]), P(pos), P(one))
         got[done] = host(one)
         done += 1
         pos.fill_(done)
@@ -356,10 +331,10 @@ def test_scan_keeps_a_write_far_away(be):
     P = lambda t: t.data_ptr()
     layer = LinearLayer(h, h, dim, vdim, 1, 1e-5, conv=P(dummy), a_log=P(dummy), dt_bias=P(dummy), a2=a2, g2=g2, norm=P(norm), ring=P(dummy), state=P(state))
     d = [dev(t) for t in (q, k, g, v, beta)]
-    ws = zeros(be.state_scan_workspace_bytes(layer, True, T) // 4)
-    be.dev_state_scan(layer, True, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(ws), 4 * ws.numel(), P(out))
+    ws = zeros(be.state_scan_workspace_bytes(layer, DELTA_RULE, T) // 4)
+    be.dev_state_scan(layer, DELTA_RULE, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(ws), 4 * ws.numel(), P(out))
     with pytest.raises(BackendError):
-        be.dev_state_scan(layer, True, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(ws), 4 * ws.numel() - 4, P(out))
+        be.dev_state_scan(layer, DELTA_RULE, P(d[0]), P(d[1]), P(d[2]), P(d[3]), h * vdim, P(d[4]), T, P(ws), 4 * ws.numel() - 4, P(out))
     close(host(out)[-1], v[3], 1e-4)
     be.dev_free(a2), be.dev_free(g2)
 
@@ -393,17 +368,6 @@ def decoder(be, name, dtype="float32", chunk=None, **kw):
         dec.PREFILL_CHUNK = chunk
     dec.capture()
     return c, weights, dec
-
-
-def feed_in(dec, ids, cuts):
-    """Logits after every token, fed in portions of the given sizes (the last one repeats)."""
-    dec.reset()
-    rows, done, i = [], 0, 0
-    while done < len(ids):
-        n = min(cuts[min(i, len(cuts) - 1)], len(ids) - done)
-        rows.append(dec.feed(ids[done:done + n], list(range(n))))
-        done, i = done + n, i + 1
-    return np.concatenate(rows)
 
 
 @pytest.mark.parametrize("name", sorted(cases.CASES))
