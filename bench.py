@@ -1105,38 +1105,78 @@ def kipirax_bench_config(size: dict, layers: int, positions: int) -> dict:
                 layers=[dict(type=kinds[i % 2], mixer=mixers[kinds[i % 2]], mlp=dict(kind="dense", ff=size["ff"])) for i in range(layers)])
 
 
-def run_kipirax(args) -> dict | None:
-    """Prompt and decode rates of the Kipirax decoder (bf16, random weights) at layer sizes of real models, beside the llama decoder (Q8_0,
-    its serving default) of equal width, ffn, heads and layer count; then every kernel of both alone, against its own roofline:
-    bytes over the HBM rate, or FLOPs over the bf16 rate (twice that for int8), whichever takes longer."""
-    import torch
-    from zeninfer_b200 import Backend, blocks
-    from zeninfer_b200.backend import ACT_INT8
-    from zeninfer_b200.kipirax import KipiraxConfig, KipiraxDecoder, random_tensor, tensor_plan
-    from zeninfer_b200.llama import LlamaConfig, LlamaDecoder
-    from zeninfer_b200.llama import tensor_plan as llama_plan
-    if int(os.environ.get("WORLD_SIZE", "1")) != 1:
-        raise SystemExit("--workload kipirax runs on one GPU")
-    be, dev = Backend(), torch.device("cuda", torch.cuda.current_device())
-    hbm, kind = peaks()
-    try:
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            tensor_peak = float(json.load(f)["bf16_tflops"])
-    except Exception:
-        tensor_peak = 1590.0
-    layers, prompt_len = args.layers or 4, args.prompt_len
-    steps, warm = (2, 1) if args.profile else (args.steps if args.steps != DEFAULT_STEPS else 100, max(3, args.warmup))
-    gen = torch.Generator(device=dev)
-    gen.manual_seed(11)
-    flush = torch.ones(64 << 20, dtype=torch.float32, device=dev)       # read between timed launches: evicts L2 without leaving dirty lines
+SIKIVIK_RANK = 16       # of the gla decays' projection, at every width
 
-    def throughput(dec, vocab):
+
+def sikivik_bench_config(size: dict, layers: int) -> dict:
+    H, G, D = size["heads"], size["kv_heads"], size["dim"]
+    rot = dict(base=1e5, dims=D)
+    window = dict(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, mask=dict(size=size["window"]), conv=4, rot=rot, v_mix=True)
+    kinds = [("attention", window), ("retention", dict(heads=H, dim=D, vdim=D, rot=rot, decay=[1.0 - 2.0 ** (-5.0 - 5.0 * h / H) for h in range(H)])),
+             ("attention", window), ("gla", dict(heads=H, dim=D, vdim=D, tau=16.0))]
+    return dict(architecture="Sikivik", width=size["width"], vocab=size["vocab"], norm=dict(eps=1e-6),
+                layers=[dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1], mlp=dict(kind="dense", ff=size["ff"])) for i in range(layers)])
+
+
+class DecoderBench:
+    """Rates of a decoder's prompt and steps, and its kernels one by one, each against its own roofline: bytes over the HBM rate, or
+    FLOPs over the bf16 rate (twice that for int8), whichever takes longer."""
+
+    def __init__(self, args, default_layers: int = 4) -> None:
+        import torch
+        from zeninfer_b200 import Backend
+        if int(os.environ.get("WORLD_SIZE", "1")) != 1:
+            raise SystemExit(f"--workload {args.workload} runs on one GPU")
+        self.be, self.dev, self.profile = Backend(), torch.device("cuda", torch.cuda.current_device()), args.profile
+        self.hbm, self.kind = peaks()
+        try:
+            with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+                self.tensor_peak = float(json.load(f)["bf16_tflops"])
+        except Exception:
+            self.tensor_peak = 1590.0
+        self.layers, self.prompt_len = args.layers or default_layers, args.prompt_len
+        self.steps, self.warm = (2, 1) if args.profile else (args.steps if args.steps != DEFAULT_STEPS else 100, max(3, args.warmup))
+        self.positions = self.prompt_len + self.warm + self.steps + 64
+        self.gen = torch.Generator(device=self.dev)
+        self.gen.manual_seed(11)
+        self.flush = torch.ones(64 << 20, dtype=torch.float32, device=self.dev)       # read between timed launches: evicts L2 without leaving dirty lines
+        self.labels = args.sizes.split(",") if not args.profile else ["2048"]
+
+    def weights(self, shapes: dict, random_tensor):
+        """tensor(name) of a made-up bf16 model: large matrices from the device's generator."""
+        import torch
+        from zeninfer_b200 import blocks
+        rng = np.random.default_rng(11)
+
+        def tensor(name):
+            shape = shapes[name]
+            if len(shape) == 2 and shape[0] * shape[1] > 1 << 16:
+                return (torch.randn(shape, generator=self.gen, device=self.dev) * shape[1] ** -0.5).to(torch.bfloat16).view(torch.int16).cpu().numpy().view(np.uint16)
+            return blocks.to_bf16(random_tensor(name, shape, rng))
+        return tensor
+
+    def rates(self, dec, vocab: int) -> dict:
+        pre_ms, step_ms, e2e = self.throughput(dec, vocab)
+        return {"prompt_ms": pre_ms, "prompt_tokens_per_s": self.prompt_len / pre_ms * 1e3, "decode_ms": step_ms, "decode_tokens_per_s": 1e3 / step_ms,
+                "generate_tokens_per_s": e2e}
+
+    def line(self, name: str, sizes: dict, clocks_line) -> dict:
+        top = list(sizes)[-1]
+        r = sizes[top][name.lower()]
+        return {"metric": f"{name.lower()}_decode_tokens_per_s", "value": r["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": self.steps, "warmup": self.warm,
+                "ms_per_step": r["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+                "config": {"model": f"{name} layers of width {top}, {self.layers} of them, random weights", "prompt": self.prompt_len,
+                           "l2": "kernels alone: L2 flushed before each; steps: weights larger than L2 at 4096", "peak_kind": self.kind, "hbm_gbs": self.hbm,
+                           "bf16_tflops": self.tensor_peak}, "clocks": clocks_line, "sizes": sizes}
+
+    def throughput(self, dec, vocab):
         """(prompt ms, ms per decoded token, tokens of generate() per second)"""
+        import torch
         dec.capture()
-        prompt = np.random.default_rng(6).integers(0, vocab, size=prompt_len, dtype=np.int64).tolist()
+        prompt = np.random.default_rng(6).integers(0, vocab, size=self.prompt_len, dtype=np.int64).tolist()
         with torch.cuda.stream(dec.stream):
             best = []
-            for _ in range(2 if args.profile else 5):
+            for _ in range(2 if self.profile else 5):
                 dec.reset()
                 a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
                 a.record(dec.stream)
@@ -1144,30 +1184,31 @@ def run_kipirax(args) -> dict | None:
                 b.record(dec.stream)
                 dec.stream.synchronize()
                 best.append(a.elapsed_time(b))
-            for _ in range(warm):
+            for _ in range(self.warm):
                 dec.step(want_token=True)
             a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             a.record(dec.stream)
-            for _ in range(steps):
+            for _ in range(self.steps):
                 dec.step(want_token=True)
             b.record(dec.stream)
             dec.stream.synchronize()
-        be.dev_check(dec.stream.cuda_stream)
-        step_ms = a.elapsed_time(b) / steps
-        if args.profile:
+        self.be.dev_check(dec.stream.cuda_stream)
+        step_ms = a.elapsed_time(b) / self.steps
+        if self.profile:
             return best[-1], step_ms, None
         stamps = []
         dec.generate(prompt, 33, on_token=lambda _t: stamps.append(time.perf_counter()))
         return statistics.median(best[1:]), step_ms, 32 / (stamps[-1] - stamps[0])
 
-    def alone(dec, table, rounds=20):
+    def alone(self, dec, table, rounds=20):
         """us of each launch by itself: L2 flushed before every one, median over the rounds."""
+        import torch
         out = {}
         with torch.cuda.stream(dec.stream):
             for name, (launch, nbytes, flops, rate) in table.items():
                 times = []
                 for r in range(rounds + 3):
-                    flush.sum()
+                    self.flush.sum()
                     a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
                     a.record(dec.stream)
                     launch()
@@ -1175,128 +1216,193 @@ def run_kipirax(args) -> dict | None:
                     dec.stream.synchronize()
                     times.append(a.elapsed_time(b) * 1e3)
                 us = statistics.median(times[3:])
-                roof = max(nbytes / (hbm * 1e3), flops / (rate * 1e6))
+                roof = max(nbytes / (self.hbm * 1e3), flops / (rate * 1e6))
                 out[name] = {"us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 4)}
-        be.dev_check(dec.stream.cuda_stream)
+        self.be.dev_check(dec.stream.cuda_stream)
         return out
 
-    P = lambda t: t.data_ptr()
-    sizes, clocks_line = {}, None
+    def kipirax(self, size: dict) -> dict:
+        """The Kipirax decoder at one size."""
+        import torch
+        from zeninfer_b200.backend import DELTA_RULE, GATED_WRITE
+        from zeninfer_b200.kipirax import KipiraxConfig, KipiraxDecoder, random_tensor, tensor_plan
+        be, P = self.be, lambda t: t.data_ptr()
+        W, F, H, G, D, V = (size[k] for k in ("width", "ff", "heads", "kv_heads", "dim", "vocab"))
+        cfg = KipiraxConfig.from_dict(kipirax_bench_config(size, self.layers, self.positions))
+        tensor = self.weights(dict(tensor_plan(cfg, size["rank"], size["rank"])), random_tensor)
+        dec = KipiraxDecoder(be, cfg, tensor, max_positions=self.positions)
+        entry = {**self.rates(dec, V), "weight_bytes_per_token": sum(be.dev_weight_bytes(h) for h in dec.handles[2:])}
+        if not self.profile:
+            T, b, st = dec.PREFILL_CHUNK, dec._prefill_buffers(), dec.stream.cuda_stream
+            ld_, lp = next(L for L in dec.layers if "delta" in L), next(L for L in dec.layers if "window" in L)
+            end = dec._end(dec._after_mixer(ld_, dec.x[0], dec.y[:1]), dec.x[1])
+            end_rows = dec._end(dec._after_mixer(ld_, b["x"][0], b["y"][:1]), b["x"][1])
+            proj = lambda L: L["proj_rows"] * W
+            keys = min(self.positions, size["window"])
+            state = H * D * D * 8
+            gemv = lambda h, x, y, **kw: (lambda: be.dev_dense_gemv([(h, x, y)], st, **kw))
+            gemm = lambda h, k, n, **kw: (lambda: be.dev_dense_gemm(h, P(b["hidden"]), k, T, P(b["proj"]), n, st, **kw))
+            pairs = T * (T + 1) // 2
+            table = {
+                "(smallest launch, for comparison)": (lambda: be.dev_advance_position(P(dec.pos), 0, st), 0, 0, 1),
+                "dense_gemv proj+norm+shift": (gemv(ld_["proj"], None, P(dec.proj), pre=dec._end(dec._after_mixer(ld_, dec.x[0], dec.y[:1]), dec.x[1], shift_of=lp)), 2 * proj(ld_), 0, 1),
+                "dense_gemv o": (gemv(ld_["o"][0], P(dec.mixed[0]), P(dec.y[0])), 2 * W * H * D, 0, 1),
+                "dense_gemv up+norm": (gemv(ld_["up"], None, P(dec.hidden), pre=end, act=1), 2 * W * F, 0, 1),
+                "dense_gemv down": (gemv(ld_["down"], P(dec.hidden), P(dec.y[0])), 2 * W * F, 0, 1),
+                "delta state_step": (lambda: be.dev_state_step(ld_["delta"], DELTA_RULE, P(dec.proj), P(dec.pos), P(dec.mixed[0]), st), state + 4 * H * D * size["rank"], 0, 1),
+                "gated state_step": (lambda: be.dev_state_step(lp["write"], GATED_WRITE, P(dec.proj), P(dec.pos), P(dec.mixed[1]), st), state, 0, 1),
+                "window_attention_step": (lambda: be.dev_window_attention_step(lp["window"], P(dec.proj), P(dec.proj) + 4 * H * D, P(dec.proj) + 4 * (H + G) * D, P(dec.proj),
+                                                                               P(dec.pos), P(dec.mixed[0]), st), 8 * keys * G * D, 0, 1),
+                "sublayer_end_rows": (lambda: be.dev_sublayer_end_rows(end_rows, T, P(b["h"]), W, True, st), T * W * 14, 0, 1),
+                "dense_gemm proj": (gemm(ld_["proj"], W, ld_["proj_rows"]), 2 * proj(ld_) + T * (2 * W + 4 * ld_["proj_rows"]), 2 * T * proj(ld_), self.tensor_peak),
+                "dense_gemm o": (gemm(ld_["o"][0], H * D, W), 2 * W * H * D + T * (2 * H * D + 4 * W), 2 * T * W * H * D, self.tensor_peak),
+                "dense_gemm up": (lambda: be.dev_dense_gemm(ld_["up"], P(b["h"]), W, T, P(b["hidden"]), F, st, out_bf16=True, act=1), 2 * W * F + 2 * T * (W + F), 2 * T * W * F, self.tensor_peak),
+                "dense_gemm down": (gemm(ld_["down"], F, W), 2 * W * F + T * (2 * F + 4 * W), 2 * T * W * F, self.tensor_peak),
+                "delta_inputs_rows": (lambda: be.dev_delta_inputs_rows(ld_["delta"], P(b["proj"]), ld_["proj_rows"], P(b["decay"]), H * D, T, P(dec.pos), P(b["q"]), P(b["k"]), P(b["g"]),
+                                                                       P(b["v"]), P(b["beta"]), st), T * H * D * 4 * 8, 0, 1),
+                "delta state_scan": (lambda: be.dev_state_scan(ld_["delta"], DELTA_RULE, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), H * D, P(b["beta"]), T, P(b["scan"]), b["scan"].numel(), P(b["o"]), st),
+                                     T * H * D * 4 * 5 + state, 0, 1),
+                "gated state_scan": (lambda: be.dev_state_scan(lp["write"], GATED_WRITE, P(b["q"]), None, P(b["g"]), P(b["v"]), H * D, None, T, P(b["right_scan"]), b["right_scan"].numel(), P(b["o"]), st), T * H * D * 4 * 4 + state, 0, 1),
+                "head_outputs_rows": (lambda: be.dev_head_outputs_rows(P(b["o"]), T, H, D, D, P(b["mixed"]), H * D, True, st, weight=ld_["delta"].norm, eps=1e-6, gate=P(b["gate"]),
+                                                                       gate_ld=H * D, gate_mode=2), T * H * D * 10, 0, 1),
+                "window_attention_rows (+ norms, append)": (lambda: be.dev_window_attention_rows(lp["window"], P(b["proj"]), P(b["proj"]) + 4 * H * D, P(b["proj"]) + 4 * (H + G) * D,
+                                                                                                  lp["proj_rows"], T, P(zero), P(b["q"]), P(b["o"]), st),
+                                                            T * D * 4 * (4 * H + 4 * G), 4 * pairs * H * D, self.tensor_peak),
+            }
+            zero = torch.zeros(1, dtype=torch.int32, device=self.dev)
+            dec.reset()
+            with torch.cuda.stream(dec.stream):
+                dec.pos.fill_(self.prompt_len)
+            entry["kernels"] = self.alone(dec, table)
+        dec.close()
+        return entry
+
+    def sikivik(self, size: dict) -> dict:
+        """The Sikivik decoder at one size."""
+        import torch
+        from zeninfer_b200.backend import DECAYED_WRITE
+        from zeninfer_b200.sikivik import SikivikConfig, SikivikDecoder, random_tensor, tensor_plan
+        be, P = self.be, lambda t: t.data_ptr()
+        W, F, H, G, D, V = (size[k] for k in ("width", "ff", "heads", "kv_heads", "dim", "vocab"))
+        cfg = SikivikConfig.from_dict(sikivik_bench_config(size, self.layers))
+        dec = SikivikDecoder(be, cfg, self.weights(dict(tensor_plan(cfg, SIKIVIK_RANK)), random_tensor), max_positions=self.positions)
+        entry = {**self.rates(dec, V), "weight_bytes_per_token": sum(be.dev_weight_bytes(h) for h in dec.handles[1:])}
+        if not self.profile:
+            T, b, st = dec.PREFILL_CHUNK, dec._prefill_buffers(), dec.stream.cuda_stream
+            win = next(L for L in dec.layers if L.get("values") == "mix")
+            fixed, ranked = (next(L for L in dec.layers if "state" in L and bool(L["state"].decay) == c) for c in (True, False))
+            N, inner = fixed["proj_rows"], H * D + F
+            end = dec._end(dict(x=dec.x[0], y=dec.y), dec.x[1], fixed["norm1"])
+            end_rows = dec._end(dict(x=b["x"][0], y=b["y"]), b["x"][1], fixed["norm1"])
+            keys, state, pairs = min(self.positions, size["window"]), H * D * D * 8, T * (T + 1) // 2
+            at = lambda L, x, n: P(x) + 4 * L["at"][n]
+            step = lambda L: (lambda: be.dev_state_step(L["state"], DECAYED_WRITE, P(dec.proj), P(dec.pos), P(L["inner"]), st))
+            scan = lambda L: (lambda: be.dev_decayed_write_scan(L["state"], P(b["proj"]), L["proj_rows"], T, P(dec.pos), P(b["scan"]), b["scan"].numel(), P(b["o"]), st))
+            table = {
+                "(smallest launch, for comparison)": (lambda: be.dev_advance_position(P(dec.pos), 0, st), 0, 0, 1),
+                "dense_gemv gate|up|proj+norm+swiglu": (lambda: be.dev_dense_gemv([(fixed["into"], None, P(dec.proj))], st, pre=end, gated=P(fixed["inner"]) + 4 * H * D, gated_pairs=F),
+                                                        2 * W * (N + 2 * F), 0, 1),
+                "dense_gemv o|down": (lambda: be.dev_dense_gemv([(fixed["out"], P(fixed["inner"]), P(dec.y))], st), 2 * W * inner, 0, 1),
+                "retention state_step": (step(fixed), state, 0, 1),
+                "gla state_step": (step(ranked), state + 2 * H * D * SIKIVIK_RANK, 0, 1),
+                "window_attention_step": (lambda: be.dev_window_attention_step(win["window"], at(win, dec.proj, "q"), at(win, dec.proj, "k"), at(win, dec.proj, "v"), at(win, dec.proj, "g"),
+                                                                               P(dec.pos), P(win["inner"]), st), 8 * keys * G * D, 0, 1),
+                "sublayer_end_rows": (lambda: be.dev_sublayer_end_rows(end_rows, T, P(b["h"]), W, True, st), T * W * 14, 0, 1),
+                "dense_gemm gate|up|proj+swiglu": (lambda: be.dev_dense_gemm(fixed["into"], P(b["h"]), W, T, P(b["proj"]), N, st, gated=P(b["inner"]) + 2 * H * D, gated_ld=inner,
+                                                                             gated_pairs=F), 2 * W * (N + 2 * F) + T * (2 * W + 4 * N + 2 * F), 2 * T * W * (N + 2 * F), self.tensor_peak),
+                "dense_gemm o|down": (lambda: be.dev_dense_gemm(fixed["out"], P(b["inner"]), inner, T, P(b["y"]), W, st), 2 * W * inner + T * (2 * inner + 4 * W), 2 * T * W * inner,
+                                      self.tensor_peak),
+                "retention scan": (scan(fixed), T * H * D * 4 * 4 + state, 0, 1),
+                "gla scan": (scan(ranked), T * H * D * 4 * 4 + state, 0, 1),
+                "head_outputs_rows": (lambda: be.dev_head_outputs_rows(P(b["o"]), T, H, D, D, P(b["inner"]), inner, True, st, weight=ranked["state"].norm, eps=1e-6,
+                                                                       gate=at(fixed, b["proj"], "g"), gate_ld=N, gate_mode=3, fill=H * D), T * H * D * 10, 0, 1),
+                "window_attention_rows (+ convolution, rotation, append)": (
+                    lambda: be.dev_window_attention_rows(win["window_rows"], at(win, b["proj"], "q"), at(win, b["proj"], "k"), at(win, b["proj"], "v"), win["proj_rows"], T, P(zero),
+                                                         P(b["q"]), P(b["o"]), st), T * D * 4 * (4 * H + 4 * G), 4 * pairs * H * D, self.tensor_peak),
+            }
+            zero = torch.zeros(1, dtype=torch.int32, device=self.dev)
+            dec.reset()
+            with torch.cuda.stream(dec.stream):
+                dec.pos.fill_(self.prompt_len)
+            entry["kernels"] = self.alone(dec, table)
+        dec.close()
+        return entry
+
+    def llama(self, size: dict) -> dict:
+        """The llama decoder (Q8_0, its serving default) of equal width, ffn, heads and layer count."""
+        import torch
+        from zeninfer_b200.backend import ACT_INT8
+        from zeninfer_b200.llama import LlamaConfig, LlamaDecoder
+        from zeninfer_b200.llama import tensor_plan as llama_plan
+        be, P = self.be, lambda t: t.data_ptr()
+        W, F, H, G, D, V = (size[k] for k in ("width", "ff", "heads", "kv_heads", "dim", "vocab"))
+        lcfg = LlamaConfig(embedding=W, layers=self.layers, heads=H, kv_heads=G, head_dim=D, ffn=F, vocab=V)
+
+        def llama_tensors():
+            for name, shape, is_matrix in llama_plan(lcfg):
+                w = torch.randn(shape, generator=self.gen, device=self.dev) * 0.02
+                yield (name, torch_q8_0_pack(w).cpu().numpy(), True) if is_matrix else (name, (1.0 + w).cpu().numpy(), False)
+
+        lam = LlamaDecoder(be, lcfg, llama_tensors(), act_mode=ACT_INT8, max_positions=self.positions)
+        entry = self.rates(lam, V)
+        if not self.profile:
+            T, b, st = lam.PREFILL_CHUNK, lam._prefill_buffers(), lam.stream.cuda_stream
+            h = lambda n: lam.h["blk.0." + n + ".weight"]
+            q8 = lambda n: n * 34 // 32
+            prod = lambda hs, outs, x, **kw: (lambda: be.dev_gemv_fused([h(n) for n in hs], outs, P(x), 1, ACT_INT8, st, **kw))
+            mm = lambda hs, outs, x: (lambda: be.dev_gemm_q8_0([h(n) for n in hs], [P(b[o]) for o in outs], P(b[x]), T, P(b["ws"]), b["ws_bytes"], st, act_mode=ACT_INT8))
+            norm = P(lam.norm["blk.0.attn_norm.weight"])
+            qkv = (H + 2 * G) * D
+            table = {
+                "gemv q|k|v+norm": (prod(["attn_q", "attn_k", "attn_v"], [P(lam.q), P(lam.k), P(lam.v)], lam.x, norm_weight=norm, norm_eps=1e-5), q8(W * qkv), 0, 1),
+                "gemv o": (prod(["attn_output"], [P(lam.x)], lam.att, accumulate=True), q8(W * H * D), 0, 1),
+                "gemv gate|up+norm+swiglu": (prod(["ffn_gate", "ffn_up"], [P(lam.hid), None], lam.x, norm_weight=norm, norm_eps=1e-5, swiglu_pair=True), q8(2 * W * F), 0, 1),
+                "gemv down": (prod(["ffn_down"], [P(lam.x)], lam.hid, accumulate=True), q8(W * F), 0, 1),
+                "attention_block": (lambda: be.dev_attention_block(P(lam.q), P(lam.k), P(lam.v), P(lam.cos), P(lam.sin), D // 2, P(lam.pos), P(lam.k_cache[0]), P(lam.v_cache[0]), P(lam.att),
+                                                                   H, G, D, self.positions, 0.0, 0, st), 8 * self.prompt_len * G * D, 0, 1),
+                "rms_norm rows": (lambda: be.dev_rms_norm(P(b["x"]), P(b["tmp"]), norm, P(b["xn"]), W, T, 1e-5, st), T * W * 16, 0, 1),
+                "gemm q|k|v": (mm(["attn_q", "attn_k", "attn_v"], ["q", "k", "v"], "xn"), 2 * W * qkv + T * 4 * (W + qkv), 2 * T * W * qkv, 2 * self.tensor_peak),
+                "gemm o": (mm(["attn_output"], ["tmp"], "att"), 2 * W * H * D + T * 4 * (W + H * D), 2 * T * W * H * D, 2 * self.tensor_peak),
+                "gemm gate|up": (mm(["ffn_gate", "ffn_up"], ["gate", "up"], "xn"), 4 * W * F + T * 4 * (W + 2 * F), 4 * T * W * F, 2 * self.tensor_peak),
+                "gemm down": (mm(["ffn_down"], ["tmp"], "hid"), 2 * W * F + T * 4 * (W + F), 2 * T * W * F, 2 * self.tensor_peak),
+                "rope_kv_append rows": (lambda: be.dev_rope_kv_append_rows(P(b["q"]), P(b["k"]), P(b["v"]), T, P(lam.cos), P(lam.sin), P(zero), H, G, D, D // 2, True, P(lam.k_cache[0]),
+                                                                           P(lam.v_cache[0]), self.positions, st), T * D * 4 * (2 * H + 5 * G), 0, 1),
+                "silu_mul rows": (lambda: be.dev_silu_mul(P(b["gate"]), P(b["up"]), P(b["hid"]), T * F, st), T * F * 12, 0, 1),
+                "attention_prefill": (lambda: be.dev_attention_prefill(P(b["q"]), P(lam.k_cache[0]), P(lam.v_cache[0]), P(zero), P(b["att"]), T, H, G, D, self.positions, 0.0, 0, st),
+                                      T * D * 4 * (2 * H + 2 * G), 2 * T * (T + 1) * H * D, self.tensor_peak),
+            }
+            zero = torch.zeros(1, dtype=torch.int32, device=self.dev)
+            lam.reset()
+            with torch.cuda.stream(lam.stream):
+                lam.pos.fill_(self.prompt_len)
+            entry["kernels"] = self.alone(lam, table)
+        lam.close()
+        return entry
+
+
+def run_kipirax(args) -> dict | None:
+    """Prompt and decode rates of the Kipirax decoder (bf16, random weights) at layer sizes of real models, beside the llama decoder;
+    then every kernel of both alone."""
+    bench, sizes = DecoderBench(args), {}
     with ClockSampler(0) as clocks:
         clocks.mark_start()
-        for label in (args.sizes.split(",") if not args.profile else ["2048"]):
-            size = KIPIRAX_SIZES[label]
-            W, F, H, G, D, V = (size[k] for k in ("width", "ff", "heads", "kv_heads", "dim", "vocab"))
-            positions = prompt_len + warm + steps + 64
-            cfg = KipiraxConfig.from_dict(kipirax_bench_config(size, layers, positions))
-            shapes, rng = dict(tensor_plan(cfg, size["rank"], size["rank"])), np.random.default_rng(11)
-
-            def tensor(name):
-                shape = shapes[name]
-                if len(shape) == 2 and shape[0] * shape[1] > 1 << 16:
-                    return (torch.randn(shape, generator=gen, device=dev) * shape[1] ** -0.5).to(torch.bfloat16).view(torch.int16).cpu().numpy().view(np.uint16)
-                return blocks.to_bf16(random_tensor(name, shape, rng))
-
-            dec = KipiraxDecoder(be, cfg, tensor, max_positions=positions)
-            pre_ms, step_ms, e2e = throughput(dec, V)
-            entry = {"kipirax": {"prompt_ms": pre_ms, "prompt_tokens_per_s": prompt_len / pre_ms * 1e3, "decode_ms": step_ms, "decode_tokens_per_s": 1e3 / step_ms,
-                                 "generate_tokens_per_s": e2e, "weight_bytes_per_token": sum(be.dev_weight_bytes(h) for h in dec.handles[2:])}}
-            if not args.profile:
-                T, b, st = dec.PREFILL_CHUNK, dec._prefill_buffers(), dec.stream.cuda_stream
-                ld_, lp = next(L for L in dec.layers if "delta" in L), next(L for L in dec.layers if "window" in L)
-                end = dec._end(dec._after_mixer(ld_, dec.x[0], dec.y[:1]), dec.x[1])
-                end_rows = dec._end(dec._after_mixer(ld_, b["x"][0], b["y"][:1]), b["x"][1])
-                proj = lambda L: L["proj_rows"] * W
-                keys = min(positions, size["window"])
-                state = H * D * D * 8
-                gemv = lambda h, x, y, **kw: (lambda: be.dev_dense_gemv([(h, x, y)], st, **kw))
-                gemm = lambda h, k, n, **kw: (lambda: be.dev_dense_gemm(h, P(b["hidden"]), k, T, P(b["proj"]), n, st, **kw))
-                pairs = T * (T + 1) // 2
-                table = {
-                    "(smallest launch, for comparison)": (lambda: be.dev_advance_position(P(dec.pos), 0, st), 0, 0, 1),
-                    "dense_gemv proj+norm+shift": (gemv(ld_["proj"], None, P(dec.proj), pre=dec._end(dec._after_mixer(ld_, dec.x[0], dec.y[:1]), dec.x[1], shift_of=lp)), 2 * proj(ld_), 0, 1),
-                    "dense_gemv o": (gemv(ld_["o"][0], P(dec.mixed[0]), P(dec.y[0])), 2 * W * H * D, 0, 1),
-                    "dense_gemv up+norm": (gemv(ld_["up"], None, P(dec.hidden), pre=end, act=1), 2 * W * F, 0, 1),
-                    "dense_gemv down": (gemv(ld_["down"], P(dec.hidden), P(dec.y[0])), 2 * W * F, 0, 1),
-                    "delta state_step": (lambda: be.dev_state_step(ld_["delta"], True, P(dec.proj), P(dec.pos), P(dec.mixed[0]), st), state + 4 * H * D * size["rank"], 0, 1),
-                    "gated state_step": (lambda: be.dev_state_step(lp["write"], False, P(dec.proj), P(dec.pos), P(dec.mixed[1]), st), state, 0, 1),
-                    "window_attention_step": (lambda: be.dev_window_attention_step(lp["window"], P(dec.proj), P(dec.proj) + 4 * H * D, P(dec.proj) + 4 * (H + G) * D, P(dec.proj),
-                                                                                   P(dec.pos), P(dec.mixed[0]), st), 8 * keys * G * D, 0, 1),
-                    "sublayer_end_rows": (lambda: be.dev_sublayer_end_rows(end_rows, T, P(b["h"]), W, True, st), T * W * 14, 0, 1),
-                    "dense_gemm proj": (gemm(ld_["proj"], W, ld_["proj_rows"]), 2 * proj(ld_) + T * (2 * W + 4 * ld_["proj_rows"]), 2 * T * proj(ld_), tensor_peak),
-                    "dense_gemm o": (gemm(ld_["o"][0], H * D, W), 2 * W * H * D + T * (2 * H * D + 4 * W), 2 * T * W * H * D, tensor_peak),
-                    "dense_gemm up": (lambda: be.dev_dense_gemm(ld_["up"], P(b["h"]), W, T, P(b["hidden"]), F, st, out_bf16=True, act=1), 2 * W * F + 2 * T * (W + F), 2 * T * W * F, tensor_peak),
-                    "dense_gemm down": (gemm(ld_["down"], F, W), 2 * W * F + T * (2 * F + 4 * W), 2 * T * W * F, tensor_peak),
-                    "delta_inputs_rows": (lambda: be.dev_delta_inputs_rows(ld_["delta"], P(b["proj"]), ld_["proj_rows"], P(b["decay"]), H * D, T, P(dec.pos), P(b["q"]), P(b["k"]), P(b["g"]),
-                                                                           P(b["v"]), P(b["beta"]), st), T * H * D * 4 * 8, 0, 1),
-                    "delta state_scan": (lambda: be.dev_state_scan(ld_["delta"], True, P(b["q"]), P(b["k"]), P(b["g"]), P(b["v"]), H * D, P(b["beta"]), T, P(b["scan"]), b["scan"].numel(), P(b["o"]), st),
-                                         T * H * D * 4 * 5 + state, 0, 1),
-                    "gated state_scan": (lambda: be.dev_state_scan(lp["write"], False, P(b["q"]), None, P(b["g"]), P(b["v"]), H * D, None, T, P(b["right_scan"]), b["right_scan"].numel(), P(b["o"]), st), T * H * D * 4 * 4 + state, 0, 1),
-                    "head_outputs_rows": (lambda: be.dev_head_outputs_rows(P(b["o"]), T, H, D, D, P(b["mixed"]), H * D, True, st, weight=ld_["delta"].norm, eps=1e-6, gate=P(b["gate"]),
-                                                                           gate_ld=H * D, gate_mode=2), T * H * D * 10, 0, 1),
-                    "window_attention_rows (+ norms, append)": (lambda: be.dev_window_attention_rows(lp["window"], P(b["proj"]), P(b["proj"]) + 4 * H * D, P(b["proj"]) + 4 * (H + G) * D,
-                                                                                                      lp["proj_rows"], T, P(zero), P(b["q"]), P(b["o"]), st),
-                                                                T * D * 4 * (4 * H + 4 * G), 4 * pairs * H * D, tensor_peak),
-                }
-                zero = torch.zeros(1, dtype=torch.int32, device=dev)
-                dec.reset()
-                with torch.cuda.stream(dec.stream):
-                    dec.pos.fill_(prompt_len)
-                entry["kipirax"]["kernels"] = alone(dec, table)
-            dec.close()
-            del dec
-
-            lcfg = LlamaConfig(embedding=W, layers=layers, heads=H, kv_heads=G, head_dim=D, ffn=F, vocab=V)
-
-            def llama_tensors():
-                for name, shape, is_matrix in llama_plan(lcfg):
-                    w = torch.randn(shape, generator=gen, device=dev) * 0.02
-                    yield (name, torch_q8_0_pack(w).cpu().numpy(), True) if is_matrix else (name, (1.0 + w).cpu().numpy(), False)
-
-            lam = LlamaDecoder(be, lcfg, llama_tensors(), act_mode=ACT_INT8, max_positions=positions)
-            pre_ms, step_ms, e2e = throughput(lam, V)
-            entry["llama"] = {"prompt_ms": pre_ms, "prompt_tokens_per_s": prompt_len / pre_ms * 1e3, "decode_ms": step_ms, "decode_tokens_per_s": 1e3 / step_ms, "generate_tokens_per_s": e2e}
-            if not args.profile:
-                T, b, st = lam.PREFILL_CHUNK, lam._prefill_buffers(), lam.stream.cuda_stream
-                h = lambda n: lam.h["blk.0." + n + ".weight"]
-                q8 = lambda n: n * 34 // 32
-                prod = lambda hs, outs, x, **kw: (lambda: be.dev_gemv_fused([h(n) for n in hs], outs, P(x), 1, ACT_INT8, st, **kw))
-                mm = lambda hs, outs, x: (lambda: be.dev_gemm_q8_0([h(n) for n in hs], [P(b[o]) for o in outs], P(b[x]), T, P(b["ws"]), b["ws_bytes"], st, act_mode=ACT_INT8))
-                norm = P(lam.norm["blk.0.attn_norm.weight"])
-                qkv = (H + 2 * G) * D
-                table = {
-                    "gemv q|k|v+norm": (prod(["attn_q", "attn_k", "attn_v"], [P(lam.q), P(lam.k), P(lam.v)], lam.x, norm_weight=norm, norm_eps=1e-5), q8(W * qkv), 0, 1),
-                    "gemv o": (prod(["attn_output"], [P(lam.x)], lam.att, accumulate=True), q8(W * H * D), 0, 1),
-                    "gemv gate|up+norm+swiglu": (prod(["ffn_gate", "ffn_up"], [P(lam.hid), None], lam.x, norm_weight=norm, norm_eps=1e-5, swiglu_pair=True), q8(2 * W * F), 0, 1),
-                    "gemv down": (prod(["ffn_down"], [P(lam.x)], lam.hid, accumulate=True), q8(W * F), 0, 1),
-                    "attention_block": (lambda: be.dev_attention_block(P(lam.q), P(lam.k), P(lam.v), P(lam.cos), P(lam.sin), D // 2, P(lam.pos), P(lam.k_cache[0]), P(lam.v_cache[0]), P(lam.att),
-                                                                       H, G, D, positions, 0.0, 0, st), 8 * prompt_len * G * D, 0, 1),
-                    "rms_norm rows": (lambda: be.dev_rms_norm(P(b["x"]), P(b["tmp"]), norm, P(b["xn"]), W, T, 1e-5, st), T * W * 16, 0, 1),
-                    "gemm q|k|v": (mm(["attn_q", "attn_k", "attn_v"], ["q", "k", "v"], "xn"), 2 * W * qkv + T * 4 * (W + qkv), 2 * T * W * qkv, 2 * tensor_peak),
-                    "gemm o": (mm(["attn_output"], ["tmp"], "att"), 2 * W * H * D + T * 4 * (W + H * D), 2 * T * W * H * D, 2 * tensor_peak),
-                    "gemm gate|up": (mm(["ffn_gate", "ffn_up"], ["gate", "up"], "xn"), 4 * W * F + T * 4 * (W + 2 * F), 4 * T * W * F, 2 * tensor_peak),
-                    "gemm down": (mm(["ffn_down"], ["tmp"], "hid"), 2 * W * F + T * 4 * (W + F), 2 * T * W * F, 2 * tensor_peak),
-                    "rope_kv_append rows": (lambda: be.dev_rope_kv_append_rows(P(b["q"]), P(b["k"]), P(b["v"]), T, P(lam.cos), P(lam.sin), P(zero), H, G, D, D // 2, True, P(lam.k_cache[0]),
-                                                                               P(lam.v_cache[0]), positions, st), T * D * 4 * (2 * H + 5 * G), 0, 1),
-                    "silu_mul rows": (lambda: be.dev_silu_mul(P(b["gate"]), P(b["up"]), P(b["hid"]), T * F, st), T * F * 12, 0, 1),
-                    "attention_prefill": (lambda: be.dev_attention_prefill(P(b["q"]), P(lam.k_cache[0]), P(lam.v_cache[0]), P(zero), P(b["att"]), T, H, G, D, positions, 0.0, 0, st),
-                                          T * D * 4 * (2 * H + 2 * G), 2 * T * (T + 1) * H * D, tensor_peak),
-                }
-                zero = torch.zeros(1, dtype=torch.int32, device=dev)
-                lam.reset()
-                with torch.cuda.stream(lam.stream):
-                    lam.pos.fill_(prompt_len)
-                entry["llama"]["kernels"] = alone(lam, table)
-            lam.close()
-            del lam
-            sizes[label] = entry
+        for label in bench.labels:
+            sizes[label] = {"kipirax": bench.kipirax(KIPIRAX_SIZES[label]), "llama": bench.llama(KIPIRAX_SIZES[label])}
         clocks.mark_end()
         clocks_line = clocks.summary()
-    top = list(sizes)[-1]
-    return {"metric": "kipirax_decode_tokens_per_s", "value": sizes[top]["kipirax"]["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warm,
-            "ms_per_step": sizes[top]["kipirax"]["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-            "config": {"model": f"Kipirax layers of width {top}, {layers} of them, random weights", "prompt": prompt_len, "l2": "kernels alone: L2 flushed before each; steps: weights larger than L2 at 4096",
-                       "peak_kind": kind, "hbm_gbs": hbm, "bf16_tflops": tensor_peak}, "clocks": clocks_line, "sizes": sizes}
+    return bench.line("Kipirax", sizes, clocks_line)
+
+
+def run_sikivik(args) -> dict | None:
+    """The same for the Sikivik decoder, beside the Kipirax decoder of equal width, ffn, heads and layer count."""
+    bench, sizes = DecoderBench(args), {}
+    with ClockSampler(0) as clocks:
+        clocks.mark_start()
+        for label in bench.labels:
+            sizes[label] = {"sikivik": bench.sikivik(KIPIRAX_SIZES[label]), "kipirax": bench.kipirax(KIPIRAX_SIZES[label])}
+        clocks.mark_end()
+        clocks_line = clocks.summary()
+    return bench.line("Sikivik", sizes, clocks_line)
 
 
 DEFAULT_STEPS = 20
@@ -1567,8 +1673,8 @@ def main() -> None:
                          "(peer stores over NVLink, the default) or by an NCCL all-gather launched after it")
     ap.add_argument("--fuse", default="nrp", help="workload decode: operators folded into the projection launches (letters n, s, r, p; see LlamaDecoder)")
     ap.add_argument("--token-prefill", action="store_true", help="workload decode: consume the prompt token by token instead of in tensor-core blocks")
-    ap.add_argument("--sizes", default="1024,2048,4096", help="workload kipirax: layer widths")
-    ap.add_argument("--prompt-len", type=int, default=512, help="workloads decode and kipirax: prompt tokens consumed before the timed steps")
+    ap.add_argument("--sizes", default="1024,2048,4096", help="workloads kipirax and sikivik: layer widths")
+    ap.add_argument("--prompt-len", type=int, default=512, help="workloads decode, kipirax and sikivik: prompt tokens consumed before the timed steps")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup) if args.impl != "reference" else args.warmup
     if args.profile:
@@ -1580,7 +1686,7 @@ def main() -> None:
         return
     world = int(os.environ.get("WORLD_SIZE", "1"))
     runners = {"q8_0_gemm": run_gemm_workload, "layer_sweep": run_layer_sweep, "lm_head": run_lm_head, "decode": run_decode, "gemm_formats": run_gemm_formats,
-               "kipirax": run_kipirax}
+               "kipirax": run_kipirax, "sikivik": run_sikivik}
     if args.workload in runners:
         line = runners[args.workload](args)
     elif args.workload == "q8_0_gemv":

@@ -174,33 +174,39 @@ __global__ void __cluster_dims__(kAttnSplit, 1, 1) __launch_bounds__(kAttnThread
     }
     const bool bad = pos < 0 || static_cast<uint32_t>(pos) >= max_positions;
     if constexpr (kInput == kAttnConvRotary) {
-        __shared__ __align__(16) float head[3][kAttnMaxD];        // q, k, v of this head, convolved; zero beyond their sizes
+        __shared__ __align__(16) float raw[2][kAttnMaxD], head[3][kAttnMaxD];        // q and k convolved; q, k, v of this head finished; zero beyond their sizes
         const AttnRotary& ro = win.rotary;
-        const uint32_t i = threadIdx.x, cq = h * d_q + i, ck = (heads + kh) * d_q + i, cv = (heads + kv_heads) * d_q + kh * d_v + i;
-        const bool on = !bad, owner = rank == 0 && h % (heads / kv_heads) == 0;
+        const uint32_t i = threadIdx.x, cq = h * d_q + i, ck = (heads + kh) * d_q + i, cv = (heads + kv_heads) * d_q + kh * d_v + i, half = ro.turn.half;
+        const bool owner = rank == 0 && h % (heads / kv_heads) == 0, turns = i < 2 * half, is_low = i < half;
         const int at = bad ? 0 : pos;
         float* slot = ro.conv.taps ? ro.conv.ring + static_cast<size_t>(static_cast<uint32_t>(at) % ro.conv.taps) * ro.conv.channels : nullptr;
-        float yq = 0.0f, yk = 0.0f, yv = 0.0f;
-        if (on && i < d_q) {
+        float c = 1.0f, s = 0.0f, yq = 0.0f, yk = 0.0f, yv = 0.0f;
+        if (turns) {
+            const size_t row = rotation_row(ro.turn, at) + (is_low ? i : i - half);
+            c = __ldg(ro.turn.cos_t + row);
+            s = __ldg(ro.turn.sin_t + row);
+        }
+        if (!bad && i < d_q) {
             yq = conv_sum(ro.conv, qh + i, 0, 0, at, cq);
             yk = conv_sum(ro.conv, knew + i, 0, 0, at, ck);
             if (slot && rank == 0) slot[cq] = __ldcg(qh + i);
             if (slot && owner) slot[ck] = __ldcg(knew + i);
         }
-        if (on && i < d_v) {
+        if (!bad && i < d_v) {
             yv = conv_sum(ro.conv, vnew + i, 0, 0, at, cv);
             if (ro.v_first) yv = mixed_value(yv, __ldcg(ro.v_first + kh * d_v + i), ro.share);
             if (ro.v_keep && owner) ro.v_keep[kh * d_v + i] = yv;
             if (slot && owner) slot[cv] = __ldcg(vnew + i);
         }
-        head[0][i] = yq;
-        head[1][i] = yk;
+        raw[0][i] = yq;
+        raw[1][i] = yk;
         head[2][i] = yv;
         __syncthreads();
-        const size_t row = rotation_row(ro.turn, at);
-        yq = rotated(ro.turn, [&](uint32_t d) { return head[0][d]; }, i, row);
-        yk = rotated(ro.turn, [&](uint32_t d) { return head[1][d]; }, i, row);
-        __syncthreads();
+        if (turns) {
+            const uint32_t other = is_low ? i + half : i - half;
+            yq = is_low ? rotated_low(yq, raw[0][other], c, s) : rotated_high(raw[0][other], yq, c, s);
+            yk = is_low ? rotated_low(yk, raw[1][other], c, s) : rotated_high(raw[1][other], yk, c, s);
+        }
         head[0][i] = yq;
         head[1][i] = yk;
         __syncthreads();

@@ -224,30 +224,60 @@ __global__ void __launch_bounds__(128) state_groups_kernel(const __grid_constant
         const uint32_t d = lane + 32 * j;
         float g[kGroup], k[kGroup], q[kGroup];
         if constexpr (kRule == kDecayedWrite) {
-            const bool real = d < l.dim;
+            // every load of a phase is unconditional (tokens past the block read its last one), so that all of them are in flight together
+            const bool real = d < l.dim, turns = d < 2 * l.turn.half, is_low = d < l.turn.half;
+            auto row_of = [&](int t) { return static_cast<size_t>(min(t0 + t, p.tokens - 1)) * p.v_ld + h * l.dim; };
+#pragma unroll
+            for (int t = 0; t < kGroup; ++t) {
+                q[t] = __ldcg(p.q + row_of(t) + (real ? d : 0u));
+                k[t] = __ldcg(p.k + row_of(t) + (real ? d : 0u));
+            }
+            if (l.turn.half) {
+                const uint32_t other = !turns ? 0u : is_low ? d + l.turn.half : d - l.turn.half, pair = !turns ? 0u : is_low ? d : d - l.turn.half;
+                float qo[kGroup], ko[kGroup], c[kGroup], s[kGroup];
+#pragma unroll
+                for (int t = 0; t < kGroup; ++t) {
+                    const size_t row = rotation_row(l.turn, pos + static_cast<int>(t0 + t)) + pair;
+                    qo[t] = __ldcg(p.q + row_of(t) + other);
+                    ko[t] = __ldcg(p.k + row_of(t) + other);
+                    c[t] = __ldg(l.turn.cos_t + row);
+                    s[t] = __ldg(l.turn.sin_t + row);
+                }
+#pragma unroll
+                for (int t = 0; t < kGroup; ++t) {
+                    if (!turns) continue;
+                    q[t] = is_low ? rotated_low(q[t], qo[t], c[t], s[t]) : rotated_high(qo[t], q[t], c[t], s[t]);
+                    k[t] = is_low ? rotated_low(k[t], ko[t], c[t], s[t]) : rotated_high(ko[t], k[t], c[t], s[t]);
+                }
+            }
             if (ranked) {
                 const float bias = real ? __ldg(l.dt_bias + h * l.dim + d) : 0.0f;
 #pragma unroll
                 for (int t = 0; t < kGroup; ++t) g[t] = bias;
-                const __nv_bfloat16* w = l.a2 + static_cast<size_t>(h * l.dim + d) * l.a2_ld;
-                for (uint32_t c = 0; c < low_ld; c += 8) {      // a2_ld is the rank rounded up to 8 as well
-                    const uint4 w8 = real ? __ldg(reinterpret_cast<const uint4*>(w + c)) : make_uint4(0, 0, 0, 0);
+                const __nv_bfloat16* w = l.a2 + static_cast<size_t>(h * l.dim + (real ? d : 0u)) * l.a2_ld;      // a2_ld is the rank rounded up to 8 as well
+                for (uint32_t c0 = 0; c0 < low_ld; c0 += 32) {
+                    uint4 w8[4];
 #pragma unroll
-                    for (int t = 0; t < kGroup; ++t) {
-                        const float4 x0 = *reinterpret_cast<const float4*>(low + t * low_ld + c), x1 = *reinterpret_cast<const float4*>(low + t * low_ld + c + 4);
-                        const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
-                        dense_fma8(w8, x, g[t]);
+                    for (int i = 0; i < 4; ++i) w8[i] = c0 + 8 * i < low_ld ? __ldg(reinterpret_cast<const uint4*>(w + c0 + 8 * i)) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        if (c0 + 8 * i >= low_ld) break;
+#pragma unroll
+                        for (int t = 0; t < kGroup; ++t) {
+                            const float4* x4 = reinterpret_cast<const float4*>(low + t * low_ld + c0 + 8 * i);
+                            const float4 x0 = x4[0], x1 = x4[1];
+                            const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+                            dense_fma8(w8[i], x, g[t]);
+                        }
                     }
                 }
             }
 #pragma unroll
             for (int t = 0; t < kGroup; ++t) {
                 const bool on = t0 + t < p.tokens;
-                const size_t at = static_cast<size_t>(t0 + t) * p.v_ld + h * l.dim, row = l.turn.half ? rotation_row(l.turn, pos + static_cast<int>(t0 + t)) : 0;
-                auto turned = [&](const float* x) { return on && real ? rotated(l.turn, [&](uint32_t i) { return __ldcg(x + at + i); }, d, row) : 0.0f; };
                 g[t] = !on ? 1.0f : ranked ? channel_decay(g[t], l.inv_tau) : fixed;
-                q[t] = q_scale * turned(p.q);
-                k[t] = turned(p.k);
+                q[t] = on && real ? q_scale * q[t] : 0.0f;
+                k[t] = on && real ? k[t] : 0.0f;
             }
         } else {
 #pragma unroll
